@@ -15,8 +15,8 @@ What is different here:
 * a group with a window gives a page back as soon as every key in it lies behind the
   window of the request's next token, not only when the request ends;
 * per-request fixed-size state lives in numbered *slots*: the request's token count and
-  position offset, and one tensor ``[max_requests, *shape]`` for every mixer that asks for
-  state of its own, zeroed when a slot is handed out.
+  position offset, and one tensor ``[max_requests, *shape]`` for every mixer (or the embedding) that
+  asks for state of its own, zeroed when a slot is handed out.
 """
 
 from __future__ import annotations
@@ -100,7 +100,10 @@ class RequestCache:
 
 
 class CacheManager:
-    def __init__(self, stops: Sequence[StopNeeds], num_pages: int, page_size: int, max_requests: int):
+    def __init__(self, stops: Sequence[StopNeeds], num_pages: int, page_size: int, max_requests: int,
+                 other_states: Optional[Dict[str, StateNeed]] = None):
+        """``other_states``: per-request state asked for by parts that are no schedule stop, by a name of the caller's;
+        ``states`` holds its tensor under that name."""
         if page_size <= 0 or num_pages <= 0 or max_requests <= 0:
             raise ValueError("page_size, num_pages and max_requests must be positive")
         self.page_size = int(page_size)
@@ -108,8 +111,8 @@ class CacheManager:
         self.max_requests = int(max_requests)
         self.groups: List[CacheGroup] = []
         self.location: Dict[int, Tuple[int, int]] = {}   # stop -> (group, layer within the group)
-        self.state_needs: Dict[int, StateNeed] = {}
-        self.states: Dict[int, torch.Tensor] = {}
+        self.state_needs: Dict[object, StateNeed] = dict(other_states or {})      # by stop, or by name
+        self.states: Dict[object, torch.Tensor] = {}
         by_need: Dict[KVCacheNeed, CacheGroup] = {}
         for i, s in enumerate(stops):
             if s.state is not None:

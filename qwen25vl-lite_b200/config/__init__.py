@@ -8,3 +8,4 @@ from .text_config import ConfigError, Qwen25VLTextConfig, read_config_json  # no
 from .rirulix_config import RirulixConfig  # noqa: F401
 from .labolix_config import LabolixConfig  # noqa: F401
 from .fatilix_config import FatilixConfig  # noqa: F401
+from .mezinex_config import MezinexConfig  # noqa: F401

@@ -6,7 +6,8 @@
 //   row[C .. C + R)  = rotate(x[C .. C + R))                                 (not normed)
 //
 // The attention kernels then read the row as the single kv head's key (C + R channels) and its first
-// C channels as the value.
+// C channels as the value.  Where the queries come through a latent of their own, a second kernel norms that; where the
+// heads' results are gated, a third multiplies them with the sigmoid of the token's gate channels.
 #include "rotary.cuh"
 
 template <typename T, bool EXACT>
@@ -50,3 +51,56 @@ Q25_EXPORT int q25_latent_store_bf16(const void* x, int xr, int C, int R, const 
                                      int layout, void* pages, const int* slot, int n, void* s) {
   return latent_store<bf16, false>(x, xr, C, R, w, eps, ang, half, layout, pages, slot, n, s);
 }
+
+// out[n] = x[n] / sqrt(mean(x[n]^2) + eps) * w for strided rows x of C channels, statistics in float.
+template <typename T>
+__global__ void latent_norm_kernel(const T* __restrict__ x, int x_row, int C, const float* __restrict__ w, float eps, T* __restrict__ out) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float scratch[32];
+  const T* xr = x + (size_t)blockIdx.x * x_row;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    const float v = to_f32(xr[c]);
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)C + eps);
+  T* o = out + (size_t)blockIdx.x * C;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) o[c] = from_f32<T>(to_f32(xr[c]) * inv * w[c]);
+}
+template <typename T>
+static int latent_norm(const void* x, int x_row, int C, const float* w, float eps, void* out, int n, void* stream) {
+  if (n <= 0) return 0;
+  if (C <= 0) return (int)cudaErrorInvalidValue;
+  launch(latent_norm_kernel<T>, dim3(n), dim3(C >= 512 ? 256 : 128), 0, (cudaStream_t)stream, (const T*)x, x_row, C, w, eps, (T*)out);
+  return launch_status();
+}
+Q25_EXPORT int q25_latent_norm_f32(const void* x, int xr, int C, const float* w, float eps, void* out, int n, void* s) {
+  return latent_norm<float>(x, xr, C, w, eps, out, n, s);
+}
+Q25_EXPORT int q25_latent_norm_bf16(const void* x, int xr, int C, const float* w, float eps, void* out, int n, void* s) {
+  return latent_norm<bf16>(x, xr, C, w, eps, out, n, s);
+}
+
+// y[n, c] *= sigmoid(g[n, c]), in place; y contiguous, g strided rows.
+template <typename T>
+__global__ void latent_gate_kernel(T* __restrict__ y, const T* __restrict__ g, int g_row, int channels) {
+  pdl_trigger();
+  pdl_wait();
+  const T* gr = g + (size_t)blockIdx.y * g_row;
+  T* yr = y + (size_t)blockIdx.y * channels;
+  for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < channels; c += gridDim.x * blockDim.x)
+    yr[c] = from_f32<T>(to_f32(yr[c]) / (1.0f + expf(-to_f32(gr[c]))));
+}
+template <typename T>
+static int latent_gate(void* y, const void* g, int g_row, int n, int channels, void* stream) {
+  if (n <= 0 || channels <= 0) return 0;
+  for (int at = 0; at < n; at += 65535) {                         // the grid's second dimension ends at 65,535
+    const int rows = n - at < 65535 ? n - at : 65535;
+    launch(latent_gate_kernel<T>, dim3((channels + 1023) / 1024, rows), dim3(256), 0, (cudaStream_t)stream, (T*)y + (size_t)at * channels,
+           (const T*)g + (size_t)at * g_row, g_row, channels);
+  }
+  return launch_status();
+}
+Q25_EXPORT int q25_latent_gate_f32(void* y, const void* g, int gr, int n, int ch, void* s) { return latent_gate<float>(y, g, gr, n, ch, s); }
+Q25_EXPORT int q25_latent_gate_bf16(void* y, const void* g, int gr, int n, int ch, void* s) { return latent_gate<bf16>(y, g, gr, n, ch, s); }

@@ -15,6 +15,9 @@
 // Per-request state [slots, taps, W] float: row 0 is S, rows 1 .. taps-1 are the last taps-1 inputs
 // xin of the request, oldest first (zeros at admission, which are the zeros before the start).
 //
+// A convolution on its own (causal_conv_kernel, with an optional silu, a history in a state of any layout and a result in
+// T) serves recurrences that keep their state elsewhere.
+//
 // The kernels: the convolution; the two gates of all blocks as one batched FMA product with the
 // decay and the input term formed in its epilogue; the scan in chunks over time, which also moves
 // the state on.
@@ -325,4 +328,155 @@ Q25_EXPORT int q25_rglru_scan_f32(const float* a, const float* bx, const void* y
 Q25_EXPORT int q25_rglru_scan_bf16(const float* a, const float* bx, const void* yx, int ld, int yo, int xo, float* st, const int* cu,
                                    const int* sl, void* out, int n_seqs, int max_q_len, float* sums, int w, int taps, void* s) {
   return rglru_scan<bf16>(a, bx, yx, ld, yo, xo, st, cu, sl, out, n_seqs, max_q_len, sums, w, taps, s);
+}
+
+// ---- a causal convolution per channel, on its own ----------------------------------------------------------------
+// out[n, c] = act(bias[c] + sum_j w[j, c] in_(t - (taps - 1) + j)[c]), the inputs before the step's first token from the
+// request's history [taps - 1, channels] (floats at state + slot * slot_floats, oldest first; zeros at admission), which
+// moves on.  A thread owns V channels of CONV_TOKENS consecutive tokens of an entry and slides a window over the inputs,
+// so an input is read once (and taps - 1 of them again per piece); the piece that holds the entry's first token is the
+// only reader of the history and writes the new one.  WIN: taps rounded up to a built size; the window's older places
+// carry weights of zero.
+#define CONV_TOKENS 32
+#define CONV_AHEAD 8         // inputs a thread asks for at once
+
+template <typename T, int V> struct ConvVec;
+template <> struct ConvVec<float, 1> { static __device__ __forceinline__ void load(const float* p, float* v) { v[0] = p[0]; }
+                                       static __device__ __forceinline__ void store(float* p, const float* v) { p[0] = v[0]; } };
+template <> struct ConvVec<bf16, 1> { static __device__ __forceinline__ void load(const bf16* p, float* v) { v[0] = to_f32(p[0]); }
+                                      static __device__ __forceinline__ void store(bf16* p, const float* v) { p[0] = from_f32<bf16>(v[0]); } };
+template <> struct ConvVec<float, 2> {
+  static __device__ __forceinline__ void load(const float* p, float* v) { const float2 a = *reinterpret_cast<const float2*>(p); v[0] = a.x; v[1] = a.y; }
+  static __device__ __forceinline__ void store(float* p, const float* v) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
+};
+template <> struct ConvVec<bf16, 2> {
+  static __device__ __forceinline__ void load(const bf16* p, float* v) {
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(p); v[0] = __low2float(a); v[1] = __high2float(a);
+  }
+  static __device__ __forceinline__ void store(bf16* p, const float* v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]); }
+};
+
+template <typename T, int WIN, int V>
+__global__ void __launch_bounds__(128)
+causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
+                   size_t slot_floats, const int* __restrict__ cu_q, const int* __restrict__ slot_ids, T* __restrict__ out, int out_stride,
+                   int channels, int taps, int silu) {
+  pdl_trigger();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  float wt[WIN][V], b[V];
+  if (c < channels) {                          // weights: no kernel ever writes them
+#pragma unroll
+    for (int j = 0; j < WIN; ++j)
+#pragma unroll
+      for (int v = 0; v < V; ++v) wt[j][v] = j >= WIN - taps ? w[(size_t)(j - (WIN - taps)) * channels + c + v] : 0.f;
+#pragma unroll
+    for (int v = 0; v < V; ++v) b[v] = bias[c + v];
+  }
+  pdl_wait();
+  const int seq = blockIdx.y, piece = blockIdx.z;
+  const int first = cu_q[seq], n = cu_q[seq + 1] - first;
+  const int t0 = piece * CONV_TOKENS;
+  if (c >= channels || t0 >= n) return;
+  const int t1 = min(n, t0 + CONV_TOKENS);
+  const T* x = in + (size_t)first * in_stride + c;
+  T* o = out + (size_t)first * out_stride + c;
+  float* hist = state + (size_t)slot_ids[seq] * slot_floats + c;
+  float win[WIN][V];                           // the last WIN inputs, the newest last
+#pragma unroll
+  for (int j = 0; j < WIN; ++j)
+#pragma unroll
+    for (int v = 0; v < V; ++v) win[j][v] = 0.f;
+  // places 1 .. WIN - 1 before the first token (they move down by one when it comes in)
+#pragma unroll
+  for (int j = 1; j < WIN; ++j) {
+    const int rel = t0 - WIN + j;
+    if (j > WIN - taps) {
+      if (rel >= 0) ConvVec<T, V>::load(x + (size_t)rel * in_stride, win[j]);
+      else if (piece == 0) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) win[j][v] = hist[(size_t)(taps - 1 + rel) * channels + v];
+      }
+    }
+  }
+  if (piece == 0) {
+    // the new history: the last taps - 1 of (old history, this entry's inputs).  The old rows are in the window; a row
+    // is written after the rows it may come from have been read
+    float keep[WIN > 1 ? WIN - 1 : 1][V];
+#pragma unroll
+    for (int j = 1; j < WIN; ++j) {
+      const int rel = n - WIN + j;             // the input this row will hold, by its place in the entry
+#pragma unroll
+      for (int v = 0; v < V; ++v) keep[j - 1][v] = 0.f;
+      if (j > WIN - taps) {
+        if (rel >= 0) ConvVec<T, V>::load(x + (size_t)rel * in_stride, keep[j - 1]);
+        else {
+#pragma unroll
+          for (int i = 1; i < WIN; ++i)
+            if (i == rel + WIN) {
+#pragma unroll
+              for (int v = 0; v < V; ++v) keep[j - 1][v] = win[i][v];
+            }
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 1; j < WIN; ++j)
+      if (j > WIN - taps) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) hist[(size_t)(j - 1 - (WIN - taps)) * channels + v] = keep[j - 1][v];
+      }
+  }
+  for (int t = t0; t < t1; t += CONV_AHEAD) {
+    float next[CONV_AHEAD][V];
+#pragma unroll
+    for (int a = 0; a < CONV_AHEAD; ++a) {
+      const int tt = min(t + a, t1 - 1);
+      ConvVec<T, V>::load(x + (size_t)tt * in_stride, next[a]);
+    }
+#pragma unroll
+    for (int a = 0; a < CONV_AHEAD; ++a) {
+      if (t + a < t1) {
+        float r[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+#pragma unroll
+          for (int j = 0; j + 1 < WIN; ++j) win[j][v] = win[j + 1][v];
+          win[WIN - 1][v] = next[a][v];
+          float acc = 0.f;
+#pragma unroll
+          for (int j = 0; j < WIN; ++j) acc = fmaf(wt[j][v], win[j][v], acc);
+          acc += b[v];
+          r[v] = silu ? acc / (1.0f + expf(-acc)) : acc;
+        }
+        ConvVec<T, V>::store(o + (size_t)(t + a) * out_stride, r);
+      }
+    }
+  }
+}
+
+template <typename T>
+static int causal_conv(const void* in, int in_stride, const float* w, const float* bias, float* state, long long slot_floats, const int* cu_q,
+                       const int* slot_ids, void* out, int out_stride, int n_seqs, int max_q_len, int channels, int taps, int silu, void* stream) {
+  if (n_seqs <= 0 || channels <= 0) return 0;
+  if (taps < 1 || taps > RG_MAX_TAPS || max_q_len < 1 || (taps > 1 && !state)) return (int)cudaErrorInvalidValue;
+  const int pieces = (max_q_len + CONV_TOKENS - 1) / CONV_TOKENS;
+  if (pieces > 65535 || n_seqs > 65535) return (int)cudaErrorInvalidValue;
+  const size_t pair = 2 * sizeof(T);
+  const bool two = channels % 2 == 0 && in_stride % 2 == 0 && out_stride % 2 == 0 && !((uintptr_t)in % pair) && !((uintptr_t)out % pair);
+  const int threads_c = two ? channels / 2 : channels;
+  const dim3 grid((threads_c + 127) / 128, n_seqs, pieces);
+  void (*kernel)(const T*, int, const float*, const float*, float*, size_t, const int*, const int*, T*, int, int, int, int) =
+      taps <= 4 ? (two ? causal_conv_kernel<T, 4, 2> : causal_conv_kernel<T, 4, 1>)
+                : (two ? causal_conv_kernel<T, RG_MAX_TAPS, 2> : causal_conv_kernel<T, RG_MAX_TAPS, 1>);
+  launch(kernel, grid, dim3(128), 0, (cudaStream_t)stream, (const T*)in, in_stride, w, bias, state, (size_t)slot_floats, cu_q, slot_ids, (T*)out,
+         out_stride, channels, taps, silu);
+  return launch_status();
+}
+Q25_EXPORT int q25_rglru_causal_conv_f32(const void* in, int is, const float* w, const float* b, float* st, long long sf, const int* cu, const int* sl,
+                                         void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, void* s) {
+  return causal_conv<float>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
+}
+Q25_EXPORT int q25_rglru_causal_conv_bf16(const void* in, int is, const float* w, const float* b, float* st, long long sf, const int* cu, const int* sl,
+                                          void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, void* s) {
+  return causal_conv<bf16>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
 }

@@ -107,6 +107,7 @@ class StepContext:
     group_kv_slot: List[torch.Tensor]
     group_block_table: List[torch.Tensor]
     cache: CacheManager
+    embedding_state: Optional[torch.Tensor] = None      # [max_requests, *shape], when the embedding asked for state
     # device copies of what the parts' ``plan_step`` returned, by plan key and array name
     plans: Dict[object, Dict[str, Optional[torch.Tensor]]] = field(default_factory=dict)
     # host copies, for parts written with torch operators (toy parts in tests)
@@ -169,7 +170,8 @@ class ModelRunner:
         self.model = model
         self.device = model.device
         self.dtype = model.dtype
-        self.cache = CacheManager(model.stop_needs(), num_pages, page_size, max_requests)
+        self.cache = CacheManager(model.stop_needs(), num_pages, page_size, max_requests,
+                                  model.other_state_needs() if hasattr(model, "other_state_needs") else None)
         self.cache.allocate_device(self.device, self.dtype)
         for stop in model.stops:
             stop.state = self.cache.states.get(stop.index)
@@ -569,7 +571,7 @@ class ModelRunner:
             max_kv_len=(max(widths, default=1) * ps if graph_key else max(s + n for s, n in zip(starts, q_lens))),
             group_kv_slot=[d(s_) for s_ in g_slot_s],
             group_block_table=[d(s_, (S, w)) for s_, w in zip(g_tab_s, widths)],
-            cache=self.cache,
+            cache=self.cache, embedding_state=self.cache.states.get("embedding"),
             plans=self._plan_views(plan_s, d),
             host_q_lens=q_lens, host_q_start=starts,
             host_slots=[e.request.cache.slot for e in entries] + ([pad_cache.slot] * (S - real) if S > real else []),

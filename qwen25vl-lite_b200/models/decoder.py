@@ -138,6 +138,11 @@ class DecoderModel:
             out.append(StopNeeds(mixer.cache_need(), mixer.state_need(), s.cache_of))
         return out
 
+    def other_state_needs(self) -> Dict[str, parts.StateNeed]:
+        """Per-request state of parts that are no schedule stop, by name."""
+        need = self.embedding.state_need() if hasattr(self.embedding, "state_need") else None
+        return {} if need is None else {"embedding": need}
+
     # ---- forward -----------------------------------------------------------------------
     @staticmethod
     def _add_pending(ctx, x, pending) -> None:

@@ -52,6 +52,13 @@ _SIGNATURES = {
     "q25_memory_row_dots": [_P, _P, _P, _P, _I, _I, _I, _P],
     "q25_memory_scan": [_P, _I, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "q25_memory_scan_chunked": [_P, _I, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
+    "q25_memory_ssd_scan": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
+    "q25_memory_ssd_output": [_P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P],
+    "q25_rglru_causal_conv": [_P, _I, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "q25_latent_norm": [_P, _I, _I, _P, _F, _P, _I, _P],
+    "q25_latent_gate": [_P, _P, _I, _I, _I, _P],
+    "q25_hyper_norm": [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
+    "q25_hyper_embed": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _LL, _LL, _LL, _I, _P],
     "q25_memory_output": [_P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P],
 }
 _UNTYPED = {
@@ -90,7 +97,8 @@ def load_library(name: str = "core") -> ctypes.CDLL:
 _SYMBOL_LIBRARY = (("q25_gemm_chain", "chain"), ("q25_attention_decode", "bf16"), ("q25_attention_prefill", "bf16"),
                    ("q25_gemm_tcgen05", "tcgen05"), ("q25_rope_angles", "bf16"), ("q25_rglru", "recurrent"),
                    ("q25_biased_attention", "biased"), ("q25_kv_store_mix", "biased"), ("q25_moe", "routed"),
-                   ("q25_rotary", "rotary"), ("q25_latent", "latent"), ("q25_retention", "retention"), ("q25_memory", "memory"))
+                   ("q25_rotary", "rotary"), ("q25_latent", "latent"), ("q25_retention", "retention"), ("q25_memory", "memory"),
+                   ("q25_hyper", "hyper"))
 
 
 def _library_of(symbol: str) -> str:
@@ -764,6 +772,22 @@ def rglru_scan(a: torch.Tensor, bx: torch.Tensor, yx: torch.Tensor, y_off: int, 
         count_replayed(1)                      # the chunk summaries' kernel, launched by the same call
 
 
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, history_off: int, cu_q: torch.Tensor,
+                slot_ids: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q_len: int, silu: bool) -> None:
+    """out[n, c] = act(bias[c] + sum_j weight[j, c] x_(t - (taps - 1) + j)[c]) over every entry's tokens, ``x`` a strided
+    view [N, channels], ``weight`` float32 [taps, channels].  ``state`` (float32 [slots, floats]): from ``history_off`` on a
+    slot holds the request's last taps - 1 inputs, which come before the step's first token; they move on."""
+    n, channels = out.shape
+    taps = weight.shape[0]
+    _dev(weight, torch.float32, "causal_conv weight"); _dev(bias, torch.float32, "causal_conv bias"); _dev(state, torch.float32, "causal_conv state")
+    if (x.shape != out.shape or x.stride(1) != 1 or out.stride(1) != 1 or out.dtype != x.dtype or weight.shape[1] != channels
+            or state.dim() != 2 or not 0 <= history_off <= state.shape[1] - (taps - 1) * channels):
+        raise KernelError(f"causal_conv: [N, {channels}] rows of one dtype and a slot with room for {taps - 1} rows behind {history_off}")
+    _check(_typed("q25_rglru_causal_conv", x.dtype)(
+        x.data_ptr(), x.stride(0), weight.data_ptr(), bias.data_ptr(), state.data_ptr() + 4 * int(history_off), state.shape[1], cu_q.data_ptr(),
+        slot_ids.data_ptr(), out.data_ptr(), out.stride(0), int(n_seqs), int(max_q_len), channels, taps, int(bool(silu)), _stream()), "causal_conv")
+
+
 # ---- attention with a distance bias, kept first tokens and values of their own size ---------------------
 
 
@@ -913,6 +937,22 @@ def latent_store(x: torch.Tensor, rank: int, rot: int, norm_weight: torch.Tensor
     _check(_typed("q25_latent_store", x.dtype)(x.data_ptr(), x.stride(0), rank, rot, norm_weight.data_ptr(), float(eps), _ptr(angles),
                                                half, ROTARY_LAYOUTS[layout], pages.data_ptr(), kv_slot.data_ptr(), x.shape[0],
                                                _stream()), "latent_store")
+
+
+def latent_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+    """out = rmsnorm(x) * weight for the strided rows ``x`` [N, C]."""
+    _dev(weight, torch.float32, "latent_norm weight"); _dev(out, x.dtype, "latent_norm out")
+    if x.stride(1) != 1 or out.shape != x.shape or weight.numel() != x.shape[1]:
+        raise KernelError("latent_norm: rows of one size and a weight per channel")
+    _check(_typed("q25_latent_norm", x.dtype)(x.data_ptr(), x.stride(0), x.shape[1], weight.data_ptr(), float(eps), out.data_ptr(), x.shape[0],
+                                              _stream()), "latent_norm")
+
+
+def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor) -> None:
+    """y *= sigmoid(gate), in place; ``gate`` is a strided view of y's shape."""
+    if gate.shape != y.shape or gate.dtype != y.dtype or gate.stride(1) != 1 or not y.is_contiguous():
+        raise KernelError("sigmoid_gate: a gate channel per channel of y, of its dtype")
+    _check(_typed("q25_latent_gate", y.dtype)(y.data_ptr(), gate.data_ptr(), gate.stride(0), y.shape[0], y.shape[1], _stream()), "sigmoid_gate")
 
 
 RETENTION_CHUNK = 64        # tokens of a chunk of a long run; entries up to this many tokens are walked whole
@@ -1294,3 +1334,87 @@ def memory_output(o_raw: torch.Tensor, m_exp: Optional[torch.Tensor], x: torch.T
     _check(_typed("q25_memory_output", x.dtype)(o_raw.data_ptr(), _ptr(m_exp), x.data_ptr(), x.stride(0), int(g_off), weight.data_ptr(),
                                                 out.data_ptr(), x.shape[0], heads, vdim, extra, float(eps), MEMORY_GATES[gate], _stream()),
            "memory_output")
+
+
+def ssd_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, steps: torch.Tensor, step_bias: torch.Tensor, rate_log: torch.Tensor,
+             state: torch.Tensor, cu_q: torch.Tensor, slot_ids: torch.Tensor, o_raw: torch.Tensor, n_seqs: int, heads: int, groups: int, dim: int,
+             vdim: int, first: Optional[torch.Tensor] = None, runs: Optional[torch.Tensor] = None, second: Optional[torch.Tensor] = None) -> None:
+    """Every entry's tokens in order through ``S = exp(-exp(rate_log) d) S + d k v^T``, ``o = S^T q`` per head, with
+    ``d = softplus(steps + step_bias)``: ``steps`` float32 [N, heads]; k and q of ``dim`` channels, one per group of
+    consecutive heads.  ``state`` (float32 [slots, floats]) begins with a slot's [heads, dim, vdim] and moves on.
+    ``first``, ``runs``, ``second``: the work lists of ``plan_memory`` for a step with long runs."""
+    for t in (steps, step_bias, rate_log, state, o_raw):
+        _dev(t, torch.float32, "ssd_scan")
+    if (state.dim() != 2 or state.shape[1] < heads * dim * vdim or x.stride(1) != 1 or o_raw.numel() != x.shape[0] * heads * vdim
+            or tuple(steps.shape) != (x.shape[0], heads) or heads % groups or step_bias.numel() != heads or rate_log.numel() != heads):
+        raise KernelError(f"ssd_scan: a slot begins with [{heads}, {dim}, {vdim}] floats, the steps are [N, {heads}]")
+    n_first, scratch, aux = 0, None, None
+    if first is not None:
+        for t in (first, runs, second):
+            _dev(t, torch.int32, "ssd_scan work list")
+        n_first = first.numel() // 5
+        scratch = torch.empty((n_first, heads, dim, vdim), dtype=torch.float32, device=x.device)
+        aux = torch.empty((n_first, heads, 2), dtype=torch.float32, device=x.device)
+    _check(_typed("q25_memory_ssd_scan", x.dtype)(
+        x.data_ptr(), x.stride(0), int(q_off), int(k_off), int(v_off), steps.data_ptr(), step_bias.data_ptr(), rate_log.data_ptr(), state.data_ptr(),
+        state.shape[1], cu_q.data_ptr(), slot_ids.data_ptr(), o_raw.data_ptr(), int(n_seqs), _ptr(first), n_first, _ptr(runs),
+        0 if runs is None else runs.numel() // 3, _ptr(second), 0 if second is None else second.numel() // 5, _ptr(scratch), _ptr(aux), heads, groups,
+        dim, vdim, _stream()), "ssd_scan")
+    if first is not None:
+        count_replayed(2)                      # the passes over the chunks, launched by the same call
+
+
+def ssd_output(o_raw: torch.Tensor, v: torch.Tensor, z: torch.Tensor, skip: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,
+               out: torch.Tensor, vdim: int) -> None:
+    """out = rms_in_parts((o_raw + skip[head] * v) * silu(z)) * weight: ``o_raw`` float32 [N, inner], ``v`` and ``z`` strided
+    views [N, inner], ``parts`` equal parts of a row that are each divided by their own root mean square."""
+    n, inner = out.shape
+    for t in (o_raw, skip, weight):
+        _dev(t, torch.float32, "ssd_output")
+    if (v.shape != out.shape or z.shape != out.shape or v.dtype != out.dtype or z.dtype != out.dtype or v.stride(1) != 1 or z.stride(1) != 1
+            or not out.is_contiguous() or o_raw.numel() != n * inner or weight.numel() != inner or skip.numel() * vdim != inner):
+        raise KernelError("ssd_output: values, gate and result are rows of one size, with a skip weight per head")
+    _check(_typed("q25_memory_ssd_output", out.dtype)(o_raw.data_ptr(), v.data_ptr(), v.stride(0), z.data_ptr(), z.stride(0), skip.data_ptr(),
+                                                      weight.data_ptr(), out.data_ptr(), n, inner, int(vdim), int(parts), float(eps), _stream()),
+           "ssd_output")
+
+
+# ---- a residual stream of several rows per token ---------------------------------------------------------
+
+
+def hyper_norm(x: torch.Tensor, y: Optional[torch.Tensor], mix: Optional[torch.Tensor], out_weights: Optional[torch.Tensor],
+               in_weights: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """``x`` float32 [N, streams, width].  With ``y``: x_t <- sum_s mix[s, t] x_s + out_weights[t] y first.  Then out =
+    rmsnorm(sum_s in_weights[s] x_s) * weight (in_weights None: the plain sum).  With ``rows`` only those tokens are
+    produced and x is left as it is."""
+    _dev(x, torch.float32, "hyper_norm x"); _dev(weight, torch.float32, "hyper_norm weight")
+    n, streams, width = x.shape
+    if y is not None:
+        _dev(y, out.dtype, "hyper_norm update"); _dev(mix, torch.float32, "hyper_norm mix"); _dev(out_weights, torch.float32, "hyper_norm out weights")
+        if tuple(y.shape) != (n, width) or tuple(mix.shape) != (streams, streams) or out_weights.numel() != streams:
+            raise KernelError(f"hyper_norm: the update is [N, {width}], the mixing matrix [{streams}, {streams}]")
+    if in_weights is not None:
+        _dev(in_weights, torch.float32, "hyper_norm in weights")
+    if rows is not None:
+        _dev(rows, torch.int32, "hyper_norm rows")
+    if weight.numel() != width or out.shape != (n if rows is None else rows.shape[0], width) or not out.is_contiguous():
+        raise KernelError("hyper_norm: a row of the stream's width per token")
+    _check(_typed("q25_hyper_norm", out.dtype)(x.data_ptr(), _ptr(y), _ptr(mix), _ptr(out_weights), _ptr(in_weights), weight.data_ptr(), float(eps),
+                                               out.data_ptr(), _ptr(rows), out.shape[0], streams, width, _stream()), "hyper_norm")
+
+
+def hyper_embed(table: torch.Tensor, pairs: Optional[torch.Tensor], ids: torch.Tensor, token_seq: torch.Tensor, cu_q: torch.Tensor,
+                q_start_pos: torch.Tensor, slot_ids: torch.Tensor, last_token: Optional[torch.Tensor], x: torch.Tensor, buckets: int = 0,
+                mul_prev: int = 0, mul_cur: int = 0) -> None:
+    """x[n, s, :] (float32 [N, streams, width]) = table[token] + pairs[row] for every s; row = (previous token * mul_prev +
+    token * mul_cur) mod buckets, or ``buckets`` for a request's first token.  ``last_token`` int32 [slots]: the token
+    before the step's first one of every request, which moves on."""
+    n, streams, width = x.shape
+    _dev(ids, torch.int32, "hyper_embed ids"); _dev(x, torch.float32, "hyper_embed out"); _dev(table, table.dtype, "hyper_embed table")
+    if pairs is not None:
+        _dev(pairs, table.dtype, "hyper_embed pairs"); _dev(last_token, torch.int32, "hyper_embed last tokens")
+        if tuple(pairs.shape) != (buckets + 1, width) or buckets < 1:
+            raise KernelError(f"hyper_embed: the pair table has one row more than its {buckets} buckets")
+    _check(_typed("q25_hyper_embed", table.dtype)(
+        table.data_ptr(), _ptr(pairs), ids.data_ptr(), token_seq.data_ptr(), cu_q.data_ptr(), q_start_pos.data_ptr(), slot_ids.data_ptr(),
+        _ptr(last_token), x.data_ptr(), n, width, table.shape[0], int(buckets), int(mul_prev), int(mul_cur), streams, _stream()), "hyper_embed")

@@ -380,15 +380,21 @@ class LatentAttention(Mixer):
     carried into the latent space, attention runs as H query heads over the single cached row as key
     (value: its first ``kv_rank`` channels), and ``Wuv_h`` is applied to the attended latent.  The two
     per-head products are batched products of the matrix library in bfloat16 and this engine's
-    ordered FMA product, head by head, in float32."""
+    ordered FMA product, head by head, in float32.
+
+    Two options.  ``q_rank``: the queries come through a latent too, ``q = Wuq (rmsnorm(Wdq h) * dq.norm)`` (tensors
+    ``dq``, ``dq.norm``, ``uq`` instead of ``q``).  ``out_gate``: the concatenated heads are multiplied channel by channel
+    with ``sigmoid(Wg h)`` (tensor ``g``).  Both products ride with the down projection's."""
 
     graph_safe = True                # forward is a fixed sequence of this engine's kernels and library products
     accepts_residual = True
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, value_dim: int, kv_rank: int, scale: float,
-                 norm_eps: float, window: Optional[int] = None, sink: Optional[str] = "learned", position=None):
+                 norm_eps: float, window: Optional[int] = None, sink: Optional[str] = "learned", position=None,
+                 q_rank: Optional[int] = None, out_gate: bool = False):
         if sink not in (None, "zero", "learned"):
             raise ValueError(f"sink is None, 'zero' or 'learned', got {sink!r}")
+        self.q_rank, self.out_gate = None if not q_rank else int(q_rank), bool(out_gate)
         self.hidden_size, self.num_heads, self.head_dim, self.rot_dim = int(hidden_size), int(num_heads), int(head_dim), int(rot_dim)
         self.value_dim, self.kv_rank = int(value_dim), int(kv_rank)
         if not 0 < self.kv_rank <= 512:
@@ -401,8 +407,14 @@ class LatentAttention(Mixer):
 
     def tensor_specs(self):
         h, H, D, R, Dv, C = self.hidden_size, self.num_heads, self.head_dim, self.rot_dim, self.value_dim, self.kv_rank
-        specs = [TensorSpec("q", (H * (D + R), h)), TensorSpec("dkv", (C + R, h)), TensorSpec("dkv.norm", (C,), "norm"),
-                 TensorSpec("uk", (H * D, C)), TensorSpec("uv", (H * Dv, C)), TensorSpec("o", (h, H * Dv))]
+        if self.q_rank:
+            specs = [TensorSpec("dq", (self.q_rank, h)), TensorSpec("dq.norm", (self.q_rank,), "norm"), TensorSpec("uq", (H * (D + R), self.q_rank))]
+        else:
+            specs = [TensorSpec("q", (H * (D + R), h))]
+        specs += [TensorSpec("dkv", (C + R, h)), TensorSpec("dkv.norm", (C,), "norm"), TensorSpec("uk", (H * D, C)), TensorSpec("uv", (H * Dv, C))]
+        if self.out_gate:
+            specs.append(TensorSpec("g", (H * Dv, h)))
+        specs.append(TensorSpec("o", (h, H * Dv)))
         if self.sink_kind == "learned":
             specs.append(TensorSpec("sink", (H,), "bias"))
         return tuple(specs)
@@ -412,8 +424,11 @@ class LatentAttention(Mixer):
 
     def load(self, tensors, device, dtype):
         H, D, Dv, C = self.num_heads, self.head_dim, self.value_dim, self.kv_rank
-        w = torch.cat([tensors["q"], tensors["dkv"]], dim=0)
+        w = torch.cat([tensors["dq" if self.q_rank else "q"], tensors["dkv"]] + ([tensors["g"]] if self.out_gate else []), dim=0)
         self.in_proj = Linear(w.to(device=device, dtype=dtype).contiguous())
+        if self.q_rank:
+            self.q_norm_weight = tensors["dq.norm"].to(device=device, dtype=torch.float32).contiguous()
+            self.uq_proj = Linear(tensors["uq"].to(device=device, dtype=dtype).contiguous())
         self.norm_weight = tensors["dkv.norm"].to(device=device, dtype=torch.float32).contiguous()
         # per head: [C, D], the matrix that carries a plain query into the latent space (y = x W^T with W = Wuk_h^T)
         self.uk_t = tensors["uk"].reshape(H, D, C).transpose(1, 2).to(device=device, dtype=dtype).contiguous()
@@ -439,9 +454,15 @@ class LatentAttention(Mixer):
     def forward(self, ctx, h, stop, residual=None):
         H, D, R, Dv, C = self.num_heads, self.head_dim, self.rot_dim, self.value_dim, self.kv_rank
         n = h.shape[0]
-        qd = self.in_proj(h)                                        # [N, H (D + R) | C + R]
-        q = qd[:, :H * (D + R)].unflatten(1, (H, D + R))
-        down = qd[:, H * (D + R):]
+        qd = self.in_proj(h)                                        # [N, H (D + R) or q_rank | C + R | gate]
+        q_cols = self.q_rank or H * (D + R)
+        down = qd[:, q_cols:q_cols + C + R]
+        if self.q_rank:
+            c_q = torch.empty((n, self.q_rank), dtype=qd.dtype, device=qd.device)
+            kernels.latent_norm(qd[:, :self.q_rank], self.q_norm_weight, self.norm_eps, c_q)
+            q = self.uq_proj(c_q).unflatten(1, (H, D + R))
+        else:
+            q = qd[:, :q_cols].unflatten(1, (H, D + R))
         kv = ctx.kv(stop)
         angles = self.position.angles(ctx) if self.position is not None else None
         layout = self.position.layout if self.position is not None else "interleaved"
@@ -458,4 +479,7 @@ class LatentAttention(Mixer):
                                           self.scale, None, None, self.sink, v_row=C + R)
         out = torch.empty((n, H, Dv), dtype=qd.dtype, device=qd.device)
         self._per_head(att.view(n, H, C), self.uv, out)
-        return self.o_proj(out.view(n, H * Dv), residual=residual)
+        out = out.view(n, H * Dv)
+        if self.out_gate:
+            kernels.sigmoid_gate(out, qd[:, q_cols + C + R:])
+        return self.o_proj(out, residual=residual)

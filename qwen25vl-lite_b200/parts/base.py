@@ -9,7 +9,7 @@ model configuration and does not know which model it is in.  Four things are ask
 * ``load(tensors, device, dtype)``: take those tensors (CPU views of the file) and keep
   what the kernels want on the device (fused, cast);
 * what it needs from the cache manager: pages of keys and values (``cache_need``) and / or
-  a fixed-size per-request state (``state_need``); only mixers have either;
+  a fixed-size per-request state (``state_need``); mixers may have either, the embedding a state;
 * ``forward``: see each class.
 
 Registering a class under a new kind (``MIXERS["my_kind"] = MyMixer``) is all it takes to

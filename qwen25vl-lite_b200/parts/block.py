@@ -44,3 +44,16 @@ class SandwichResidualBlock(Block):
             return mixed
         h = self.norms[2].forward(ctx, x, mixed)
         return PendingUpdate(self.feed_forward.forward(ctx, h), self.norms[3])
+
+
+@register_block("hyper_residual")
+class HyperResidualBlock(Block):
+    """Pre-norm sublayers over a stream of several rows per token (``parts.norm.HyperRMSNorm``): each sublayer's norm reads
+    the weighted sum of the rows, and its result is handed on as a ``PendingUpdate`` which the next norm's kernel writes
+    into all rows with that sublayer's connection.  A layer without a feed-forward has the mixer's norm only at work."""
+
+    def forward(self, ctx, x, pending, stop):
+        mixed = PendingUpdate(self.mixer.forward(ctx, self.norms[0].forward(ctx, x, pending), stop), self.norms[0])
+        if self.feed_forward is None:
+            return mixed
+        return PendingUpdate(self.feed_forward.forward(ctx, self.norms[1].forward(ctx, x, mixed)), self.norms[1])

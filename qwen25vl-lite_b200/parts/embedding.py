@@ -9,7 +9,7 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import Linear
-from .base import Part, TensorSpec, register_embedding, register_head
+from .base import Part, StateNeed, TensorSpec, register_embedding, register_head
 
 
 @register_embedding("token_embedding")
@@ -36,6 +36,47 @@ class TokenEmbedding(Part):
         x = torch.empty((ctx.n_tokens, self.hidden_size), dtype=torch.float32, device=self.weight.device)
         kernels.embed_gather(self.weight, ctx.token_ids, x, self.scale)
         return x
+
+
+@register_embedding("pair_embedding")
+class PairEmbedding(Part):
+    """``x = E[token] + P[(previous token * mul_prev + token * mul_cur) mod buckets]``: a token table and a hashed table of
+    token pairs, whose last row (number ``buckets``) stands for the pair of a request's first token.  ``buckets`` None: no
+    pair table.  The stream starts with ``streams`` equal rows per token ([N, streams, width]; None: [N, width]).  The token before a
+    step's first one is per-request state, so a prompt may be cut anywhere; it lives on the device, where a step that was
+    packed ahead of its token finds it.  One kernel."""
+
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+
+    def __init__(self, vocab_size: int, hidden_size: int, streams=None, buckets=None, mul_prev: int = 0, mul_cur: int = 0,
+                 names=("weight", "pairs")):
+        self.vocab_size, self.hidden_size, self.streams = int(vocab_size), int(hidden_size), None if streams is None else int(streams)
+        self.buckets, self.mul_prev, self.mul_cur = None if not buckets else int(buckets), int(mul_prev), int(mul_cur)
+        self.token_name, self.pair_name = names
+        self.weight = self.pairs = None
+
+    def tensor_specs(self):
+        specs = [TensorSpec(self.token_name, (self.vocab_size, self.hidden_size))]
+        if self.buckets:
+            specs.append(TensorSpec(self.pair_name, (self.buckets + 1, self.hidden_size)))
+        return tuple(specs)
+
+    def state_need(self):
+        return StateNeed((), "int32") if self.buckets else None
+
+    def load(self, tensors, device, dtype):
+        self.weight = tensors[self.token_name].to(device=device, dtype=dtype).contiguous()
+        if self.buckets:
+            self.pairs = tensors[self.pair_name].to(device=device, dtype=dtype).contiguous()
+
+    def exports(self):
+        return {self.token_name: self.weight}
+
+    def forward(self, ctx):
+        x = torch.empty((ctx.n_tokens, self.streams or 1, self.hidden_size), dtype=torch.float32, device=self.weight.device)
+        kernels.hyper_embed(self.weight, self.pairs, ctx.token_ids, ctx.token_seq, ctx.cu_q, ctx.q_start_pos, ctx.slot_ids, ctx.embedding_state, x,
+                            self.buckets or 0, self.mul_prev, self.mul_cur)
+        return x if self.streams is not None else x.view(ctx.n_tokens, self.hidden_size)
 
 
 @register_embedding("learned_position_embedding")

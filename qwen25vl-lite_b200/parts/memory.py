@@ -1,6 +1,6 @@
 """Mixers that keep a matrix memory per head, with gates that depend on the token.
 
-Both read ``q = Wq h * dim^(-1/2)``, ``k = Wk h`` (heads x dim), ``v = Wv h`` (heads x value_dim) and carry, per head
+The first two read ``q = Wq h * dim^(-1/2)``, ``k = Wk h`` (heads x dim), ``v = Wv h`` (heads x value_dim) and carry, per head
 and request, a float32 state ``S`` [dim, value_dim] from token to token: ``S_t = diag(a_t) S_(t-1) + b_t k_t v_t^T``,
 ``o_t = S_t^T q_t``.
 
@@ -15,9 +15,16 @@ and request, a float32 state ``S`` [dim, value_dim] from token to token: ``S_t =
   (``m_0 = 0``), ``a_t = exp(f + m_(t-1) - m_t)``, ``b_t = exp(i - m_t)``; a normaliser ``n_t = a_t n_(t-1) + b_t k_t``;
   ``o_t`` is divided by ``max(|n_t . q_t|, exp(-m_t)) + 1e-6``, then by its root mean square per head, the heads are
   concatenated, multiplied by a weight over all heads' channels and by ``sigmoid(Wg h)``, and projected by ``Wo``.
+* ``mamba2`` (Dao, Gu, "Transformers are SSMs: Generalized Models and Efficient Algorithms Through Structured State Space
+  Duality"): ``[z | x | B | C | d] = Wi h``; x, B and C pass a causal convolution per channel with bias and silu; per head
+  a step ``d_t = softplus(d + bias)``, ``a_t = exp(-exp(A_log) d_t)`` for every channel, ``b_t = d_t``, k = B and q = C
+  shared by groups of consecutive heads, v = x; ``y_t = o_t + D x_t``, the heads are concatenated, multiplied by
+  ``silu(z)``, RMS-normed in equal parts with a weight over all channels, and projected by ``Wo``.  The state keeps the
+  convolution's last inputs beside S.
 
 Float32 in both dtypes: the decays and gates from their pre-activations on (the gate rows of ``mlstm`` and the second
-factor of the decay's projection are float32 products in a fixed order), S, n, m, o and the norms.  The state is zero
+factor of the decay's projection are float32 products in a fixed order; the steps of ``mamba2`` leave their product in
+float32), S, n, m, o and the norms.  The state is zero
 at admission, so a run of tokens may be cut anywhere.  Single tokens and short runs are walked token by token; a
 long run is cut into chunks that are walked in parallel, twice, with a fold over the chunks' sums in between
 (``plan_step``).  Kernels: ``csrc/gated_memory.cu``.
@@ -153,3 +160,68 @@ class MLSTM(_MatrixMemory):
         out = torch.empty((n, H * Dv), dtype=x.dtype, device=x.device)
         kernels.memory_output(o_raw, m_exp, x, 2 * H * D + H * Dv, self.norm_weight, self.norm_eps, "sigmoid", out, H, Dv)
         return self.o_proj(out, residual=residual)
+
+
+@register_mixer("mamba2")
+class Mamba2(Mixer):
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+    accepts_residual = True          # the output projection can add into the residual stream itself
+
+    def __init__(self, hidden_size: int, num_heads: int, value_dim: int, state_dim: int, groups: int, conv: int, norm_groups: int,
+                 norm_eps: float, position=None):
+        self.hidden_size, self.num_heads, self.value_dim, self.state_dim = int(hidden_size), int(num_heads), int(value_dim), int(state_dim)
+        self.groups, self.conv, self.norm_groups, self.norm_eps = int(groups), int(conv), int(norm_groups), float(norm_eps)
+        self.inner = self.num_heads * self.value_dim
+        self.channels = self.inner + 2 * self.groups * self.state_dim      # what the convolution runs over: x | B | C
+        if self.groups < 1 or self.num_heads % self.groups:
+            raise ValueError(f"{num_heads} heads cannot share {groups} groups of B and C")
+        if self.norm_groups < 1 or self.inner % self.norm_groups:
+            raise ValueError(f"a norm over {self.inner} channels cannot be cut into {norm_groups} equal parts")
+        if not 0 < self.state_dim <= 512:
+            raise ValueError(f"a state has 1 to 512 rows, got {state_dim}")
+        if not 1 <= self.conv <= 16:
+            raise ValueError(f"the convolution takes 1 to 16 taps, got {conv}")
+        self.in_proj = self.step_proj = self.out_proj = None
+
+    def tensor_specs(self):
+        h, H, c = self.hidden_size, self.num_heads, self.channels
+        return (TensorSpec("in", (self.inner + c + H, h)), TensorSpec("conv", (c, self.conv), "matrix_wide"), TensorSpec("conv.b", (c,), "bias"),
+                TensorSpec("dt_bias", (H,), "bias"), TensorSpec("A_log", (H,), "bias"), TensorSpec("D", (H,), "norm"),
+                TensorSpec("norm", (self.inner,), "norm"), TensorSpec("o", (h, self.inner)))
+
+    @property
+    def _memory_floats(self) -> int:
+        return self.num_heads * self.state_dim * self.value_dim
+
+    def state_need(self):
+        # S [heads, state, value_dim], then the last conv - 1 inputs of the convolution [conv - 1, channels]
+        return StateNeed((self._memory_floats + (self.conv - 1) * self.channels,), "float32")
+
+    plan_key, plan_step = _MatrixMemory.plan_key, _MatrixMemory.plan_step       # the same work lists as the other memories
+
+    def load(self, tensors, device, dtype):
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        w = tensors["in"]
+        rows = self.inner + self.channels
+        # the steps' rows are a product of their own, whose result stays in float32
+        self.in_proj = Linear(w[:rows].to(device=device, dtype=dtype).contiguous())
+        self.step_proj = Linear(w[rows:].to(device=device, dtype=dtype).contiguous())
+        self.out_proj = Linear(tensors["o"].to(device=device, dtype=dtype).contiguous())
+        self.conv_w, self.conv_b = f32(tensors["conv"].t()), f32(tensors["conv.b"])            # [taps, channels]
+        self.step_bias, self.rate_log, self.skip, self.norm_weight = (f32(tensors[n]) for n in ("dt_bias", "A_log", "D", "norm"))
+
+    def forward(self, ctx, h, stop, residual=None):
+        n, inner, ch = h.shape[0], self.inner, self.channels
+        zx = self.in_proj(h)                                            # [N, z | x | B | C]
+        steps = self.step_proj(h, out_dtype=torch.float32)              # [N, heads]
+        xbc = torch.empty((n, ch), dtype=zx.dtype, device=zx.device)
+        kernels.causal_conv(zx[:, inner:], self.conv_w, self.conv_b, stop.state, self._memory_floats, ctx.cu_q, ctx.slot_ids, xbc, ctx.n_seqs,
+                            ctx.max_q_len, silu=True)
+        o_raw = torch.empty((n, inner), dtype=torch.float32, device=zx.device)
+        plan = ctx.plan(self)
+        kernels.ssd_scan(xbc, inner + self.groups * self.state_dim, inner, 0, steps, self.step_bias, self.rate_log, stop.state, ctx.cu_q,
+                         ctx.slot_ids, o_raw, ctx.n_seqs, self.num_heads, self.groups, self.state_dim, self.value_dim, plan.get("first"),
+                         plan.get("runs"), plan.get("second"))
+        out = torch.empty((n, inner), dtype=zx.dtype, device=zx.device)
+        kernels.ssd_output(o_raw, xbc[:, :inner], zx[:, :inner], self.skip, self.norm_weight, self.norm_groups, self.norm_eps, out, self.value_dim)
+        return self.out_proj(out, residual=residual)

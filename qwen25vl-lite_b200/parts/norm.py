@@ -1,4 +1,5 @@
-"""Normalisations fused with the residual update: RMS norm, Dynamic Tanh, layer norm, and no norm at all.
+"""Normalisations fused with the residual update: RMS norm (of one stream or of several), Dynamic Tanh, layer
+norm, and no norm at all.
 
 Formula (reference src/qwen25vl_lite/layers.py:27-31): ``x * rsqrt(mean(x^2) + eps) * w``,
 statistics in float32, plain (not 1 + w) weight.  With ``groups`` > 1 the vector is cut into
@@ -77,6 +78,53 @@ class RMSNorm(Norm):
                 raise TypeError("a pending update can be normalised by an rmsnorm only")
             kernels.add_norm_groups(x, delta, None if post is None else post.weight, 0.0 if post is None else post.eps,
                                     1 if post is None else post.groups, self.weight, self.eps, self.groups, out, rows)
+        return out
+
+
+@register_norm("hyper_rmsnorm")
+class HyperRMSNorm(Norm):
+    """The RMS norm of a sublayer under hyper-connections (Zhu, Huang, Huang, Zeng, Mao, Wu, Min, Zhou,
+    "Hyper-Connections"): the stream x is [N, streams, dim]; the sublayer reads the norm of ``u = sum_s in[s] x_s``, and
+    its result y enters all rows at once, ``x_t <- sum_s mix[s, t] x_s + out[t] y``.  The tensors ``in``, ``out`` and
+    ``mix`` stand under ``connection`` (relative to the part's prefix) in a checkpoint.  A block returns the sublayer's
+    result as a ``PendingUpdate`` with this norm, and the next norm's kernel does both: the write with the pending
+    update's connection, the read with its own.  ``connection`` None: the plain sum of the rows (the model's last norm,
+    which has nothing to write).  ``gain``: a constant folded into the weight."""
+
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+
+    def __init__(self, dim: int, eps: float, streams: int, name: str = "weight", connection: str = None, optional: bool = False,
+                 gain: float = 1.0):
+        self.dim, self.eps, self.streams, self.name = int(dim), float(eps), int(streams), name
+        self.connection, self.optional, self.gain = connection, bool(optional), float(gain)
+        if not 1 <= self.streams <= 16:
+            raise ValueError(f"a stream has 1 to 16 rows per token, got {streams}")
+        self.weight = self.in_weights = self.out_weights = self.mix = None
+
+    def tensor_specs(self):
+        specs, s, o = [TensorSpec(self.name, (self.dim,), init="norm", optional=self.optional)], self.streams, self.optional
+        if self.connection:
+            specs += [TensorSpec(f"{self.connection}.in", (s,), "fraction", o), TensorSpec(f"{self.connection}.out", (s,), "fraction", o),
+                      TensorSpec(f"{self.connection}.mix", (s, s), "fraction", o)]
+        return tuple(specs)
+
+    def load(self, tensors, device, dtype):
+        if self.optional and not all(ts.name in tensors for ts in self.tensor_specs()):
+            return
+        f32 = lambda name: tensors[name].to(device=device, dtype=torch.float32).contiguous()
+        self.weight = (f32(self.name) * self.gain).contiguous()
+        if self.connection:
+            self.in_weights, self.out_weights, self.mix = (f32(f"{self.connection}.{n}") for n in ("in", "out", "mix"))
+
+    def forward(self, ctx, x, delta, rows=None, defer=False):
+        back = None
+        if delta is not None:
+            if not isinstance(delta, PendingUpdate) or not isinstance(delta.norm, HyperRMSNorm) or delta.norm.mix is None:
+                raise TypeError("an update of a stream of several rows comes with the connection of its sublayer")
+            back, delta = delta.norm, delta.value
+        out = torch.empty((x.shape[0] if rows is None else rows.shape[0], self.dim), dtype=ctx.dtype, device=x.device)
+        kernels.hyper_norm(x, delta, None if back is None else back.mix, None if back is None else back.out_weights, self.in_weights, self.weight,
+                           self.eps, out, rows)
         return out
 
 
