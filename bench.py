@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Decode and prefill throughput of the engine at Qwen2.5-VL sizes, random bfloat16 weights.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 3b|7b-trace|32b|rirulix|labolix|mozutar|fatilix]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 3b|7b-trace|32b|rirulix|labolix|mozutar|fatilix|mezinex]
 
 One "step" is one decode step of the whole batch.  The default run (``--config 3b``) has the 3B
 layer sizes: the headline ``value`` is decoded tokens a second at batch 8 after 2,048-token
@@ -11,7 +11,7 @@ out every step).  The same line carries the 2,048-token prefill, the decode step
 decode at batch 1 and 64, the clocks seen while timing, and the number of this engine's kernel
 launches in the timed region.  ``--config 7b-trace`` runs a continuous-batching trace of 128
 requests at the 7B sizes, ``--config 32b`` decode at batch 1 / 8 / 32 after 8,192-token prompts and
-a 2,048-token prefill at the 32B sizes, ``--config rirulix`` / ``--config labolix`` / ``--config mozutar`` / ``--config fatilix`` prefill and decode of the Rirulix / Labolix / Mozutar / Fatilix design
+a 2,048-token prefill at the 32B sizes, ``--config rirulix`` / ``--config labolix`` / ``--config mozutar`` / ``--config fatilix`` / ``--config mezinex`` prefill and decode of the Rirulix / Labolix / Mozutar / Fatilix / Mezinex design
 at a few layer sizes beside this decoder at equal size; each prints one line of its own.
 The engine is single-GPU: for --gpus N > 1 one line says so and the exit code is 2.
 """
@@ -560,6 +560,35 @@ FATILIX_SIZES = {
 }
 
 
+def _mezinex_sizes(width, layers, ssm_heads, groups, latent_heads, latent_dim, rot_dim, kv_rank, q_rank, blocks, ff, streams, vocab):
+    """A Mezinex model of ``layers`` layers (state space, latent attention, gated linear recurrence, and so on; heads of 64
+    on a state of 128) and the Qwen2.5-VL text decoder of equal size beside it: the same width, layers, feed-forward and
+    vocabulary, heads of 128."""
+    mlp = {"kind": "dense", "ff": ff}
+    ssm = {"type": "mamba2", "mixer": {"heads": ssm_heads, "vdim": 64, "state": 128, "groups": groups, "norm_groups": groups, "conv": 4}}
+    latent = {"type": "latent_attention", "mixer": {"heads": latent_heads, "dim": latent_dim, "rot_dim": rot_dim, "vdim": latent_dim, "kv_rank": kv_rank,
+                                                    "q_rank": q_rank, "scale": (latent_dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 10000.0}}}
+    rec = {"type": "rglru", "mixer": {"width": width, "blocks": blocks, "conv": 4}}
+    ours = {"architecture": "Mezinex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": streams, "logit_scale": 1.0,
+            "embedding": {"bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 17}}, "layers": [dict((ssm, latent, rec)[i % 3], mlp=mlp) for i in range(layers)]}
+    heads = width // 128
+    closest = _sizes(width, layers, heads, max(2, heads // 8), ff, vocab, False)
+    closest["text_config"]["rope_scaling"]["mrope_section"] = [16, 24, 24]
+    return ours, closest
+
+
+MEZINEX_SIZES = {
+    "w1024": _mezinex_sizes(1024, 6, 32, 1, 8, 64, 32, 64, 256, 8, 2816, 2, 32000),
+    "w2048": _mezinex_sizes(2048, 6, 64, 1, 16, 128, 64, 128, 512, 16, 5632, 4, 32000),
+    "w2560": _mezinex_sizes(2560, 6, 80, 2, 20, 64, 32, 128, 768, 10, 6912, 4, 32000),
+}
+
+
+def run_mezinex(args):
+    """The same measurement for the Mezinex design."""
+    return _run_design(args, "Mezinex", "mezinex", MEZINEX_SIZES)
+
+
 def run_rirulix(args):
     """Prefill and decode throughput of the Rirulix design at a few layer sizes, each beside the
     Qwen2.5-VL text decoder of equal size, random weights: a 2,048-token prompt in one step, and
@@ -639,9 +668,9 @@ def main(argv=None):
     ap.add_argument("--only-batch", type=int, default=0, help="time decode steps at this batch size only (for profilers)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32 times the true 32-bit path of the 3b configuration (fewer --layers advised)")
-    ap.add_argument("--only-size", default="", help="with --config rirulix, labolix, mozutar or fatilix: one of its sizes only (for profilers)")
-    ap.add_argument("--config", default="3b", choices=["3b", "7b-trace", "32b", "rirulix", "labolix", "mozutar", "fatilix"],
-                    help="3b: the headline line (default); 7b-trace, 32b: the other workloads, one line each; rirulix, labolix, mozutar, fatilix: "
+    ap.add_argument("--only-size", default="", help="with --config rirulix, labolix, mozutar, fatilix or mezinex: one of its sizes only (for profilers)")
+    ap.add_argument("--config", default="3b", choices=["3b", "7b-trace", "32b", "rirulix", "labolix", "mozutar", "fatilix", "mezinex"],
+                    help="3b: the headline line (default); 7b-trace, 32b: the other workloads, one line each; rirulix, labolix, mozutar, fatilix, mezinex: "
                          "that design at a few layer sizes beside the Qwen2.5-VL decoder of equal size")
     args = ap.parse_args(argv)
     if args.gpus != 1:
@@ -654,7 +683,7 @@ def main(argv=None):
             print(json.dumps({"impl": "reference", "unavailable": "the reference arm measures the 3b configuration only"}))
             return 0
         return run_reference(args)
-    return {"3b": run_ours, "7b-trace": run_7b_trace, "32b": run_32b, "rirulix": run_rirulix, "labolix": run_labolix, "mozutar": run_mozutar, "fatilix": run_fatilix}[args.config](args)
+    return {"3b": run_ours, "7b-trace": run_7b_trace, "32b": run_32b, "rirulix": run_rirulix, "labolix": run_labolix, "mozutar": run_mozutar, "fatilix": run_fatilix, "mezinex": run_mezinex}[args.config](args)
 
 
 if __name__ == "__main__":

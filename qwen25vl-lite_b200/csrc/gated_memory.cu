@@ -571,7 +571,8 @@ Q25_EXPORT int q25_memory_output_bf16(const float* o, const float* me, const voi
 }
 
 // The state space of Mamba-2 by the same walk: x holds the values (heads side by side at v_off) and, per group of heads, k
-// and q; raw steps z [N, H] float.  first == nullptr: every entry is walked whole; else the chunked passes.
+// and q; raw steps z [N, H] float.  first == nullptr: every entry is walked whole, or with `second` what that lists; else the
+// chunked passes.
 template <typename T>
 static int ssd_scan(const void* x, int x_stride, int q_off, int k_off, int v_off, const float* z, const float* step_bias, const float* rate_log,
                     float* state, long long slot_floats, const int* cu_q, const int* slot_ids, float* o_raw, int n_seqs, const int* first,
@@ -585,7 +586,10 @@ static int ssd_scan(const void* x, int x_stride, int q_off, int k_off, int v_off
   p.step_bias = step_bias; p.rate_log = rate_log; p.q_scale = 1.f; p.state = state; p.slot_floats = (size_t)slot_floats; p.share = H / groups;
   p.cu_q = cu_q; p.slot_ids = slot_ids; p.o_raw = o_raw; p.m_exp = nullptr; p.H = H; p.D = D; p.Dv = Dv; p.extra = 0;
   p.items = nullptr; p.scratch = scratch; p.aux = aux;
-  if (!first) return memory_scan_rows<T, false>(p, n_seqs, (cudaStream_t)stream);
+  if (!first) {
+    p.items = second;
+    return memory_scan_rows<T, false>(p, second ? n_second : n_seqs, (cudaStream_t)stream);
+  }
   return memory_chunked_passes<T>(p, first, n_first, runs, n_runs, second, n_second, (cudaStream_t)stream);
 }
 Q25_EXPORT int q25_memory_ssd_scan_f32(const void* x, int xs, int qo, int ko, int vo, const float* z, const float* sb, const float* rl, float* state,

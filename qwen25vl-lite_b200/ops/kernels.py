@@ -98,7 +98,7 @@ _SYMBOL_LIBRARY = (("q25_gemm_chain", "chain"), ("q25_attention_decode", "bf16")
                    ("q25_gemm_tcgen05", "tcgen05"), ("q25_rope_angles", "bf16"), ("q25_rglru", "recurrent"),
                    ("q25_biased_attention", "biased"), ("q25_kv_store_mix", "biased"), ("q25_moe", "routed"),
                    ("q25_rotary", "rotary"), ("q25_latent", "latent"), ("q25_retention", "retention"), ("q25_memory", "memory"),
-                   ("q25_hyper", "hyper"))
+                   ("q25_hyper", "hyper"), ("q25_state_space", "state_space"))
 
 
 def _library_of(symbol: str) -> str:
@@ -1342,7 +1342,8 @@ def ssd_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, steps: torch.T
     """Every entry's tokens in order through ``S = exp(-exp(rate_log) d) S + d k v^T``, ``o = S^T q`` per head, with
     ``d = softplus(steps + step_bias)``: ``steps`` float32 [N, heads]; k and q of ``dim`` channels, one per group of
     consecutive heads.  ``state`` (float32 [slots, floats]) begins with a slot's [heads, dim, vdim] and moves on.
-    ``first``, ``runs``, ``second``: the work lists of ``plan_memory`` for a step with long runs."""
+    ``first``, ``runs``, ``second``: the work lists of ``plan_memory`` for a step with long runs; ``second`` alone: only the
+    entries it lists are walked."""
     for t in (steps, step_bias, rate_log, state, o_raw):
         _dev(t, torch.float32, "ssd_scan")
     if (state.dim() != 2 or state.shape[1] < heads * dim * vdim or x.stride(1) != 1 or o_raw.numel() != x.shape[0] * heads * vdim
@@ -1362,6 +1363,32 @@ def ssd_scan(x: torch.Tensor, q_off: int, k_off: int, v_off: int, steps: torch.T
         dim, vdim, _stream()), "ssd_scan")
     if first is not None:
         count_replayed(2)                      # the passes over the chunks, launched by the same call
+
+
+STATE_SPACE_ROWS = (32, 64, 128)         # state sizes the tensor-core kernel is built for
+
+
+def state_space_mma_supports(dtype: torch.dtype, heads: int, groups: int, dim: int, vdim: int) -> bool:
+    """Sizes of ``state_space_mma`` for rows that hold nothing but [v | k | q] (every offset a multiple of 8 channels)."""
+    return dtype == torch.bfloat16 and dim in STATE_SPACE_ROWS and vdim % 8 == 0 and heads % groups == 0
+
+
+def state_space_mma(x: torch.Tensor, q_off: int, k_off: int, v_off: int, steps: torch.Tensor, step_bias: torch.Tensor, rate_log: torch.Tensor,
+                    state: torch.Tensor, slot_ids: torch.Tensor, o_raw: torch.Tensor, heads: int, groups: int, dim: int, vdim: int,
+                    runs: torch.Tensor) -> None:
+    """``ssd_scan`` on tensor cores for the runs listed in ``runs`` (int32, (first token row, end, entry) each): bfloat16
+    rows, chunks of 64 tokens, the state and every decay in float32."""
+    for t in (steps, step_bias, rate_log, state, o_raw):
+        _dev(t, torch.float32, "state_space_mma")
+    _dev(runs, torch.int32, "state_space_mma runs")
+    if (not state_space_mma_supports(x.dtype, heads, groups, dim, vdim) or state.dim() != 2 or state.shape[1] < heads * dim * vdim or x.stride(1) != 1
+            or o_raw.numel() != x.shape[0] * heads * vdim or tuple(steps.shape) != (x.shape[0], heads) or step_bias.numel() != heads
+            or rate_log.numel() != heads or (x.stride(0) | q_off | k_off | v_off) % 8):
+        raise KernelError(f"state_space_mma: unsupported sizes: {heads} heads, state {dim} x {vdim}, offsets {v_off}, {k_off}, {q_off}")
+    _check(_fn("q25_state_space_bf16", [_P, _I, _I, _I, _I, _P, _P, _P, _P, _LL, _P, _P, _I, _P, _I, _I, _I, _I, _P])(
+        x.data_ptr(), x.stride(0), int(q_off), int(k_off), int(v_off), steps.data_ptr(), step_bias.data_ptr(), rate_log.data_ptr(), state.data_ptr(),
+        state.shape[1], slot_ids.data_ptr(), runs.data_ptr(), runs.numel() // 3, o_raw.data_ptr(), heads, groups, dim, vdim, _stream()),
+        "state_space_mma")
 
 
 def ssd_output(o_raw: torch.Tensor, v: torch.Tensor, z: torch.Tensor, skip: torch.Tensor, weight: torch.Tensor, parts: int, eps: float,

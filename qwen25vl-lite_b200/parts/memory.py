@@ -35,7 +35,7 @@ from __future__ import annotations
 import numpy as np
 import torch
 
-from ..ops import kernels
+from ..ops import kernels, state_space
 from ..ops.linear import Linear
 from .base import Mixer, StateNeed, TensorSpec, register_mixer
 
@@ -197,7 +197,17 @@ class Mamba2(Mixer):
         # S [heads, state, value_dim], then the last conv - 1 inputs of the convolution [conv - 1, channels]
         return StateNeed((self._memory_floats + (self.conv - 1) * self.channels,), "float32")
 
-    plan_key, plan_step = _MatrixMemory.plan_key, _MatrixMemory.plan_step       # the same work lists as the other memories
+    @property
+    def _tensor_cores(self) -> bool:
+        """Whether this mixer's runs of tokens can go to the tensor-core kernel."""
+        return self.out_proj is not None and kernels.state_space_mma_supports(self.out_proj.weight.dtype, self.num_heads, self.groups, self.state_dim,
+                                                                              self.value_dim)
+
+    def plan_key(self):
+        return ("state_space",) if self._tensor_cores else ("matrix_memory",)
+
+    def plan_step(self, host):
+        return state_space.plan(host.q_lens, self._tensor_cores)
 
     def load(self, tensors, device, dtype):
         f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
@@ -218,10 +228,8 @@ class Mamba2(Mixer):
         kernels.causal_conv(zx[:, inner:], self.conv_w, self.conv_b, stop.state, self._memory_floats, ctx.cu_q, ctx.slot_ids, xbc, ctx.n_seqs,
                             ctx.max_q_len, silu=True)
         o_raw = torch.empty((n, inner), dtype=torch.float32, device=zx.device)
-        plan = ctx.plan(self)
-        kernels.ssd_scan(xbc, inner + self.groups * self.state_dim, inner, 0, steps, self.step_bias, self.rate_log, stop.state, ctx.cu_q,
-                         ctx.slot_ids, o_raw, ctx.n_seqs, self.num_heads, self.groups, self.state_dim, self.value_dim, plan.get("first"),
-                         plan.get("runs"), plan.get("second"))
+        state_space.run(ctx.plan(self), ctx, xbc, inner + self.groups * self.state_dim, inner, 0, steps, self.step_bias, self.rate_log, stop.state,
+                        o_raw, self.num_heads, self.groups, self.state_dim, self.value_dim)
         out = torch.empty((n, inner), dtype=zx.dtype, device=zx.device)
         kernels.ssd_output(o_raw, xbc[:, :inner], zx[:, :inner], self.skip, self.norm_weight, self.norm_groups, self.norm_eps, out, self.value_dim)
         return self.out_proj(out, residual=residual)
