@@ -610,7 +610,7 @@ Q25_EXPORT int q25_memory_ssd_scan_bf16(const void* x, int xs, int qo, int ko, i
 // out[n] = rms_in_parts((o[n] + D_head v[n]) * silu(z[n])) * weight; o float [N, inner], v and z rows of T.  A CTA per token;
 // every part's squares are summed by one warp, lanes striding, then a butterfly.
 template <typename T>
-__global__ void __launch_bounds__(256) ssd_output_kernel(const float* __restrict__ o_raw, const T* __restrict__ v, int v_stride,
+__global__ void __launch_bounds__(512) ssd_output_kernel(const float* __restrict__ o_raw, const T* __restrict__ v, int v_stride,
                                                          const T* __restrict__ z, int z_stride, const float* __restrict__ skip,
                                                          const float* __restrict__ weight, T* __restrict__ out, int inner, int Dv, int parts,
                                                          float eps, int vec) {
@@ -683,7 +683,7 @@ static int ssd_output(const float* o_raw, const void* v, int v_stride, const voi
   const size_t row = 4 * sizeof(T);
   const int vec = Dv % 4 == 0 && (inner / parts) % 4 == 0 && v_stride % 4 == 0 && z_stride % 4 == 0 &&
                   !((uintptr_t)v % row) && !((uintptr_t)z % row) && !((uintptr_t)out % row) && !(((uintptr_t)o_raw | (uintptr_t)weight) & 15);
-  launch(ssd_output_kernel<T>, dim3(n_tokens), dim3(inner >= 1024 ? 256 : 128), smem, (cudaStream_t)stream, o_raw, (const T*)v, v_stride,
+  launch(ssd_output_kernel<T>, dim3(n_tokens), dim3(inner >= 2048 && n_tokens <= 256 ? 512 : inner >= 1024 ? 256 : 128), smem, (cudaStream_t)stream, o_raw, (const T*)v, v_stride,
          (const T*)z, z_stride, skip, weight, (T*)out, inner, Dv, parts, eps, vec);
   return launch_status();
 }

@@ -21,7 +21,7 @@ __device__ __forceinline__ float4 fma4(float s, float4 v, float4 acc) {
 
 // STREAMS: their number, or 0 for any up to HC_MAX_STREAMS (`streams` says how many).  VEC: four channels at a time.
 template <typename T, int STREAMS, bool VEC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 hyper_norm_kernel(float* __restrict__ x, const T* __restrict__ y, const float* __restrict__ mix, const float* __restrict__ out_w,
                   const float* __restrict__ in_w, const float* __restrict__ w, float eps, T* __restrict__ h,
                   const int* __restrict__ row_ids, int streams, int width) {
@@ -126,7 +126,9 @@ static int hyper_norm_shape(float* x, const void* y, const float* mix, const flo
     const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  launch(kernel, dim3(n_out), dim3(width >= 1024 ? 256 : 128), smem, (cudaStream_t)stream, x, (const T*)y, mix, out_w, in_w, w, eps, (T*)h, row_ids,
+  // a few rows finish sooner with more threads to a row; many share the SMs better with fewer
+  const int threads = width >= 2048 && n_out <= 256 ? 512 : width >= 1024 ? 256 : 128;
+  launch(kernel, dim3(n_out), dim3(threads), smem, (cudaStream_t)stream, x, (const T*)y, mix, out_w, in_w, w, eps, (T*)h, row_ids,
          streams, width);
   return launch_status();
 }

@@ -6,17 +6,32 @@
 //   row[C .. C + R)  = rotate(x[C .. C + R))                                 (not normed)
 //
 // The attention kernels then read the row as the single kv head's key (C + R channels) and its first
-// C channels as the value.  Where the queries come through a latent of their own, a second kernel norms that; where the
-// heads' results are gated, a third multiplies them with the sigmoid of the token's gate channels.
+// C channels as the value.  Where the queries come through a latent of their own, the same launch norms that too (a
+// second row of CTAs).  Where the heads' results are gated, another kernel multiplies them with the sigmoid of the
+// token's gate channels.
 #include "rotary.cuh"
 
 template <typename T, bool EXACT>
 __global__ void latent_store_kernel(const T* __restrict__ x, int x_row, int C, int R, const float* __restrict__ w, float eps,
                                     const float* __restrict__ angles, int half, int layout, T* __restrict__ pages,
-                                    const int* __restrict__ kv_slot) {
+                                    const int* __restrict__ kv_slot, const T* __restrict__ q, int q_row, int Cq,
+                                    const float* __restrict__ q_w, T* __restrict__ q_out) {
   pdl_trigger();
   pdl_wait();
   __shared__ float scratch[32];
+  if (blockIdx.y == 1 || !pages) {            // the queries' latent
+    const T* qr = q + (size_t)blockIdx.x * q_row;
+    float sq = 0.f;
+    for (int c = threadIdx.x; c < Cq; c += blockDim.x) {
+      const float v = to_f32(qr[c]);
+      sq = fmaf(v, v, sq);
+    }
+    const float q_total = block_sum(sq, scratch);
+    const float q_inv = EXACT ? 1.0f / sqrtf(q_total / (float)Cq + eps) : rsqrtf(q_total / (float)Cq + eps);
+    T* o = q_out + (size_t)blockIdx.x * Cq;
+    for (int c = threadIdx.x; c < Cq; c += blockDim.x) o[c] = from_f32<T>(to_f32(qr[c]) * q_inv * q_w[c]);
+    return;
+  }
   const int tok = blockIdx.x;
   const T* xr = x + (size_t)tok * x_row;
   float ss = 0.f;
@@ -36,50 +51,20 @@ __global__ void latent_store_kernel(const T* __restrict__ x, int x_row, int C, i
 
 template <typename T, bool EXACT>
 static int latent_store(const void* x, int x_row, int C, int R, const float* w, float eps, const float* angles, int half, int layout,
-                        void* pages, const int* kv_slot, int n, void* stream) {
-  if (n <= 0) return 0;
-  if (C <= 0 || R < 0 || 2 * half > R) return (int)cudaErrorInvalidValue;
-  launch(latent_store_kernel<T, EXACT>, dim3(n), dim3(128), 0, (cudaStream_t)stream, (const T*)x, x_row, C, R, w, eps, angles, half,
-         layout, (T*)pages, kv_slot);
+                        void* pages, const int* kv_slot, int n, const void* q, int q_row, int Cq, const float* q_w, void* q_out, void* stream) {
+  if (n <= 0 || (!pages && !q)) return 0;
+  if (C <= 0 || R < 0 || 2 * half > R || (pages && !kv_slot) || (q && (Cq <= 0 || !q_w || !q_out))) return (int)cudaErrorInvalidValue;
+  launch(latent_store_kernel<T, EXACT>, dim3(n, pages && q ? 2 : 1), dim3(128), 0, (cudaStream_t)stream, (const T*)x, x_row, C, R, w, eps, angles,
+         half, layout, (T*)pages, kv_slot, (const T*)q, q_row, Cq, q_w, (T*)q_out);
   return launch_status();
 }
 Q25_EXPORT int q25_latent_store_f32(const void* x, int xr, int C, int R, const float* w, float eps, const float* ang, int half,
-                                    int layout, void* pages, const int* slot, int n, void* s) {
-  return latent_store<float, true>(x, xr, C, R, w, eps, ang, half, layout, pages, slot, n, s);
+                                    int layout, void* pages, const int* slot, int n, const void* q, int qr, int Cq, const float* qw, void* qo, void* s) {
+  return latent_store<float, true>(x, xr, C, R, w, eps, ang, half, layout, pages, slot, n, q, qr, Cq, qw, qo, s);
 }
 Q25_EXPORT int q25_latent_store_bf16(const void* x, int xr, int C, int R, const float* w, float eps, const float* ang, int half,
-                                     int layout, void* pages, const int* slot, int n, void* s) {
-  return latent_store<bf16, false>(x, xr, C, R, w, eps, ang, half, layout, pages, slot, n, s);
-}
-
-// out[n] = x[n] / sqrt(mean(x[n]^2) + eps) * w for strided rows x of C channels, statistics in float.
-template <typename T>
-__global__ void latent_norm_kernel(const T* __restrict__ x, int x_row, int C, const float* __restrict__ w, float eps, T* __restrict__ out) {
-  pdl_trigger();
-  pdl_wait();
-  __shared__ float scratch[32];
-  const T* xr = x + (size_t)blockIdx.x * x_row;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    const float v = to_f32(xr[c]);
-    ss = fmaf(v, v, ss);
-  }
-  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)C + eps);
-  T* o = out + (size_t)blockIdx.x * C;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) o[c] = from_f32<T>(to_f32(xr[c]) * inv * w[c]);
-}
-template <typename T>
-static int latent_norm(const void* x, int x_row, int C, const float* w, float eps, void* out, int n, void* stream) {
-  if (n <= 0) return 0;
-  if (C <= 0) return (int)cudaErrorInvalidValue;
-  launch(latent_norm_kernel<T>, dim3(n), dim3(C >= 512 ? 256 : 128), 0, (cudaStream_t)stream, (const T*)x, x_row, C, w, eps, (T*)out);
-  return launch_status();
-}
-Q25_EXPORT int q25_latent_norm_f32(const void* x, int xr, int C, const float* w, float eps, void* out, int n, void* s) {
-  return latent_norm<float>(x, xr, C, w, eps, out, n, s);
-}
-Q25_EXPORT int q25_latent_norm_bf16(const void* x, int xr, int C, const float* w, float eps, void* out, int n, void* s) {
-  return latent_norm<bf16>(x, xr, C, w, eps, out, n, s);
+                                     int layout, void* pages, const int* slot, int n, const void* q, int qr, int Cq, const float* qw, void* qo, void* s) {
+  return latent_store<bf16, false>(x, xr, C, R, w, eps, ang, half, layout, pages, slot, n, q, qr, Cq, qw, qo, s);
 }
 
 // y[n, c] *= sigmoid(g[n, c]), in place; y contiguous, g strided rows.

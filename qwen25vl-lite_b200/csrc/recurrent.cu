@@ -9,45 +9,19 @@
 //   out_t = S_t * gelu_tanh(ybranch_t)
 //
 // xin and ybranch are the two halves of one projection (activation dtype T); everything from u on
-// is float: the gates' products are plain FMA chains over the block's channels in index order, so
+// is float: the gates' products are sums over the block's channels in an order that the block's size alone decides, so
 // a token's gates do not depend on the batch, and the state S is carried in float from step to step.
 //
 // Per-request state [slots, taps, W] float: row 0 is S, rows 1 .. taps-1 are the last taps-1 inputs
 // xin of the request, oldest first (zeros at admission, which are the zeros before the start).
 //
-// A convolution on its own (causal_conv_kernel, with an optional silu, a history in a state of any layout and a result in
-// T) serves recurrences that keep their state elsewhere.
-//
-// The kernels: the convolution; the two gates of all blocks as one batched FMA product with the
-// decay and the input term formed in its epilogue; the scan in chunks over time, which also moves
-// the state on.
-#include "common.cuh"
+// The kernels: the convolution, which moves its inputs on (it also serves mixers that keep other state beside
+// them); the two gates of all blocks as one batched product with the decay and the input term formed in its
+// epilogue (float FMAs; for long steps whose gate matrices are bfloat16 numbers, tensor cores with u as a sum of
+// three bfloat16 numbers); the scan in chunks over time, which moves S on.
+#include "mma.cuh"
 
 #define RG_MAX_TAPS 16
-
-template <typename T>
-__global__ void rglru_conv_kernel(const T* __restrict__ yx, int ld, int x_off, const float* __restrict__ conv_w,
-                                  const float* __restrict__ conv_b, const float* __restrict__ state,
-                                  const int* __restrict__ token_seq, const int* __restrict__ cu_q,
-                                  const int* __restrict__ slot_ids, float* __restrict__ u, int row0, int width, int taps) {
-  pdl_trigger();
-  pdl_wait();
-  // a row of blocks per token: what depends on the token alone is looked up once
-  const int n = row0 + blockIdx.y;
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= width) return;
-  const int seq = token_seq[n];
-  const int first = cu_q[seq];
-  const int t = n - first;
-  const float* hist = state + ((size_t)slot_ids[seq] * taps + 1) * width + c;      // rows 1 .. taps-1
-  float acc = 0.f;
-  for (int j = 0; j < taps; ++j) {
-    const int rel = t - (taps - 1) + j;
-    const float v = rel >= 0 ? to_f32(yx[(size_t)(first + rel) * ld + x_off + c]) : hist[(size_t)(taps - 1 + rel) * width];
-    acc = fmaf(conv_w[(size_t)c * taps + j], v, acc);
-  }
-  u[(size_t)n * width + c] = acc + conv_b[c];
-}
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -169,6 +143,98 @@ rglru_gates_small_kernel(const float* __restrict__ u, const float* __restrict__ 
   bx_out[at] = sqrtf(-expm1f(2.0f * log_a)) * g * u[at];
 }
 
+// Both gates for long steps on tensor cores (mma.sync, float accumulators), for gate matrices whose entries are bfloat16
+// numbers.  u is float: it enters as the sum of three bfloat16 numbers (the rounded value, what the rounding left,
+// rounded, and what that left), which is u itself to 24 bits, in three products each; so the sums are float sums of
+// exact products, as in the kernels above.  A CTA takes 64 tokens x 64 channels of one block; warp (m, h) 16 tokens x
+// 32 channels of both gates.
+#define RGM_K 64
+#define RGM_P (RGM_K + 8)
+
+__global__ void __launch_bounds__(256)
+rglru_gates_mma_kernel(const float* __restrict__ u, const bf16* __restrict__ ra, const float* __restrict__ ra_b, const bf16* __restrict__ ri,
+                       const float* __restrict__ ri_b, const float* __restrict__ lam, float gain, float* __restrict__ a_out,
+                       float* __restrict__ bx_out, int n_tokens, int width, int bw) {
+  pdl_trigger();
+  __shared__ __align__(16) bf16 Us[3][64][RGM_P];
+  __shared__ __align__(16) bf16 Ws[2][64][RGM_P];
+  const int b = blockIdx.z, m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wm = (warp & 3) * 16, wn = (warp >> 2) * 32;
+  float acc[2][4][4];
+#pragma unroll
+  for (int g = 0; g < 2; ++g)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[g][i][e] = 0.f;
+  pdl_wait();
+  for (int k0 = 0; k0 < bw; k0 += RGM_K) {
+    for (int i = tid; i < 2 * 64 * (RGM_K / 8); i += 256) {
+      const int gate = i / (64 * (RGM_K / 8)), r = i / (RGM_K / 8) % 64, c = (i % (RGM_K / 8)) * 8;
+      const bool ok = n0 + r < bw && k0 + c < bw;
+      const bf16* src = (gate ? ri : ra) + (size_t)b * bw * bw;
+      cp_async16(&Ws[gate][r][c], ok ? src + (size_t)(n0 + r) * bw + k0 + c : src, ok);
+    }
+    cp_async_commit();
+    for (int i = tid; i < 64 * (RGM_K / 4); i += 256) {
+      const int r = i / (RGM_K / 4), c = (i % (RGM_K / 4)) * 4;
+      const bool ok = m0 + r < n_tokens && k0 + c < bw;
+      float4 v = ok ? *reinterpret_cast<const float4*>(u + (size_t)(m0 + r) * width + (size_t)b * bw + k0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int part = 0; part < 3; ++part) {
+        store4<bf16>(&Us[part][r][c], v);
+        const float4 took = load4<bf16>(&Us[part][r][c]);
+        v.x -= took.x; v.y -= took.y; v.z -= took.z; v.w -= took.w;
+      }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < RGM_K / 16; ++k) {
+      unsigned a[3][4];
+#pragma unroll
+      for (int part = 0; part < 3; ++part) ldmatrix_x4(a[part], &Us[part][wm + (lane & 15)][k * 16 + (lane >> 4) * 8]);
+#pragma unroll
+      for (int g = 0; g < 2; ++g)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          unsigned w[4];
+          ldmatrix_x4(w, &Ws[g][wn + i * 16 + (lane & 7) + ((lane >> 4) << 3)][k * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+          for (int part = 2; part >= 0; --part) {
+            mma_bf16(acc[g][2 * i], a[part], w[0], w[1]);
+            mma_bf16(acc[g][2 * i + 1], a[part], w[2], w[3]);
+          }
+        }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int gn = n0 + wn + i * 8 + (lane & 3) * 2;
+    if (gn >= bw) continue;
+    const int c = b * bw + gn;
+    const float sp[2] = {softplus_f(lam[c]), softplus_f(lam[c + 1])};
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int gm = m0 + wm + (lane >> 2) + e * 8;
+      if (gm >= n_tokens) continue;
+      const size_t at = (size_t)gm * width + c;
+      const float2 uu = *reinterpret_cast<const float2*>(u + at);
+      float av[2], bv[2];
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const float r = sigmoid_f(acc[0][i][2 * e + q] + ra_b[c + q]), g = sigmoid_f(acc[1][i][2 * e + q] + ri_b[c + q]);
+        const float log_a = -gain * r * sp[q];
+        av[q] = expf(log_a);
+        bv[q] = sqrtf(-expm1f(2.0f * log_a)) * g * (q ? uu.y : uu.x);
+      }
+      *reinterpret_cast<float2*>(a_out + at) = make_float2(av[0], av[1]);
+      *reinterpret_cast<float2*>(bx_out + at) = make_float2(bv[0], bv[1]);
+    }
+  }
+}
+
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
@@ -182,8 +248,7 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 //   rglru_scan_kernel: one thread per (entry, chunk, channel) folds the summaries of the chunks
 //     before its own onto the request's S (a short chain of FMAs over values that all chunks of
 //     the entry read, so they stay in cache), then runs its chunk and writes out = S * gelu_tanh(y).
-//     The thread of the last chunk moves the state on: S, and the last taps-1 inputs of (old
-//     inputs ++ this entry's inputs).
+//     The thread of the last chunk moves S on.
 // A step whose entries all have up to RG_CHUNK tokens (every decode step) runs the second kernel
 // alone: one chunk per entry, S read from the state itself.
 // sums: [n_seqs, max_chunks, 2, width] (A, B), then [n_seqs, width] (the requests' S before the step).
@@ -215,7 +280,7 @@ __global__ void rglru_chunk_kernel(const float* __restrict__ a, const float* __r
 
 template <typename T>
 __global__ void rglru_scan_kernel(const float* __restrict__ a, const float* __restrict__ bx, const T* __restrict__ yx, int ld,
-                                  int y_off, int x_off, float* __restrict__ state, const int* __restrict__ cu_q,
+                                  int y_off, float* __restrict__ state, const int* __restrict__ cu_q,
                                   const int* __restrict__ slot_ids, T* __restrict__ out, const float* __restrict__ sums,
                                   int n_seqs, int width, int taps, int max_chunks) {
   pdl_trigger();
@@ -240,32 +305,6 @@ __global__ void rglru_scan_kernel(const float* __restrict__ a, const float* __re
   }
   if (t1 < n) return;                          // the last chunk's thread moves the state on; nobody else reads it here
   st[0] = S;
-  float keep[RG_MAX_TAPS];
-#pragma unroll
-  for (int k = 0; k < RG_MAX_TAPS - 1; ++k) {
-    if (k < taps - 1) {
-      const int rel = n - (taps - 1) + k;
-      keep[k] = rel >= 0 ? to_f32(yx[(size_t)(first + rel) * ld + x_off + c]) : st[(size_t)(1 + k + n) * width];
-    }
-  }
-#pragma unroll
-  for (int k = 0; k < RG_MAX_TAPS - 1; ++k)
-    if (k < taps - 1) st[(size_t)(1 + k) * width] = keep[k];
-}
-
-template <typename T>
-static int rglru_conv(const void* yx, int ld, int x_off, const float* conv_w, const float* conv_b, const float* state,
-                      const int* token_seq, const int* cu_q, const int* slot_ids, float* u, int n_tokens, int width, int taps,
-                      void* stream) {
-  if (n_tokens <= 0) return 0;
-  if (taps < 1 || taps > RG_MAX_TAPS) return (int)cudaErrorInvalidValue;
-  if (n_tokens > 65535 * 32) return (int)cudaErrorInvalidValue;
-  for (int at = 0; at < n_tokens; at += 65535) {                  // the grid's second dimension ends at 65,535
-    const int rows = n_tokens - at < 65535 ? n_tokens - at : 65535;
-    launch(rglru_conv_kernel<T>, dim3((width + 255) / 256, rows), dim3(256), 0, (cudaStream_t)stream, (const T*)yx, ld, x_off, conv_w,
-           conv_b, state, token_seq, cu_q, slot_ids, u, at, width, taps);
-  }
-  return launch_status();
 }
 
 // Floats of scratch memory the scan needs for a step whose longest entry has max_q_len tokens (0: none).
@@ -275,7 +314,7 @@ Q25_EXPORT long long q25_rglru_scan_scratch_floats(int n_seqs, int max_q_len, in
 }
 
 template <typename T>
-static int rglru_scan(const float* a, const float* bx, const void* yx, int ld, int y_off, int x_off, float* state, const int* cu_q,
+static int rglru_scan(const float* a, const float* bx, const void* yx, int ld, int y_off, float* state, const int* cu_q,
                       const int* slot_ids, void* out, int n_seqs, int max_q_len, float* sums, int width, int taps, void* stream) {
   if (n_seqs <= 0) return 0;
   if (taps < 1 || taps > RG_MAX_TAPS || max_q_len < 1) return (int)cudaErrorInvalidValue;
@@ -285,19 +324,11 @@ static int rglru_scan(const float* a, const float* bx, const void* yx, int ld, i
   if (max_chunks > 1)
     launch(rglru_chunk_kernel, grid, dim3(128), 0, (cudaStream_t)stream, a, bx, (const float*)state, cu_q, slot_ids, sums, n_seqs, width,
            taps, max_chunks);
-  launch(rglru_scan_kernel<T>, grid, dim3(128), 0, (cudaStream_t)stream, a, bx, (const T*)yx, ld, y_off, x_off, state, cu_q, slot_ids,
+  launch(rglru_scan_kernel<T>, grid, dim3(128), 0, (cudaStream_t)stream, a, bx, (const T*)yx, ld, y_off, state, cu_q, slot_ids,
          (T*)out, (const float*)(max_chunks > 1 ? sums : nullptr), n_seqs, width, taps, max_chunks);
   return launch_status();
 }
 
-Q25_EXPORT int q25_rglru_conv_f32(const void* yx, int ld, int xo, const float* cw, const float* cb, const float* st, const int* ts,
-                                  const int* cu, const int* sl, float* u, int n, int w, int taps, void* s) {
-  return rglru_conv<float>(yx, ld, xo, cw, cb, st, ts, cu, sl, u, n, w, taps, s);
-}
-Q25_EXPORT int q25_rglru_conv_bf16(const void* yx, int ld, int xo, const float* cw, const float* cb, const float* st, const int* ts,
-                                   const int* cu, const int* sl, float* u, int n, int w, int taps, void* s) {
-  return rglru_conv<bf16>(yx, ld, xo, cw, cb, st, ts, cu, sl, u, n, w, taps, s);
-}
 Q25_EXPORT int q25_rglru_gates(const float* u, const float* ra, const float* ra_b, const float* ri, const float* ri_b,
                                const float* lam, float gain, float* a_out, float* bx_out, int n_tokens, int width, int blocks,
                                void* stream) {
@@ -321,45 +352,53 @@ Q25_EXPORT int q25_rglru_gates(const float* u, const float* ra, const float* ra_
   }
   return launch_status();
 }
-Q25_EXPORT int q25_rglru_scan_f32(const float* a, const float* bx, const void* yx, int ld, int yo, int xo, float* st, const int* cu,
-                                  const int* sl, void* out, int n_seqs, int max_q_len, float* sums, int w, int taps, void* s) {
-  return rglru_scan<float>(a, bx, yx, ld, yo, xo, st, cu, sl, out, n_seqs, max_q_len, sums, w, taps, s);
+// The same with bfloat16 gate matrices; the blocks' width is a multiple of 8.
+Q25_EXPORT int q25_rglru_gates_mma(const float* u, const void* ra, const float* ra_b, const void* ri, const float* ri_b, const float* lam, float gain,
+                                   float* a_out, float* bx_out, int n_tokens, int width, int blocks, void* stream) {
+  if (n_tokens <= 0) return 0;
+  if (blocks <= 0 || width % blocks || (width / blocks) % 8 || (((uintptr_t)u | (uintptr_t)ra | (uintptr_t)ri | (uintptr_t)a_out | (uintptr_t)bx_out) & 15))
+    return (int)cudaErrorInvalidValue;
+  const int bw = width / blocks;
+  launch(rglru_gates_mma_kernel, dim3((bw + 63) / 64, (n_tokens + 63) / 64, blocks), dim3(256), 0, (cudaStream_t)stream, u, (const bf16*)ra, ra_b,
+         (const bf16*)ri, ri_b, lam, gain, a_out, bx_out, n_tokens, width, bw);
+  return launch_status();
 }
-Q25_EXPORT int q25_rglru_scan_bf16(const float* a, const float* bx, const void* yx, int ld, int yo, int xo, float* st, const int* cu,
+Q25_EXPORT int q25_rglru_scan_f32(const float* a, const float* bx, const void* yx, int ld, int yo, float* st, const int* cu,
+                                  const int* sl, void* out, int n_seqs, int max_q_len, float* sums, int w, int taps, void* s) {
+  return rglru_scan<float>(a, bx, yx, ld, yo, st, cu, sl, out, n_seqs, max_q_len, sums, w, taps, s);
+}
+Q25_EXPORT int q25_rglru_scan_bf16(const float* a, const float* bx, const void* yx, int ld, int yo, float* st, const int* cu,
                                    const int* sl, void* out, int n_seqs, int max_q_len, float* sums, int w, int taps, void* s) {
-  return rglru_scan<bf16>(a, bx, yx, ld, yo, xo, st, cu, sl, out, n_seqs, max_q_len, sums, w, taps, s);
+  return rglru_scan<bf16>(a, bx, yx, ld, yo, st, cu, sl, out, n_seqs, max_q_len, sums, w, taps, s);
 }
 
-// ---- a causal convolution per channel, on its own ----------------------------------------------------------------
+// ---- the causal convolution per channel ----------------------------------------------------------------
 // out[n, c] = act(bias[c] + sum_j w[j, c] in_(t - (taps - 1) + j)[c]), the inputs before the step's first token from the
 // request's history [taps - 1, channels] (floats at state + slot * slot_floats, oldest first; zeros at admission), which
 // moves on.  A thread owns V channels of CONV_TOKENS consecutive tokens of an entry and slides a window over the inputs,
 // so an input is read once (and taps - 1 of them again per piece); the piece that holds the entry's first token is the
-// only reader of the history and writes the new one.  WIN: taps rounded up to a built size; the window's older places
+// only reader of the history and writes the new one.  TO: the result's dtype.  WIN: taps rounded up to a built size; the window's older places
 // carry weights of zero.
-#define CONV_TOKENS 32
+#define CONV_TOKENS 16
 #define CONV_AHEAD 8         // inputs a thread asks for at once
 
-template <typename T, int V> struct ConvVec;
-template <> struct ConvVec<float, 1> { static __device__ __forceinline__ void load(const float* p, float* v) { v[0] = p[0]; }
-                                       static __device__ __forceinline__ void store(float* p, const float* v) { p[0] = v[0]; } };
-template <> struct ConvVec<bf16, 1> { static __device__ __forceinline__ void load(const bf16* p, float* v) { v[0] = to_f32(p[0]); }
-                                      static __device__ __forceinline__ void store(bf16* p, const float* v) { p[0] = from_f32<bf16>(v[0]); } };
-template <> struct ConvVec<float, 2> {
-  static __device__ __forceinline__ void load(const float* p, float* v) { const float2 a = *reinterpret_cast<const float2*>(p); v[0] = a.x; v[1] = a.y; }
-  static __device__ __forceinline__ void store(float* p, const float* v) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
-};
-template <> struct ConvVec<bf16, 2> {
-  static __device__ __forceinline__ void load(const bf16* p, float* v) {
-    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(p); v[0] = __low2float(a); v[1] = __high2float(a);
+template <typename T, int V> __device__ __forceinline__ void conv_load(const T* p, float (&v)[V]) {
+  if constexpr (V == 4) {
+    const float4 a = load4<T>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  } else {
+    v[0] = to_f32(p[0]);
   }
-  static __device__ __forceinline__ void store(bf16* p, const float* v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]); }
-};
+}
+template <typename T, int V> __device__ __forceinline__ void conv_store(T* p, const float (&v)[V]) {
+  if constexpr (V == 4) store4<T>(p, make_float4(v[0], v[1], v[2], v[3]));
+  else p[0] = from_f32<T>(v[0]);
+}
 
-template <typename T, int WIN, int V>
+template <typename T, typename TO, int WIN, int V>
 __global__ void __launch_bounds__(128)
 causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ state,
-                   size_t slot_floats, const int* __restrict__ cu_q, const int* __restrict__ slot_ids, T* __restrict__ out, int out_stride,
+                   size_t slot_floats, const int* __restrict__ cu_q, const int* __restrict__ slot_ids, TO* __restrict__ out, int out_stride,
                    int channels, int taps, int silu) {
   pdl_trigger();
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
@@ -379,7 +418,7 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
   if (c >= channels || t0 >= n) return;
   const int t1 = min(n, t0 + CONV_TOKENS);
   const T* x = in + (size_t)first * in_stride + c;
-  T* o = out + (size_t)first * out_stride + c;
+  TO* o = out + (size_t)first * out_stride + c;
   float* hist = state + (size_t)slot_ids[seq] * slot_floats + c;
   float win[WIN][V];                           // the last WIN inputs, the newest last
 #pragma unroll
@@ -391,7 +430,7 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
   for (int j = 1; j < WIN; ++j) {
     const int rel = t0 - WIN + j;
     if (j > WIN - taps) {
-      if (rel >= 0) ConvVec<T, V>::load(x + (size_t)rel * in_stride, win[j]);
+      if (rel >= 0) conv_load<T, V>(x + (size_t)rel * in_stride, win[j]);
       else if (piece == 0) {
 #pragma unroll
         for (int v = 0; v < V; ++v) win[j][v] = hist[(size_t)(taps - 1 + rel) * channels + v];
@@ -408,7 +447,7 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
 #pragma unroll
       for (int v = 0; v < V; ++v) keep[j - 1][v] = 0.f;
       if (j > WIN - taps) {
-        if (rel >= 0) ConvVec<T, V>::load(x + (size_t)rel * in_stride, keep[j - 1]);
+        if (rel >= 0) conv_load<T, V>(x + (size_t)rel * in_stride, keep[j - 1]);
         else {
 #pragma unroll
           for (int i = 1; i < WIN; ++i)
@@ -431,7 +470,7 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
 #pragma unroll
     for (int a = 0; a < CONV_AHEAD; ++a) {
       const int tt = min(t + a, t1 - 1);
-      ConvVec<T, V>::load(x + (size_t)tt * in_stride, next[a]);
+      conv_load<T, V>(x + (size_t)tt * in_stride, next[a]);
     }
 #pragma unroll
     for (int a = 0; a < CONV_AHEAD; ++a) {
@@ -448,35 +487,35 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
           acc += b[v];
           r[v] = silu ? acc / (1.0f + expf(-acc)) : acc;
         }
-        ConvVec<T, V>::store(o + (size_t)(t + a) * out_stride, r);
+        conv_store<TO, V>(o + (size_t)(t + a) * out_stride, r);
       }
     }
   }
 }
 
-template <typename T>
+template <typename T, typename TO>
 static int causal_conv(const void* in, int in_stride, const float* w, const float* bias, float* state, long long slot_floats, const int* cu_q,
                        const int* slot_ids, void* out, int out_stride, int n_seqs, int max_q_len, int channels, int taps, int silu, void* stream) {
   if (n_seqs <= 0 || channels <= 0) return 0;
   if (taps < 1 || taps > RG_MAX_TAPS || max_q_len < 1 || (taps > 1 && !state)) return (int)cudaErrorInvalidValue;
   const int pieces = (max_q_len + CONV_TOKENS - 1) / CONV_TOKENS;
   if (pieces > 65535 || n_seqs > 65535) return (int)cudaErrorInvalidValue;
-  const size_t pair = 2 * sizeof(T);
-  const bool two = channels % 2 == 0 && in_stride % 2 == 0 && out_stride % 2 == 0 && !((uintptr_t)in % pair) && !((uintptr_t)out % pair);
-  const int threads_c = two ? channels / 2 : channels;
+  const bool four = channels % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && !((uintptr_t)in % (4 * sizeof(T))) && !((uintptr_t)out % (4 * sizeof(TO)));
+  const int threads_c = four ? channels / 4 : channels;
   const dim3 grid((threads_c + 127) / 128, n_seqs, pieces);
-  void (*kernel)(const T*, int, const float*, const float*, float*, size_t, const int*, const int*, T*, int, int, int, int) =
-      taps <= 4 ? (two ? causal_conv_kernel<T, 4, 2> : causal_conv_kernel<T, 4, 1>)
-                : (two ? causal_conv_kernel<T, RG_MAX_TAPS, 2> : causal_conv_kernel<T, RG_MAX_TAPS, 1>);
-  launch(kernel, grid, dim3(128), 0, (cudaStream_t)stream, (const T*)in, in_stride, w, bias, state, (size_t)slot_floats, cu_q, slot_ids, (T*)out,
+  void (*kernel)(const T*, int, const float*, const float*, float*, size_t, const int*, const int*, TO*, int, int, int, int) =
+      taps <= 4 ? (four ? causal_conv_kernel<T, TO, 4, 4> : causal_conv_kernel<T, TO, 4, 1>)
+                : (four ? causal_conv_kernel<T, TO, RG_MAX_TAPS, 4> : causal_conv_kernel<T, TO, RG_MAX_TAPS, 1>);
+  launch(kernel, grid, dim3(128), 0, (cudaStream_t)stream, (const T*)in, in_stride, w, bias, state, (size_t)slot_floats, cu_q, slot_ids, (TO*)out,
          out_stride, channels, taps, silu);
   return launch_status();
 }
 Q25_EXPORT int q25_rglru_causal_conv_f32(const void* in, int is, const float* w, const float* b, float* st, long long sf, const int* cu, const int* sl,
-                                         void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, void* s) {
-  return causal_conv<float>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
+                                         void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, int out_f32, void* s) {
+  return causal_conv<float, float>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
 }
 Q25_EXPORT int q25_rglru_causal_conv_bf16(const void* in, int is, const float* w, const float* b, float* st, long long sf, const int* cu, const int* sl,
-                                          void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, void* s) {
-  return causal_conv<bf16>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
+                                          void* out, int os, int n_seqs, int max_q_len, int channels, int taps, int silu, int out_f32, void* s) {
+  return out_f32 ? causal_conv<bf16, float>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s)
+                 : causal_conv<bf16, bf16>(in, is, w, b, st, sf, cu, sl, out, os, n_seqs, max_q_len, channels, taps, silu, s);
 }

@@ -29,13 +29,12 @@ _SIGNATURES = {
     "q25_embed_position_norm": [_P, _P, _P, _P, _P, _F, _P, _I, _I, _I, _I, _I, _F, _P],
     "q25_add_norm_groups": [_P, _P, _P, _F, _I, _P, _F, _I, _P, _P, _I, _I, _P],
     "q25_glu_clamped": [_P, _P, _I, _I, _F, _F, _F, _I, _P],
-    "q25_rglru_conv": [_P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _P],
-    "q25_rglru_scan": [_P, _P, _P, _I, _I, _I, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P],
+    "q25_rglru_scan": [_P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P],
     "q25_biased_attention_generic": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _I, _F, _P, _I, _I, _P],
     "q25_biased_attention_qk_norm_store": [_P, _I, _P, _P, _F, _I, _P, _I, _I, _P, _F, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "q25_add_dyt": [_P, _P, _P, _P, _F, _P, _P, _I, _I, _P],
     "q25_rotary_apply": [_P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
-    "q25_latent_store": [_P, _I, _I, _I, _P, _F, _P, _I, _I, _P, _P, _I, _P],
+    "q25_latent_store": [_P, _I, _I, _I, _P, _F, _P, _I, _I, _P, _P, _I, _P, _I, _I, _P, _P, _P],
     "q25_retention": [_P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _P, _I, _P, _I, _I, _P],
     "q25_kv_store_mix": [_P, _I, _P, _I, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "q25_moe_route": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
@@ -54,8 +53,7 @@ _SIGNATURES = {
     "q25_memory_scan_chunked": [_P, _I, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
     "q25_memory_ssd_scan": [_P, _I, _I, _I, _I, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _P],
     "q25_memory_ssd_output": [_P, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P],
-    "q25_rglru_causal_conv": [_P, _I, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
-    "q25_latent_norm": [_P, _I, _I, _P, _F, _P, _I, _P],
+    "q25_rglru_causal_conv": [_P, _I, _P, _P, _P, _LL, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "q25_latent_gate": [_P, _P, _I, _I, _I, _P],
     "q25_hyper_norm": [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
     "q25_hyper_embed": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _LL, _LL, _LL, _I, _P],
@@ -725,38 +723,30 @@ def glu_clamped(gate_up: torch.Tensor, out: torch.Tensor, limit: float, alpha: f
 # ---- the gated linear recurrence -------------------------------------------------------------------
 
 
-def rglru_conv(yx: torch.Tensor, x_off: int, conv_w: torch.Tensor, conv_b: torch.Tensor, state: torch.Tensor,
-               token_seq: torch.Tensor, cu_q: torch.Tensor, slot_ids: torch.Tensor, u_out: torch.Tensor) -> None:
-    """u_out[n, c] (float32) = causal convolution over the request's inputs ``yx[:, x_off + c]``, the
-    ``taps - 1`` inputs before the step's first token taken from ``state`` [slots, taps, width]."""
-    n, width = u_out.shape
-    taps = conv_w.shape[1]
-    _dev(u_out, torch.float32, "rglru_conv out"); _dev(state, torch.float32, "rglru_conv state")
-    _dev(conv_w, torch.float32, "rglru_conv weight"); _dev(conv_b, torch.float32, "rglru_conv bias")
-    if tuple(state.shape[1:]) != (taps, width) or yx.stride(1) != 1:
-        raise KernelError(f"rglru_conv: state must be [slots, {taps}, {width}]")
-    _check(_typed("q25_rglru_conv", yx.dtype)(yx.data_ptr(), yx.stride(0), int(x_off), conv_w.data_ptr(), conv_b.data_ptr(),
-                                              state.data_ptr(), token_seq.data_ptr(), cu_q.data_ptr(), slot_ids.data_ptr(),
-                                              u_out.data_ptr(), n, width, taps, _stream()), "rglru_conv")
+RGLRU_MMA_ROWS = 128                     # up to this many tokens the FMA kernel that holds a block's whole depth is as fast
 
 
 def rglru_gates(u: torch.Tensor, ra: torch.Tensor, ra_b: torch.Tensor, ri: torch.Tensor, ri_b: torch.Tensor, lam: torch.Tensor,
                 gain: float, a_out: torch.Tensor, bx_out: torch.Tensor) -> None:
     """The recurrence's decay a = exp(-gain * sigmoid(Ra u + b) * softplus(lam)) and input term
-    sqrt(1 - a^2) * sigmoid(Ri u + b) * u, per block of channels, all float32."""
+    sqrt(1 - a^2) * sigmoid(Ri u + b) * u, per block of channels, all float32.  bfloat16 ``ra`` and ``ri``: the products
+    run on tensor cores, with u carried to 24 bits."""
     n, width = u.shape
     blocks = ra.shape[0]
-    for t in (u, ra, ra_b, ri, ri_b, lam, a_out, bx_out):
+    for t in (u, ra_b, ri_b, lam, a_out, bx_out):
         _dev(t, torch.float32, "rglru_gates")
-    _check(_fn("q25_rglru_gates", [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P])(
+    mma = ra.dtype == torch.bfloat16
+    for t in (ra, ri):
+        _dev(t, torch.bfloat16 if mma else torch.float32, "rglru_gates matrix")
+    _check(_fn("q25_rglru_gates_mma" if mma else "q25_rglru_gates", [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P])(
         u.data_ptr(), ra.data_ptr(), ra_b.data_ptr(), ri.data_ptr(), ri_b.data_ptr(), lam.data_ptr(), float(gain),
         a_out.data_ptr(), bx_out.data_ptr(), n, width, blocks, _stream()), "rglru_gates")
 
 
-def rglru_scan(a: torch.Tensor, bx: torch.Tensor, yx: torch.Tensor, y_off: int, x_off: int, state: torch.Tensor,
+def rglru_scan(a: torch.Tensor, bx: torch.Tensor, yx: torch.Tensor, y_off: int, state: torch.Tensor,
                cu_q: torch.Tensor, slot_ids: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q_len: int) -> None:
     """S = a S + bx over every entry's tokens from the request's state (row 0 of ``state``), out = S *
-    gelu_tanh(yx[:, y_off + c]); the state (S and the last taps - 1 inputs) moves on.  ``max_q_len``:
+    gelu_tanh(yx[:, y_off + c]); S moves on (the other rows are the convolution's).  ``max_q_len``:
     the step's longest entry; entries beyond a chunk of tokens are scanned in chunks, in parallel."""
     width = out.shape[1]
     taps = state.shape[1]
@@ -765,7 +755,7 @@ def rglru_scan(a: torch.Tensor, bx: torch.Tensor, yx: torch.Tensor, y_off: int, 
     need.restype = ctypes.c_longlong
     floats = need(int(n_seqs), int(max_q_len), width)
     sums = torch.empty(floats, dtype=torch.float32, device=out.device) if floats else None
-    _check(_typed("q25_rglru_scan", yx.dtype)(a.data_ptr(), bx.data_ptr(), yx.data_ptr(), yx.stride(0), int(y_off), int(x_off),
+    _check(_typed("q25_rglru_scan", yx.dtype)(a.data_ptr(), bx.data_ptr(), yx.data_ptr(), yx.stride(0), int(y_off),
                                               state.data_ptr(), cu_q.data_ptr(), slot_ids.data_ptr(), out.data_ptr(), int(n_seqs),
                                               int(max_q_len), _ptr(sums), width, taps, _stream()), "rglru_scan")
     if floats:
@@ -776,16 +766,18 @@ def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state
                 slot_ids: torch.Tensor, out: torch.Tensor, n_seqs: int, max_q_len: int, silu: bool) -> None:
     """out[n, c] = act(bias[c] + sum_j weight[j, c] x_(t - (taps - 1) + j)[c]) over every entry's tokens, ``x`` a strided
     view [N, channels], ``weight`` float32 [taps, channels].  ``state`` (float32 [slots, floats]): from ``history_off`` on a
-    slot holds the request's last taps - 1 inputs, which come before the step's first token; they move on."""
+    slot holds the request's last taps - 1 inputs, which come before the step's first token; they move on.  ``out`` is of
+    x's dtype or float32."""
     n, channels = out.shape
     taps = weight.shape[0]
     _dev(weight, torch.float32, "causal_conv weight"); _dev(bias, torch.float32, "causal_conv bias"); _dev(state, torch.float32, "causal_conv state")
-    if (x.shape != out.shape or x.stride(1) != 1 or out.stride(1) != 1 or out.dtype != x.dtype or weight.shape[1] != channels
+    if (x.shape != out.shape or x.stride(1) != 1 or out.stride(1) != 1 or out.dtype not in (x.dtype, torch.float32) or weight.shape[1] != channels
             or state.dim() != 2 or not 0 <= history_off <= state.shape[1] - (taps - 1) * channels):
         raise KernelError(f"causal_conv: [N, {channels}] rows of one dtype and a slot with room for {taps - 1} rows behind {history_off}")
     _check(_typed("q25_rglru_causal_conv", x.dtype)(
         x.data_ptr(), x.stride(0), weight.data_ptr(), bias.data_ptr(), state.data_ptr() + 4 * int(history_off), state.shape[1], cu_q.data_ptr(),
-        slot_ids.data_ptr(), out.data_ptr(), out.stride(0), int(n_seqs), int(max_q_len), channels, taps, int(bool(silu)), _stream()), "causal_conv")
+        slot_ids.data_ptr(), out.data_ptr(), out.stride(0), int(n_seqs), int(max_q_len), channels, taps, int(bool(silu)),
+        int(out.dtype == torch.float32), _stream()), "causal_conv")
 
 
 # ---- attention with a distance bias, kept first tokens and values of their own size ---------------------
@@ -927,25 +919,23 @@ def rotary_apply(src: torch.Tensor, dst: torch.Tensor, heads: int, width: int, a
 
 
 def latent_store(x: torch.Tensor, rank: int, rot: int, norm_weight: torch.Tensor, eps: float, angles: Optional[torch.Tensor],
-                 layout: str, pages: torch.Tensor, kv_slot: torch.Tensor) -> None:
+                 layout: str, pages: Optional[torch.Tensor], kv_slot: Optional[torch.Tensor], q_latent: Optional[torch.Tensor] = None,
+                 q_weight: Optional[torch.Tensor] = None, q_out: Optional[torch.Tensor] = None) -> None:
     """Rows of ``x`` [N, rank + rot] (a strided view) -> cache rows [rank + rot] at ``kv_slot``: the first
-    ``rank`` channels RMS-normed with the weight, the last ``rot`` rotated by ``angles``."""
+    ``rank`` channels RMS-normed with the weight, the last ``rot`` rotated by ``angles``; pages None: none are written.
+    ``q_latent`` (a strided view [N, q_rank]): ``q_out`` = rmsnorm(q_latent) * q_weight in the same launch."""
     _dev(norm_weight, torch.float32, "latent_store weight")
-    if x.stride(1) != 1 or x.shape[1] != rank + rot or pages.dtype != x.dtype or pages.shape[-1] != rank + rot:
+    if x.stride(1) != 1 or x.shape[1] != rank + rot or (pages is not None and (pages.dtype != x.dtype or pages.shape[-1] != rank + rot)):
         raise KernelError(f"latent_store: rows and pages must hold {rank} + {rot} channels of one dtype")
+    if q_latent is not None:
+        _dev(q_weight, torch.float32, "latent_store query weight"); _dev(q_out, x.dtype, "latent_store query latent")
+        if q_latent.stride(1) != 1 or q_latent.dtype != x.dtype or q_out.shape != q_latent.shape or q_weight.numel() != q_latent.shape[1]:
+            raise KernelError("latent_store: the queries' latents are rows of one size with a weight per channel")
     half = 0 if angles is None else angles.shape[1]
     _check(_typed("q25_latent_store", x.dtype)(x.data_ptr(), x.stride(0), rank, rot, norm_weight.data_ptr(), float(eps), _ptr(angles),
-                                               half, ROTARY_LAYOUTS[layout], pages.data_ptr(), kv_slot.data_ptr(), x.shape[0],
-                                               _stream()), "latent_store")
-
-
-def latent_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
-    """out = rmsnorm(x) * weight for the strided rows ``x`` [N, C]."""
-    _dev(weight, torch.float32, "latent_norm weight"); _dev(out, x.dtype, "latent_norm out")
-    if x.stride(1) != 1 or out.shape != x.shape or weight.numel() != x.shape[1]:
-        raise KernelError("latent_norm: rows of one size and a weight per channel")
-    _check(_typed("q25_latent_norm", x.dtype)(x.data_ptr(), x.stride(0), x.shape[1], weight.data_ptr(), float(eps), out.data_ptr(), x.shape[0],
-                                              _stream()), "latent_norm")
+                                               half, ROTARY_LAYOUTS[layout], _ptr(pages), _ptr(kv_slot), x.shape[0], _ptr(q_latent),
+                                               0 if q_latent is None else q_latent.stride(0), 0 if q_latent is None else q_latent.shape[1],
+                                               _ptr(q_weight), _ptr(q_out), _stream()), "latent_store")
 
 
 def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor) -> None:

@@ -457,17 +457,14 @@ class LatentAttention(Mixer):
         qd = self.in_proj(h)                                        # [N, H (D + R) or q_rank | C + R | gate]
         q_cols = self.q_rank or H * (D + R)
         down = qd[:, q_cols:q_cols + C + R]
-        if self.q_rank:
-            c_q = torch.empty((n, self.q_rank), dtype=qd.dtype, device=qd.device)
-            kernels.latent_norm(qd[:, :self.q_rank], self.q_norm_weight, self.norm_eps, c_q)
-            q = self.uq_proj(c_q).unflatten(1, (H, D + R))
-        else:
-            q = qd[:, :q_cols].unflatten(1, (H, D + R))
         kv = ctx.kv(stop)
         angles = self.position.angles(ctx) if self.position is not None else None
         layout = self.position.layout if self.position is not None else "interleaved"
-        if stop.owns_cache:
-            kernels.latent_store(down, C, R, self.norm_weight, self.norm_eps, angles, layout, kv.k_pages, kv.kv_slot)
+        c_q = torch.empty((n, self.q_rank), dtype=qd.dtype, device=qd.device) if self.q_rank else None
+        if stop.owns_cache or self.q_rank:
+            kernels.latent_store(down, C, R, self.norm_weight, self.norm_eps, angles, layout, kv.k_pages if stop.owns_cache else None, kv.kv_slot,
+                                 qd[:, :self.q_rank] if self.q_rank else None, self.q_norm_weight if self.q_rank else None, c_q)
+        q = (self.uq_proj(c_q) if self.q_rank else qd[:, :q_cols]).unflatten(1, (H, D + R))
         # every head's query in the latent space, then its rotated part: rows of C + R channels like the cached ones
         q_lat = torch.empty((n, H, C + R), dtype=qd.dtype, device=qd.device)
         self._per_head(q[:, :, :D], self.uk_t, q_lat[:, :, :C])

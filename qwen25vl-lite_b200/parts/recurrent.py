@@ -9,7 +9,7 @@ channels are cut into ``blocks`` equal parts; in each, two gates from square mat
 ``a = exp(-gain * r * softplus(lam))`` and ``S_t = a S_(t-1) + sqrt(1 - a^2) * i * u`` from S = 0, and
 the mixer returns ``Wo (S * y)``.
 
-What is float32 in both dtypes: u, the gates and their products (plain FMA chains, so that a
+What is float32 in both dtypes: u, the gates and their products (sums in an order of their own, so that a
 token's gates do not depend on the batch), the decay, S.  The request's state is S and the last
 ``conv - 1`` inputs of the convolution, one float32 tensor [conv, width] per slot, zero at
 admission (the zeros before the start), carried from step to step.
@@ -27,6 +27,7 @@ from .base import Mixer, StateNeed, TensorSpec, register_mixer
 @register_mixer("rglru")
 class RGLRU(Mixer):
     graph_safe = True                # forward is a fixed sequence of this engine's kernels
+    gates16 = None
 
     def __init__(self, hidden_size: int, width: int, blocks: int, conv: int, gain: float = 8.0, position=None):
         self.hidden_size, self.width, self.blocks, self.conv = int(hidden_size), int(width), int(blocks), int(conv)
@@ -55,16 +56,24 @@ class RGLRU(Mixer):
         b = torch.cat([tensors["y.b"], tensors["x.b"]], dim=0).to(device=device, dtype=torch.float32).contiguous()
         self.in_proj = Linear(w, b)
         self.out_proj = Linear(tensors["o"].to(device=device, dtype=dtype).contiguous())
-        self.conv_w, self.conv_b = f32("conv"), f32("conv.b")
+        self.conv_w, self.conv_b = f32("conv").t().contiguous(), f32("conv.b")                # [taps, width]
         self.ra, self.ra_b, self.ri, self.ri_b, self.lam = f32("ra"), f32("ra.b"), f32("ri"), f32("ri.b"), f32("lam")
+        # long bfloat16 steps take the gates' products to the tensor cores, when the matrices are bfloat16 numbers as they are
+        self.gates16 = None
+        if dtype == torch.bfloat16 and (self.width // self.blocks) % 8 == 0:
+            pair = tuple(m.to(torch.bfloat16) for m in (self.ra, self.ri))
+            if all(bool((h.float() == m).all()) for h, m in zip(pair, (self.ra, self.ri))):
+                self.gates16 = pair
 
     def forward(self, ctx, h, stop):
         n, w = h.shape[0], self.width
         yx = self.in_proj(h)                                    # [N, 2 width]: the y branch, then the convolution's input
         u = torch.empty((n, w), dtype=torch.float32, device=h.device)
-        kernels.rglru_conv(yx, w, self.conv_w, self.conv_b, stop.state, ctx.token_seq, ctx.cu_q, ctx.slot_ids, u)
+        kernels.causal_conv(yx[:, w:], self.conv_w, self.conv_b, stop.state.view(stop.state.shape[0], -1), w, ctx.cu_q, ctx.slot_ids, u, ctx.n_seqs,
+                            ctx.max_q_len, silu=False)
         a, bx = torch.empty_like(u), torch.empty_like(u)
-        kernels.rglru_gates(u, self.ra, self.ra_b, self.ri, self.ri_b, self.lam, self.gain, a, bx)
+        ra, ri = self.gates16 if self.gates16 is not None and n > kernels.RGLRU_MMA_ROWS else (self.ra, self.ri)
+        kernels.rglru_gates(u, ra, self.ra_b, ri, self.ri_b, self.lam, self.gain, a, bx)
         out = torch.empty((n, w), dtype=ctx.dtype, device=h.device)
-        kernels.rglru_scan(a, bx, yx, 0, w, stop.state, ctx.cu_q, ctx.slot_ids, out, ctx.n_seqs, ctx.max_q_len)
+        kernels.rglru_scan(a, bx, yx, 0, stop.state, ctx.cu_q, ctx.slot_ids, out, ctx.n_seqs, ctx.max_q_len)
         return self.out_proj(out)

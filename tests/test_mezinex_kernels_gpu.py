@@ -102,7 +102,7 @@ def portions_of(total, sizes):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("channels,taps", [(96, 4), (75, 3), (64, 1), (130, 2), (33, 7), (40, 16)])
-@pytest.mark.parametrize("silu", [True, False])
+@pytest.mark.parametrize("silu", [True, False])            # False: the result in float32
 def test_convolution_over_portions(dtype, channels, taps, silu):
     """Two requests at once, one whole in long portions, one in portions shorter than the window; the history sits behind
     other state in the slots; what the slots hold elsewhere is left alone."""
@@ -118,7 +118,7 @@ def test_convolution_over_portions(dtype, channels, taps, silu):
         live = [i for i in range(2) if k < len(cuts[i])]
         lens = [cuts[i][k] for i in live]
         x = torch.cat([wide[i, at[i]:at[i] + n] for i, n in zip(live, lens)])[:, 4:4 + channels]
-        out = torch.empty(sum(lens), channels, dtype=dtype, device=DEV)
+        out = torch.empty(sum(lens), channels, dtype=dtype if silu else torch.float32, device=DEV)
         kernels.causal_conv(x, w, b, state, off, i32(np.cumsum([0] + lens)), i32([slots[i] for i in live]), out, len(live), max(lens), silu)
         for i, part in zip(live, torch.split(out, lens)):
             got[i].append(npy(part))
@@ -254,6 +254,33 @@ def test_state_space_output(dtype, H, V, parts):
     np.testing.assert_allclose(npy(out), want, **(dict(rtol=3e-5, atol=3e-5) if dtype == torch.float32 else dict(rtol=1e-2, atol=1e-2)))
 
 
+# ---- the recurrence's gates on tensor cores ----------------------------------------------------------------------------
+
+
+@pytest.mark.parametrize("n,width,blocks", [(129, 64, 4), (200, 96, 2), (150, 128, 1), (333, 240, 3), (64, 512, 2)])
+def test_gates_of_bfloat16_matrices_equal_the_float_products(n, width, blocks):
+    """u of many sizes, whose low bits weigh in: large entries that cancel in the product, beside small ones."""
+    g = torch.Generator(device=DEV).manual_seed(10)
+    bw = width // blocks
+    u = torch.randn(n, width, generator=g, device=DEV) * 10.0 ** torch.randint(-2, 2, (n, width), generator=g, device=DEV)
+    ra, ri = ((torch.randn(blocks, bw, bw, generator=g, device=DEV) * 0.2).bfloat16() for _ in range(2))
+    for m in (ra, ri):
+        m[:, :, 1] = -m[:, :, 0]
+    u[:, 1::bw] = u[:, 0::bw] * (1 + 2.0 ** -12)
+    u[:, 0::bw] *= 1.0
+    ra_b, ri_b, lam = (torch.randn(width, generator=g, device=DEV) for _ in range(3))
+    a, bx, a0, bx0 = (torch.empty(n, width, device=DEV) for _ in range(4))
+    kernels.rglru_gates(u, ra, ra_b.view(blocks, bw), ri, ri_b.view(blocks, bw), lam, 8.0, a, bx)
+    kernels.rglru_gates(u, ra.float(), ra_b.view(blocks, bw), ri.float(), ri_b.view(blocks, bw), lam, 8.0, a0, bx0)
+    parts = npy(u).reshape(n, blocks, bw)
+    gate = lambda m, b: plain.sigmoid(np.einsum("tbi,boi->tbo", parts, npy(m)).reshape(n, width) + npy(b))
+    log_a = -8.0 * gate(ra, ra_b) * plain.softplus(npy(lam))
+    want_a, want_b = np.exp(log_a), np.sqrt(-np.expm1(2 * log_a)) * gate(ri, ri_b) * npy(u)
+    for got_a, got_b in ((a, bx), (a0, bx0)):
+        np.testing.assert_allclose(npy(got_a), want_a, rtol=2e-4, atol=2e-6)
+        np.testing.assert_allclose(npy(got_b), want_b, rtol=2e-4, atol=2e-6)
+
+
 # ---- the latents ----------------------------------------------------------------------------------------------------
 
 
@@ -264,9 +291,16 @@ def test_query_latent_norm_and_output_gate(dtype, channels):
     wide = (torch.randn(11, channels + 5, generator=g, device=DEV) * 3).to(dtype)
     w = torch.randn(channels, generator=g, device=DEV) + 1.0
     out = torch.empty(11, channels, dtype=dtype, device=DEV)
-    kernels.latent_norm(wide[:, 3:3 + channels], w, 1e-2, out)
+    down, dw = torch.randn(11, 20, generator=g, device=DEV).to(dtype), torch.ones(12, device=DEV)
+    pages = torch.zeros(2, 1, 8, 20, dtype=dtype, device=DEV)
     tol = dict(rtol=1e-5, atol=1e-5) if dtype == torch.float32 else dict(rtol=1e-2, atol=1e-2)
-    np.testing.assert_allclose(npy(out), plain.rms_unit(npy(wide[:, 3:3 + channels]), 1e-2) * npy(w), **tol)
+    for own in (True, False):                                   # with and without a cache row of its own
+        out.zero_()
+        kernels.latent_store(down, 12, 8, dw, 1e-2, None, "interleaved", pages if own else None, i32(np.arange(11) + 3), wide[:, 3:3 + channels], w, out)
+        np.testing.assert_allclose(npy(out), plain.rms_unit(npy(wide[:, 3:3 + channels]), 1e-2) * npy(w), **tol)
+    row = np.concatenate([plain.rms_unit(npy(down)[:, :12], 1e-2), npy(down)[:, 12:]], axis=1)
+    np.testing.assert_allclose(npy(pages).reshape(16, 20)[3:14], row, **tol)
+    assert (pages.view(16, 20)[:3] == 0).all() and (pages.view(16, 20)[14:] == 0).all()
     y = torch.randn(11, channels, generator=g, device=DEV).to(dtype)
     want = npy(y) * plain.sigmoid(npy(wide[:, 5:]))
     kernels.sigmoid_gate(y, wide[:, 5:])

@@ -129,9 +129,10 @@ def test_recurrence_in_portions_with_state(dtype, width, blocks, taps):
         slots = torch.tensor([slot[k] for k in names], dtype=torch.int32, device=DEV)
         u, a, bx = (torch.empty(n, width, device=DEV) for _ in range(3))
         out = torch.empty(n, width, dtype=dtype, device=DEV)
-        kernels.rglru_conv(rows, width, conv_w, conv_b, state, token_seq, cu, slots, u)
+        kernels.causal_conv(rows[:, width:], conv_w.t().contiguous(), conv_b, state.view(state.shape[0], -1), width, cu, slots, u, len(names), max(step.values()),
+                            silu=False)
         kernels.rglru_gates(u, ra, ra_b, ri, ri_b, lam, 8.0, a, bx)
-        kernels.rglru_scan(a, bx, rows, 0, width, state, cu, slots, out, len(names), max(step.values()))
+        kernels.rglru_scan(a, bx, rows, 0, state, cu, slots, out, len(names), max(step.values()))
         at = 0
         for k in names:
             got[k].append(out[at:at + step[k]])
