@@ -570,7 +570,7 @@ def _mezinex_sizes(width, layers, ssm_heads, groups, latent_heads, latent_dim, r
                                                     "q_rank": q_rank, "scale": (latent_dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 10000.0}}}
     rec = {"type": "rglru", "mixer": {"width": width, "blocks": blocks, "conv": 4}}
     ours = {"architecture": "Mezinex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": streams, "logit_scale": 1.0,
-            "embedding": {"bigram": {"buckets": 4093, "mul_prev": 31, "mul_cur": 17}}, "layers": [dict((ssm, latent, rec)[i % 3], mlp=mlp) for i in range(layers)]}
+            "embedding": {"bigram": {"buckets": 4093, "mul_prev": 37, "mul_cur": 19}}, "layers": [dict((ssm, latent, rec)[i % 3], mlp=mlp) for i in range(layers)]}
     heads = width // 128
     closest = _sizes(width, layers, heads, max(2, heads // 8), ff, vocab, False)
     closest["text_config"]["rope_scaling"]["mrope_section"] = [16, 24, 24]

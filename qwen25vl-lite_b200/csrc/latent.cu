@@ -68,22 +68,33 @@ Q25_EXPORT int q25_latent_store_bf16(const void* x, int xr, int C, int R, const 
 }
 
 // y[n, c] *= sigmoid(g[n, c]), in place; y contiguous, g strided rows.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void latent_gate_kernel(T* __restrict__ y, const T* __restrict__ g, int g_row, int channels) {
   pdl_trigger();
   pdl_wait();
   const T* gr = g + (size_t)blockIdx.y * g_row;
   T* yr = y + (size_t)blockIdx.y * channels;
-  for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < channels; c += gridDim.x * blockDim.x)
-    yr[c] = from_f32<T>(to_f32(yr[c]) / (1.0f + expf(-to_f32(gr[c]))));
+  if (VEC) {
+    for (int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4; c < channels; c += gridDim.x * blockDim.x * 4) {
+      const float4 v = load4<T>(yr + c), z = load4<T>(gr + c);
+      store4<T>(yr + c, make_float4(v.x / (1.0f + expf(-z.x)), v.y / (1.0f + expf(-z.y)), v.z / (1.0f + expf(-z.z)), v.w / (1.0f + expf(-z.w))));
+    }
+  } else {
+    for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < channels; c += gridDim.x * blockDim.x)
+      yr[c] = from_f32<T>(to_f32(yr[c]) / (1.0f + expf(-to_f32(gr[c]))));
+  }
 }
 template <typename T>
 static int latent_gate(void* y, const void* g, int g_row, int n, int channels, void* stream) {
   if (n <= 0 || channels <= 0) return 0;
+  const bool vec = channels % 4 == 0 && g_row % 4 == 0 && !(((uintptr_t)y | (uintptr_t)g) & (4 * sizeof(T) - 1));
+  const dim3 block(256);
   for (int at = 0; at < n; at += 65535) {                         // the grid's second dimension ends at 65,535
-    const int rows = n - at < 65535 ? n - at : 65535;
-    launch(latent_gate_kernel<T>, dim3((channels + 1023) / 1024, rows), dim3(256), 0, (cudaStream_t)stream, (T*)y + (size_t)at * channels,
-           (const T*)g + (size_t)at * g_row, g_row, channels);
+    const dim3 grid((channels + 1023) / 1024, n - at < 65535 ? n - at : 65535);
+    T* yy = (T*)y + (size_t)at * channels;
+    const T* gg = (const T*)g + (size_t)at * g_row;
+    if (vec) launch(latent_gate_kernel<T, true>, grid, block, 0, (cudaStream_t)stream, yy, gg, g_row, channels);
+    else launch(latent_gate_kernel<T, false>, grid, block, 0, (cudaStream_t)stream, yy, gg, g_row, channels);
   }
   return launch_status();
 }

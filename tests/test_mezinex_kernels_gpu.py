@@ -56,7 +56,7 @@ def test_stream_is_written_and_read(dtype, streams, width):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("buckets,mul_prev,mul_cur", [(509, 31, 17), (7, 900_000_007, 4_000_000_019), (1, 2, 3)])
+@pytest.mark.parametrize("buckets,mul_prev,mul_cur", [(601, 29, 13), (7, 900_000_007, 4_000_000_019), (1, 2, 3)])
 def test_pairs_of_tokens_across_cuts_and_slots(dtype, buckets, mul_prev, mul_cur):
     """Three requests in turns of uneven portions through slots in another order than the batch; then one slot is used
     again by a new request, whose first token must not see the old one's last."""
@@ -167,7 +167,7 @@ def run_ssd(rows, steps, bias, a_log, H, G, N, V, lens, starts, slots, state, te
 
 
 SSD_SIZES = [(4, 2, 32, 16), (6, 3, 24, 20), (5, 5, 10, 14), (3, 1, 128, 64), (2, 1, 64, 64), (4, 1, 128, 128), (2, 2, 160, 40), (8, 1, 64, 32),
-             (8, 2, 32, 48), (6, 3, 128, 40), (96, 4, 64, 64), (90, 1, 128, 64)]
+             (6, 2, 32, 56), (6, 3, 128, 40), (96, 4, 64, 64), (90, 1, 128, 64)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -285,10 +285,10 @@ def test_gates_of_bfloat16_matrices_equal_the_float_products(n, width, blocks):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("channels", [7, 64, 80, 1536])
+@pytest.mark.parametrize("channels", [7, 64, 88, 1536])
 def test_query_latent_norm_and_output_gate(dtype, channels):
     g = torch.Generator(device=DEV).manual_seed(8)
-    wide = (torch.randn(11, channels + 5, generator=g, device=DEV) * 3).to(dtype)
+    wide = (torch.randn(11, channels + 8, generator=g, device=DEV) * 3).to(dtype)
     w = torch.randn(channels, generator=g, device=DEV) + 1.0
     out = torch.empty(11, channels, dtype=dtype, device=DEV)
     down, dw = torch.randn(11, 20, generator=g, device=DEV).to(dtype), torch.ones(12, device=DEV)
@@ -302,13 +302,14 @@ def test_query_latent_norm_and_output_gate(dtype, channels):
     np.testing.assert_allclose(npy(pages).reshape(16, 20)[3:14], row, **tol)
     assert (pages.view(16, 20)[:3] == 0).all() and (pages.view(16, 20)[14:] == 0).all()
     y = torch.randn(11, channels, generator=g, device=DEV).to(dtype)
-    want = npy(y) * plain.sigmoid(npy(wide[:, 5:]))
-    kernels.sigmoid_gate(y, wide[:, 5:])
-    np.testing.assert_allclose(npy(y), want, **tol)
+    for off in (5, 4):                                          # rows that start where four channels can be read at once, and not
+        want = npy(y) * plain.sigmoid(npy(wide[:, off:off + channels]))
+        kernels.sigmoid_gate(y, wide[:, off:off + channels])
+        np.testing.assert_allclose(npy(y), want, **tol)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,rank,rot", [(4, 64, 32), (3, 24, 12), (20, 64, 32), (16, 128, 64)])
+@pytest.mark.parametrize("heads,rank,rot", [(5, 64, 32), (3, 24, 12), (20, 64, 32), (16, 128, 64)])
 def test_one_far_latent_carries_the_weight(dtype, heads, rank, rot):
     """Queries of runs and of single tokens whose score on one cached row stands out by 30 among hundreds: the first row, rows
     at a page's border, the row of the token itself; a row beyond the token (a later one of its own run) made to stand

@@ -58,7 +58,7 @@ Z1 = _config(211, 96, 1e-5, 3, 0.7, (37, 5, 3), [
 # width 128, two rows, no loop: a latent of tensor-core sizes first, a state of 64 shared by all heads, one norm part,
 # three taps, multipliers whose products leave 32 bits
 Z2 = _config(300, 128, 1e-6, 2, 3.0, (97, 900_000_007, 12_345), [
-    _latent(4, 32, 32, 48, 64, 40, 0.2, 10000.0, 72), _ssm(4, 32, 64, 1, 1, 3, 80), _rec(128, 1, 4, 64)], None)
+    _latent(5, 32, 32, 40, 64, 56, 0.14, 10000.0, 72), _ssm(4, 32, 64, 1, 1, 3, 80), _rec(128, 1, 4, 64)], None)
 # nothing a multiple of 8: width 100, one row, no pair table; the recurrence alone runs twice; no sharing of B and C, a
 # convolution of one tap, a norm in 7 parts that straddle the heads
 Z3 = _config(77, 100, 1e-5, 1, 1.0, None, [
