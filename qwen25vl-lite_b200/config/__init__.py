@@ -9,3 +9,4 @@ from .rirulix_config import RirulixConfig  # noqa: F401
 from .labolix_config import LabolixConfig  # noqa: F401
 from .fatilix_config import FatilixConfig  # noqa: F401
 from .mezinex_config import MezinexConfig  # noqa: F401
+from .sudilorn_config import SudilornConfig  # noqa: F401

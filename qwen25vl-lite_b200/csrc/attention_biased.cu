@@ -32,7 +32,7 @@ __global__ void biased_attention_generic_kernel(
     const int* __restrict__ token_seq, const int* __restrict__ cu_q, const int* __restrict__ q_start_pos,
     int n_tokens, int nq, int nkv, int dk, int dv, int page_size, int window, int keep_first, float scale,
     const float* __restrict__ r1, const float* __restrict__ r2, const float* __restrict__ sink, int v_row, float softcap,
-    const float* __restrict__ dist_bias, int dist_rows, int gate_off) {
+    const float* __restrict__ dist_bias, int dist_rows, int gate_off, int out_stride) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char att_smem[];
@@ -106,7 +106,7 @@ __global__ void biased_attention_generic_kernel(
       __syncwarp();
     }
   }
-  T* o = out + (size_t)token * nq * dv + (size_t)head * dv;
+  T* o = out + (size_t)token * out_stride + (size_t)head * dv;
   if (sink) l += expf(sink[head] - m);                // a score without key or value: it only takes its share of the weight
   const float inv_l = 1.0f / l;
   const T* gate = gate_off >= 0 ? qkv + (size_t)token * qkv_stride + gate_off + (size_t)head * dv : nullptr;
@@ -156,7 +156,7 @@ static int biased_attention_generic(const void* qkv, int qkv_stride, void* out, 
                                     const int* block_table, int table_width, const int* token_seq, const int* cu_q,
                                     const int* q_start_pos, int n_tokens, int nq, int nkv, int dk, int dv, int page_size,
                                     int window, int keep_first, float scale, const float* r1, const float* r2, const float* sink,
-                                    int v_row, float softcap, const float* dist_bias, int dist_rows, int gate_off, void* stream) {
+                                    int v_row, float softcap, const float* dist_bias, int dist_rows, int gate_off, int out_stride, void* stream) {
   if (n_tokens <= 0) return 0;
   if (v_row <= 0) v_row = dv;
   if (dk <= 0 || dv <= 0 || dv > BATT_MAX_D || dk > 4096 || nkv <= 0 || nq % nkv || window < 0 || keep_first < 0 ||
@@ -171,7 +171,7 @@ static int biased_attention_generic(const void* qkv, int qkv_stride, void* out, 
   }
   launch(biased_attention_generic_kernel<T>, dim3(blocks), dim3(BATT_WARPS * 32), smem, (cudaStream_t)stream, (const T*)qkv,
          qkv_stride, (T*)out, (const T*)kpages, (const T*)vpages, block_table, table_width, token_seq, cu_q, q_start_pos, n_tokens,
-         nq, nkv, dk, dv, page_size, window, keep_first, scale, r1, r2, sink, v_row, softcap, dist_bias, dist_rows, gate_off);
+         nq, nkv, dk, dv, page_size, window, keep_first, scale, r1, r2, sink, v_row, softcap, dist_bias, dist_rows, gate_off, out_stride);
   return launch_status();
 }
 
@@ -186,13 +186,13 @@ static int kv_store_mix(void* qkv, int qkv_stride, const void* v_other, int ld_o
 
 Q25_EXPORT int q25_biased_attention_generic_f32(const void* qkv, int qs, void* out, const void* kp, const void* vp, const int* bt,
         int tw, const int* ts, const int* cu, const int* sp, int n, int nq, int nkv, int dk, int dv, int ps, int window, int keep, float scale,
-        const float* r1, const float* r2, const float* sink, int v_row, float softcap, const float* db, int db_rows, int gate_off, void* s) {
-  return biased_attention_generic<float>(qkv, qs, out, kp, vp, bt, tw, ts, cu, sp, n, nq, nkv, dk, dv, ps, window, keep, scale, r1, r2, sink, v_row, softcap, db, db_rows, gate_off, s);
+        const float* r1, const float* r2, const float* sink, int v_row, float softcap, const float* db, int db_rows, int gate_off, int os, void* s) {
+  return biased_attention_generic<float>(qkv, qs, out, kp, vp, bt, tw, ts, cu, sp, n, nq, nkv, dk, dv, ps, window, keep, scale, r1, r2, sink, v_row, softcap, db, db_rows, gate_off, os, s);
 }
 Q25_EXPORT int q25_biased_attention_generic_bf16(const void* qkv, int qs, void* out, const void* kp, const void* vp, const int* bt,
         int tw, const int* ts, const int* cu, const int* sp, int n, int nq, int nkv, int dk, int dv, int ps, int window, int keep, float scale,
-        const float* r1, const float* r2, const float* sink, int v_row, float softcap, const float* db, int db_rows, int gate_off, void* s) {
-  return biased_attention_generic<bf16>(qkv, qs, out, kp, vp, bt, tw, ts, cu, sp, n, nq, nkv, dk, dv, ps, window, keep, scale, r1, r2, sink, v_row, softcap, db, db_rows, gate_off, s);
+        const float* r1, const float* r2, const float* sink, int v_row, float softcap, const float* db, int db_rows, int gate_off, int os, void* s) {
+  return biased_attention_generic<bf16>(qkv, qs, out, kp, vp, bt, tw, ts, cu, sp, n, nq, nkv, dk, dv, ps, window, keep, scale, r1, r2, sink, v_row, softcap, db, db_rows, gate_off, os, s);
 }
 Q25_EXPORT int q25_kv_store_mix_f32(void* qkv, int qs, const void* vo, int ldo, float mix, void* kp, void* vp, const int* slot, int n,
                                     int nq, int nkv, int dk, int dv, int ps, void* s) {
@@ -212,13 +212,14 @@ Q25_EXPORT int q25_kv_store_mix_bf16(void* qkv, int qs, const void* vo, int ldo,
 // 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1), p its position (a query temperature that grows with the
 // context).  Queries are written back in place.  Keys go to their page slot normed and turned; with keys_as_values
 // the key as projected (before norm and rotation) is the token's value and goes to the value pages; with dv > 0 the
-// row's own values go there.  Statistics, weights, angles and the temperature in float.
+// row's own values go there.  pack: that many neighbouring key heads make up one wide key row of the cache, side by side
+// (its key/value heads are nkv / pack).  Statistics, weights, angles and the temperature in float.
 template <typename T>
 __global__ void qk_norm_store_kernel(T* __restrict__ qk, int qk_stride, const float* __restrict__ wq, const float* __restrict__ wk,
                                      float eps, int unit_norm, const float* __restrict__ angles, int half, int layout,
                                      const int* __restrict__ positions, float temp_coef, int temp_every, T* __restrict__ kpages,
                                      T* __restrict__ vpages, const int* __restrict__ kv_slot, int nq, int nkv, int dk, int dv,
-                                     int page_size, int keys_as_values) {
+                                     int page_size, int keys_as_values, int pack) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) float qkn_smem[];        // a row of dk floats per warp
@@ -229,11 +230,13 @@ __global__ void qk_norm_store_kernel(T* __restrict__ qk, int qk_stride, const fl
   const int page = slot / page_size, in_page = slot % page_size;
   const float* ang = half > 0 ? angles + (size_t)n * half * 2 : nullptr;
   const float temper = temp_every > 0 ? 1.0f + temp_coef * logf((float)((positions[n] + 1) / temp_every) + 1.0f) : 1.0f;
+  const int kvs = nkv / pack;                            // key/value heads of the cache
   for (int head = blockIdx.y * n_warps + warp; head < nq + nkv; head += gridDim.y * n_warps) {
     T* row = qk + (size_t)n * qk_stride + (size_t)head * dk;
     const bool is_key = head >= nq;
     const float* w = is_key ? wk : wq;
-    const size_t page_row = is_key ? ((size_t)page * nkv + (head - nq)) * page_size + in_page : 0;
+    const size_t page_row = is_key ? ((size_t)page * kvs + (head - nq) / pack) * page_size + in_page : 0;
+    T* krow = kpages + (page_row * pack + (is_key ? (head - nq) % pack : 0)) * dk;
     float sq = 0.f;
     for (int c = lane; c < dk; c += 32) {
       const float v = to_f32(row[c]);
@@ -249,15 +252,15 @@ __global__ void qk_norm_store_kernel(T* __restrict__ qk, int qk_stride, const fl
     __syncwarp();
     for (int c = lane; c < dk; c += 32) {
       const float r = rotary_channel<float>(vals, c, half, layout, ang);
-      if (is_key) { if (slot >= 0) kpages[page_row * dk + c] = from_f32<T>(r); }
+      if (is_key) { if (slot >= 0) krow[c] = from_f32<T>(r); }
       else row[c] = from_f32<T>(r * temper);
     }
     __syncwarp();
   }
   if (dv > 0 && !keys_as_values && slot >= 0) {
     const T* vrow = qk + (size_t)n * qk_stride + (size_t)(nq + nkv) * dk;
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < nkv * dv; c += gridDim.y * blockDim.x)
-      vpages[(((size_t)page * nkv + c / dv) * page_size + in_page) * dv + c % dv] = vrow[c];
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < kvs * dv; c += gridDim.y * blockDim.x)
+      vpages[(((size_t)page * kvs + c / dv) * page_size + in_page) * dv + c % dv] = vrow[c];
   }
 }
 
@@ -287,12 +290,13 @@ template <typename T>
 __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, const float* __restrict__ wq, const float* __restrict__ wk,
                                           float eps, int unit_norm, const int* __restrict__ positions, float temp_coef, int temp_every,
                                           T* __restrict__ kpages, T* __restrict__ vpages, const int* __restrict__ kv_slot, int n_tokens,
-                                          int nq, int nkv, int dk, int dv, int page_size, int keys_as_values) {
+                                          int nq, int nkv, int dk, int dv, int page_size, int keys_as_values, int pack) {
   pdl_trigger();
   pdl_wait();
   typedef typename Raw4<T>::type R4;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int heads = nq + nkv + (dv > 0 && !keys_as_values ? nkv : 0);
+  const int kvs = nkv / pack;                            // key/value heads of the cache
+  const int heads = nq + nkv + (dv > 0 && !keys_as_values ? kvs : 0);
   const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
   if (item >= (long long)n_tokens * heads) return;
   const int n = (int)(item / heads), head = (int)(item % heads);
@@ -302,7 +306,7 @@ __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, con
     if (slot < 0) return;
     const int vh = head - nq - nkv;
     const T* src = qk + (size_t)n * qk_stride + (size_t)(nq + nkv) * dk + (size_t)vh * dv;
-    T* dst = vpages + (((size_t)page * nkv + vh) * page_size + in_page) * dv;
+    T* dst = vpages + (((size_t)page * kvs + vh) * page_size + in_page) * dv;
     if (dv % 4 == 0) {
       for (int c = lane * 4; c < dv; c += 128) *reinterpret_cast<R4*>(dst + c) = *reinterpret_cast<const R4*>(src + c);
     } else {
@@ -313,7 +317,8 @@ __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, con
   T* row = qk + (size_t)n * qk_stride + (size_t)head * dk;
   const bool is_key = head >= nq;
   const float* w = is_key ? wk : wq;
-  const size_t page_row = is_key ? ((size_t)page * nkv + (head - nq)) * page_size + in_page : 0;
+  const size_t page_row = is_key ? ((size_t)page * kvs + (head - nq) / pack) * page_size + in_page : 0;
+  T* krow = kpages + (page_row * pack + (is_key ? (head - nq) % pack : 0)) * dk;
   float4 v[QK_FLAT_CHUNKS];
   float sq = 0.f;
 #pragma unroll
@@ -339,7 +344,7 @@ __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, con
       if (!is_key) { x.x *= temper; x.y *= temper; x.z *= temper; x.w *= temper; }
       R4 raw;
       f32_raw4(x, raw);
-      *reinterpret_cast<R4*>(is_key ? kpages + page_row * dk + c : row + c) = raw;
+      *reinterpret_cast<R4*>(is_key ? krow + c : row + c) = raw;
     }
   }
 }
@@ -347,8 +352,9 @@ __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, con
 template <typename T>
 static int qk_norm_store(void* qk, int qk_stride, const float* wq, const float* wk, float eps, int unit_norm, const float* angles, int half,
                          int layout, const int* positions, float temp_coef, int temp_every, void* kpages, void* vpages, const int* kv_slot,
-                         int n_tokens, int nq, int nkv, int dk, int dv, int page_size, int keys_as_values, void* stream) {
+                         int n_tokens, int nq, int nkv, int dk, int dv, int page_size, int keys_as_values, int pack, void* stream) {
   if (n_tokens <= 0) return 0;
+  if (pack < 1 || nkv % pack || (pack > 1 && keys_as_values)) return (int)cudaErrorInvalidValue;
   if (half < 0 || 2 * half > dk || (layout != ROTARY_INTERLEAVED && layout != ROTARY_HALVES) || (half > 0 && !angles) || dk > 2048 ||
       temp_every < 0 || (temp_every > 0 && !positions) || dv < 0)
     return (int)cudaErrorInvalidValue;
@@ -356,28 +362,28 @@ static int qk_norm_store(void* qk, int qk_stride, const float* wq, const float* 
   const int chunk = 4;                                      // channels of a vector access
   const bool aligned = !(((uintptr_t)qk | (uintptr_t)kpages | (uintptr_t)vpages) & (4 * sizeof(T) - 1)) && !(((uintptr_t)wq | (uintptr_t)wk) & 15);
   if (half == 0 && dk % chunk == 0 && dk <= 128 * QK_FLAT_CHUNKS && qk_stride % chunk == 0 && aligned && (keys_as_values || dv % chunk == 0)) {
-    const long long heads = nq + nkv + (dv > 0 && !keys_as_values ? nkv : 0);
+    const long long heads = nq + nkv + (dv > 0 && !keys_as_values ? nkv / pack : 0);
     const unsigned blocks = (unsigned)(((long long)n_tokens * heads + 7) / 8);
     launch(qk_norm_store_flat_kernel<T>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (T*)qk, qk_stride, wq, wk, eps, unit_norm, positions,
-           temp_coef, temp_every, (T*)kpages, (T*)vpages, kv_slot, n_tokens, nq, nkv, dk, dv, page_size, keys_as_values);
+           temp_coef, temp_every, (T*)kpages, (T*)vpages, kv_slot, n_tokens, nq, nkv, dk, dv, page_size, keys_as_values, pack);
     return launch_status();
   }
   // as many blocks a token as its heads fill: a warp that walks several heads one after the other waits for each one's loads
   const int per_token = (nq + nkv + warps - 1) / warps;
   launch(qk_norm_store_kernel<T>, dim3(n_tokens, per_token), dim3(warps * 32), (size_t)warps * dk * sizeof(float), (cudaStream_t)stream, (T*)qk,
          qk_stride, wq, wk, eps, unit_norm, angles, half, layout, positions, temp_coef, temp_every, (T*)kpages, (T*)vpages, kv_slot, nq,
-         nkv, dk, dv, page_size, keys_as_values);
+         nkv, dk, dv, page_size, keys_as_values, pack);
   return launch_status();
 }
 Q25_EXPORT int q25_biased_attention_qk_norm_store_f32(void* qk, int qs, const float* wq, const float* wk, float eps, int unit, const float* ang,
         int half, int layout, const int* pos, float tc, int te, void* kp, void* vp, const int* slot, int n, int nq, int nkv, int dk, int dv,
-        int ps, int kav, void* s) {
-  return qk_norm_store<float>(qk, qs, wq, wk, eps, unit, ang, half, layout, pos, tc, te, kp, vp, slot, n, nq, nkv, dk, dv, ps, kav, s);
+        int ps, int kav, int pack, void* s) {
+  return qk_norm_store<float>(qk, qs, wq, wk, eps, unit, ang, half, layout, pos, tc, te, kp, vp, slot, n, nq, nkv, dk, dv, ps, kav, pack, s);
 }
 Q25_EXPORT int q25_biased_attention_qk_norm_store_bf16(void* qk, int qs, const float* wq, const float* wk, float eps, int unit, const float* ang,
         int half, int layout, const int* pos, float tc, int te, void* kp, void* vp, const int* slot, int n, int nq, int nkv, int dk, int dv,
-        int ps, int kav, void* s) {
-  return qk_norm_store<bf16>(qk, qs, wq, wk, eps, unit, ang, half, layout, pos, tc, te, kp, vp, slot, n, nq, nkv, dk, dv, ps, kav, s);
+        int ps, int kav, int pack, void* s) {
+  return qk_norm_store<bf16>(qk, qs, wq, wk, eps, unit, ang, half, layout, pos, tc, te, kp, vp, slot, n, nq, nkv, dk, dv, ps, kav, pack, s);
 }
 
 // ================================================================================================
@@ -398,12 +404,13 @@ Q25_EXPORT int q25_biased_attention_qk_norm_store_bf16(void* qk, int qs, const f
 // key range per token (long contexts) the ranges leave (max, sum, unnormalised output) in scratch
 // memory and a second kernel adds them up in order.
 // ================================================================================================
-#include "attention_decode.cuh"
+#include "attention_walk.cuh"
 
 struct BiasedArgs {
   const bf16* qkv;
   int qkv_stride;
   bf16* out;
+  int out_stride;      // channels between two tokens' results
   const bf16* kpages;
   const bf16* vpages;
   const int* block_table;
@@ -425,173 +432,6 @@ struct BiasedArgs {
   float* part_o;   // [items, nq, splits, DV]
   float* part_ml;  // [items, nq, splits, 2]
 };
-
-// sigmoid of two neighbouring gate channels (an even channel offset: one 32-bit load).
-__device__ __forceinline__ float2 gate_pair(const bf16* g) {
-  const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g));
-  return make_float2(1.0f / (1.0f + __expf(-z.x)), 1.0f / (1.0f + __expf(-z.y)));
-}
-__device__ __forceinline__ float gate_one(const bf16* g) { return 1.0f / (1.0f + __expf(-__bfloat162float(*g))); }
-
-// The tiles of keys that queries at positions p_first .. p_last walk.
-struct KeyWalk {
-  int kept, lo, hi, sink_tiles, win_key0, n_tiles;
-  __device__ __forceinline__ void set(int p_first, int p_last, int window, int keep_first, int bn) {
-    lo = window > 0 ? max(0, p_first - window + 1) : 0;
-    if (lo <= keep_first) lo = 0;
-    kept = lo > 0 ? keep_first : 0;
-    hi = p_last;
-    sink_tiles = (kept + bn - 1) / bn;
-    win_key0 = lo / bn * bn;
-    n_tiles = sink_tiles + (hi - win_key0) / bn + 1;
-  }
-  // first key of tile i, and the range of keys [rl, rh] that count in it
-  __device__ __forceinline__ void tile(int i, int bn, int& key0, int& rl, int& rh) const {
-    if (i < sink_tiles) { key0 = i * bn; rl = 0; rh = kept - 1; }
-    else { key0 = win_key0 + (i - sink_tiles) * bn; rl = lo; rh = hi; }
-  }
-};
-
-// Copies keys [key0, key0 + BN) of one kv head into K and V tiles (zeros past `last`), by NT threads:
-// NT / BN threads share a key, so a thread looks one page up and takes that row's 16-byte chunks
-// (of the key and of the value) in turn.
-template <int DK, int DV, int BN, int NT>
-__device__ __forceinline__ void biased_load_tile(unsigned char* ks, unsigned char* vs, const BiasedArgs& a, const int* table, int kvh,
-                                                 int key0, int last, int tid) {
-  constexpr int CK = DK / 8, CV = DV / 8, TPK = NT / BN;
-  static_assert(NT % BN == 0 && CK % TPK == 0 && CV % TPK == 0, "the chunks of a row divide among its threads");
-  const int key = tid / TPK, part = tid % TPK;
-  const int kidx = key0 + key;
-  const bool valid = kidx <= last;
-  const int kc = valid ? kidx : last;                       // a readable address also for the zero-filled rows
-  const int page = table[kc / a.page_size];
-  const size_t row = ((size_t)page * a.nkv + kvh) * a.page_size + kc % a.page_size;
-  const bf16* kr = a.kpages + row * DK;
-  const bf16* vr = a.vpages + row * a.v_row;
-#pragma unroll
-  for (int i = 0; i < CK / TPK; ++i) {
-    const int ch = part + i * TPK;
-    cp_async16(ks + key * Tile<DK>::PITCH + ch * 16, kr + ch * 8, valid);
-  }
-#pragma unroll
-  for (int i = 0; i < CV / TPK; ++i) {
-    const int ch = part + i * TPK;
-    cp_async16(vs + key * Tile<DV>::PITCH + ch * 16, vr + ch * 8, valid);
-  }
-}
-
-// One tile of keys for the warp's 16 rows.  p0/p1: positions of rows g and g+8 (-1: no such row);
-// b1x/b2x: the bias numbers of the rows' heads; [rl, rh]: the keys of the tile that count.  FULL: the
-// caller has seen that every key of the tile counts for every row of the warp, so nothing is masked.
-// TABLE: the rows' heads add tab0 / tab1 [min(distance, dist_rows - 1) * nq] to their scores (a build of
-// its own, so that the kernels without a table carry none of it).
-template <int DK, int DV, int BN, bool FULL, bool TABLE>
-__device__ __forceinline__ void biased_tile(const unsigned (&qf)[DK / 16][4], const unsigned char* ks, const unsigned char* vs,
-                                            int key0, int rl, int rh, int p0, int p1, int window, int keep_first, float scale_log2,
-                                            float cap_log2, float scale_over_cap, float b10, float b20, float b11, float b21,
-                                            const float* __restrict__ tab0, const float* __restrict__ tab1, int dist_rows, int nq,
-                                            float (&m)[2], float (&l)[2], float (&o)[DV / 8][4]) {
-  constexpr int PK = Tile<DK>::PITCH, PV = Tile<DV>::PITCH;
-  const int lane = threadIdx.x & 31, t = lane & 3;
-  float s[BN / 8][4];
-#pragma unroll
-  for (int j = 0; j < BN / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
-#pragma unroll
-  for (int kk = 0; kk < DK / 16; ++kk) {
-    unsigned b[BN / 8][2];
-#pragma unroll
-    for (int j = 0; j < BN / 8; ++j) ldmatrix_x2(b[j], ks + (j * 8 + (lane & 7)) * PK + (kk * 16 + 8 * ((lane >> 3) & 1)) * 2);
-#pragma unroll
-    for (int j = 0; j < BN / 8; ++j) mma_bf16(s[j], qf[kk], b[j][0], b[j][1]);
-  }
-  // distance of the row's query to the thread's first key of the tile, as a float; the other keys
-  // of the thread lie constants further on
-  const float d0 = (float)(p0 - key0 - 2 * t), d1 = (float)(p1 - key0 - 2 * t);
-  // the distance table: a row whose nearest key of the tile lies at the table's last row or beyond adds one number
-  // to all its scores; the table's entries are natural-log scores, the kernel's live in the base-2 domain
-  constexpr float LOG2E = 1.4426950408889634f;
-  const int last_row = dist_rows - 1;
-  const bool far0 = TABLE && p0 - (key0 + BN - 1) >= last_row, far1 = TABLE && p1 - (key0 + BN - 1) >= last_row;
-  const float fb0 = far0 ? tab0[(size_t)last_row * nq] * LOG2E : 0.f, fb1 = far1 ? tab1[(size_t)last_row * nq] * LOG2E : 0.f;
-  float mx0 = -INFINITY, mx1 = -INFINITY;
-#pragma unroll
-  for (int j = 0; j < BN / 8; ++j) {
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float fd = (e < 2 ? d0 : d1) - (float)(j * 8 + (e & 1));
-      const float b1 = e < 2 ? b10 : b11, b2 = e < 2 ? b20 : b21;
-      float v = cap_log2 > 0.f ? cap_log2 * tanhf(s[j][e] * scale_over_cap) - b1 * __log2f(fmaf(b2, fd, 1.0f))
-                               : fmaf(s[j][e], scale_log2, -b1 * __log2f(fmaf(b2, fd, 1.0f)));
-      if (TABLE) {
-        if (e < 2 ? far0 : far1) {
-          v += e < 2 ? fb0 : fb1;
-        } else {
-          const int dist = (e < 2 ? p0 : p1) - (key0 + j * 8 + 2 * t + (e & 1));
-          v = fmaf((e < 2 ? tab0 : tab1)[(size_t)min(max(dist, 0), last_row) * nq], LOG2E, v);
-        }
-      }
-      if (!FULL) {
-        const int kidx = key0 + j * 8 + 2 * t + (e & 1);
-        const int dist = (e < 2 ? p0 : p1) - kidx;
-        const bool ok = kidx >= rl && kidx <= rh && dist >= 0 && (window <= 0 || dist < window || kidx < keep_first);
-        v = ok ? v : -INFINITY;
-      }
-      s[j][e] = v;
-    }
-    mx0 = fmaxf(mx0, fmaxf(s[j][0], s[j][1]));
-    mx1 = fmaxf(mx1, fmaxf(s[j][2], s[j][3]));
-  }
-  mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-  mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-  mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-  mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-  const float mn0 = fmaxf(m[0], mx0), mn1 = fmaxf(m[1], mx1);
-  const float ms0 = mn0 == -INFINITY ? 0.f : mn0, ms1 = mn1 == -INFINITY ? 0.f : mn1;  // nothing seen yet
-  const float c0 = exp2f(m[0] - ms0), c1 = exp2f(m[1] - ms1);
-  m[0] = mn0;
-  m[1] = mn1;
-  float sum0 = 0.f, sum1 = 0.f;
-#pragma unroll
-  for (int j = 0; j < BN / 8; ++j) {
-    s[j][0] = exp2f(s[j][0] - ms0);
-    s[j][1] = exp2f(s[j][1] - ms0);
-    s[j][2] = exp2f(s[j][2] - ms1);
-    s[j][3] = exp2f(s[j][3] - ms1);
-    sum0 += s[j][0] + s[j][1];
-    sum1 += s[j][2] + s[j][3];
-  }
-  l[0] = l[0] * c0 + sum0;  // per-thread partial sums; the quad is reduced once at the end
-  l[1] = l[1] * c1 + sum1;
-#pragma unroll
-  for (int nb = 0; nb < DV / 8; ++nb) {
-    o[nb][0] *= c0;
-    o[nb][1] *= c0;
-    o[nb][2] *= c1;
-    o[nb][3] *= c1;
-  }
-#pragma unroll
-  for (int kk = 0; kk < BN / 16; ++kk) {
-    unsigned pa[4];
-    pa[0] = pack_bf16(s[2 * kk][0], s[2 * kk][1]);
-    pa[1] = pack_bf16(s[2 * kk][2], s[2 * kk][3]);
-    pa[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
-    pa[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
-    const unsigned char* vrow = vs + (kk * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * PV;
-#pragma unroll
-    for (int np = 0; np < DV / 16; ++np) {
-      unsigned b[4];
-      ldmatrix_x4_trans(b, vrow + (np * 16 + 8 * (lane >> 4)) * 2);
-      mma_bf16(o[2 * np], pa, b[0], b[1]);
-      mma_bf16(o[2 * np + 1], pa, b[2], b[3]);
-    }
-  }
-}
-
-// Whether every key of the tile [key0, key0 + bn) counts for every query of positions p_min .. p_max.
-__device__ __forceinline__ bool tile_is_full(int key0, int bn, int rl, int rh, int p_min, int p_max, int window, int keep_first) {
-  const int last = key0 + bn - 1;
-  return p_min >= 0 && last <= p_min && key0 >= rl && last <= rh && (window <= 0 || p_max - key0 < window || last < keep_first);
-}
 
 // EXTRA: what a build carries beyond scores, masks and sinks: 0 nothing, 1 the output gate, 2 the gate and the distance
 // table (kernels of models that have neither are built without a trace of them).
@@ -674,8 +514,8 @@ __global__ void __launch_bounds__(128) biased_prefill_kernel(BiasedArgs a) {
       if (g0) { const float2 z = gate_pair(g0 + c); y0 *= z.x; y1 *= z.y; }
       if (g1) { const float2 z = gate_pair(g1 + c); y2 *= z.x; y3 *= z.y; }
     }
-    if (tok0 >= 0) *reinterpret_cast<unsigned*>(a.out + (size_t)(first + tok0) * a.nq * DV + (size_t)h0 * DV + c) = pack_bf16(y0, y1);
-    if (tok1 >= 0) *reinterpret_cast<unsigned*>(a.out + (size_t)(first + tok1) * a.nq * DV + (size_t)h1 * DV + c) = pack_bf16(y2, y3);
+    if (tok0 >= 0) *reinterpret_cast<unsigned*>(a.out + (size_t)(first + tok0) * a.out_stride + (size_t)h0 * DV + c) = pack_bf16(y0, y1);
+    if (tok1 >= 0) *reinterpret_cast<unsigned*>(a.out + (size_t)(first + tok1) * a.out_stride + (size_t)h1 * DV + c) = pack_bf16(y2, y3);
   }
 }
 
@@ -771,7 +611,7 @@ __global__ void __launch_bounds__(128) biased_decode_kernel(BiasedArgs a) {
       if (a.sink && mm != -INFINITY) sum += exp2f(a.sink[head] * 1.4426950408889634f - mm);
       float y = sum > 0.f ? acc / sum : 0.f;
       if (GATE && a.gate_off >= 0) y *= gate_one(a.qkv + (size_t)token * a.qkv_stride + a.gate_off + (size_t)head * DV + c);
-      a.out[(size_t)token * a.nq * DV + (size_t)head * DV + c] = __float2bfloat16_rn(y);
+      a.out[(size_t)token * a.out_stride + (size_t)head * DV + c] = __float2bfloat16_rn(y);
     } else {
       const size_t at = ((size_t)item * a.nq + head) * a.n_splits + split;
       a.part_o[at * DV + c] = acc;
@@ -800,7 +640,7 @@ __global__ void biased_combine_kernel(BiasedArgs a) {
   if (a.sink && mm != -INFINITY) sum += exp2f(a.sink[head] * 1.4426950408889634f - mm);
   float y = sum > 0.f ? acc / sum : 0.f;
   if (a.gate_off >= 0) y *= gate_one(a.qkv + (size_t)token * a.qkv_stride + a.gate_off + (size_t)head * DV + c);
-  a.out[(size_t)token * a.nq * DV + (size_t)head * DV + c] = __float2bfloat16_rn(y);
+  a.out[(size_t)token * a.out_stride + (size_t)head * DV + c] = __float2bfloat16_rn(y);
 }
 
 template <int DK, int DV, int EXTRA>
@@ -850,13 +690,13 @@ Q25_EXPORT int q25_biased_attention_mma_bf16(const void* qkv, int qkv_stride, vo
                                              int n_items, int nq, int nkv, int dk, int dv, int ps, int window, int keep, float scale,
                                              const float* r1, const float* r2, const float* sink, int v_row, int n_splits, float* part_o,
                                              float* part_ml, float softcap, const float* dist_bias, int dist_rows, int gate_off,
-                                             void* stream) {
+                                             int out_stride, void* stream) {
   if (n_tiles <= 0 && n_items <= 0) return 0;
   if (nkv <= 0 || nq % nkv || ps <= 0 || n_splits < 1 || (n_items > 0 && nq / nkv > 16) || v_row % 8 || (dist_bias && dist_rows < 1) ||
-      (gate_off >= 0 && gate_off % 2))
+      (gate_off >= 0 && gate_off % 2) || out_stride % 2 || ((uintptr_t)out & 3))
     return (int)cudaErrorInvalidValue;
   BiasedArgs a;
-  a.qkv = (const bf16*)qkv; a.qkv_stride = qkv_stride; a.out = (bf16*)out; a.kpages = (const bf16*)kp; a.vpages = (const bf16*)vp;
+  a.qkv = (const bf16*)qkv; a.qkv_stride = qkv_stride; a.out = (bf16*)out; a.out_stride = out_stride; a.kpages = (const bf16*)kp; a.vpages = (const bf16*)vp;
   a.block_table = bt; a.table_width = tw; a.cu_q = cu; a.q_start_pos = sp; a.items = nullptr;
   a.nq = nq; a.nkv = nkv; a.page_size = ps; a.window = window; a.keep_first = keep;
   a.scale_log2 = scale * 1.4426950408889634f;

@@ -161,8 +161,9 @@ __global__ void embed_position_norm_kernel(const T* __restrict__ table, const T*
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = row_cache[c] * inv[c / width] * w[c];
 }
 
-// x[row] += d, where d = delta[row] as it is (dw == nullptr) or norm_in_groups(delta[row]) * dw (a
-// sublayer that is normalised after as well as before); then out[r] = norm_in_groups(x[row]) * w.
+// x[row] += d, where d = delta[row] as it is (dw == nullptr), norm_in_groups(delta[row]) * dw (a
+// sublayer that is normalised after as well as before), or delta[row] * dw (d_groups == 0: a scale per channel
+// and no norm); then out[r] = norm_in_groups(x[row]) * w.
 // rows as in add_rmsnorm_kernel: with rows the sum is formed for those rows only and x is left alone.
 // out == nullptr: only the addition.  w == nullptr: out[r] = x[row] as it is, in T (a sublayer that reads
 // the stream itself).
@@ -183,29 +184,30 @@ __global__ void add_norm_groups_kernel(float* __restrict__ x, const T* __restric
   constexpr int STEP = VEC ? 4 : 1;
   if (delta) {
     const T* dr = delta + (size_t)row * hidden;
-    if (dw) {
+    const bool d_norm = dw && d_groups > 0;
+    if (d_norm) {
       for (int c = threadIdx.x * STEP; c < hidden; c += blockDim.x * STEP) {
         if (VEC) *reinterpret_cast<float4*>(d_cache + c) = load4<T>(dr + c);
         else d_cache[c] = to_f32(dr[c]);
       }
       group_inverse_rms<EXACT>(d_cache, hidden, d_groups, d_eps, d_inv, scratch);
     }
-    const int dwidth = dw ? hidden / d_groups : hidden;
+    const int dwidth = d_norm ? hidden / d_groups : hidden;
     for (int c = threadIdx.x * STEP; c < hidden; c += blockDim.x * STEP) {
       if (VEC) {
         float4 v = *reinterpret_cast<const float4*>(xr + c);
-        if (dw) {
+        if (d_norm) {
           const float4 d = *reinterpret_cast<const float4*>(d_cache + c), ww = *reinterpret_cast<const float4*>(dw + c);
           const float s = d_inv[c / dwidth];
           v.x += d.x * s * ww.x; v.y += d.y * s * ww.y; v.z += d.z * s * ww.z; v.w += d.w * s * ww.w;
         } else {
-          const float4 d = load4<T>(dr + c);
-          v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+          const float4 d = load4<T>(dr + c), ww = dw ? *reinterpret_cast<const float4*>(dw + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+          v.x = fmaf(d.x, ww.x, v.x); v.y = fmaf(d.y, ww.y, v.y); v.z = fmaf(d.z, ww.z, v.z); v.w = fmaf(d.w, ww.w, v.w);
         }
         *reinterpret_cast<float4*>(row_cache + c) = v;
         if (!rows) *reinterpret_cast<float4*>(xr + c) = v;
       } else {
-        const float v = xr[c] + (dw ? d_cache[c] * d_inv[c / dwidth] * dw[c] : to_f32(dr[c]));
+        const float v = xr[c] + (d_norm ? d_cache[c] * d_inv[c / dwidth] * dw[c] : dw ? to_f32(dr[c]) * dw[c] : to_f32(dr[c]));
         row_cache[c] = v;
         if (!rows) xr[c] = v;
       }
@@ -339,7 +341,7 @@ static int add_norm_groups(float* x, const void* delta, const float* dw, float d
                            int groups, void* out, const int* rows, int n_out, int hidden, void* stream) {
   if (n_out <= 0) return 0;
   if (groups <= 0 || groups > NORM_MAX_GROUPS || hidden % groups) return (int)cudaErrorInvalidValue;
-  if (dw && (d_groups <= 0 || d_groups > NORM_MAX_GROUPS || hidden % d_groups)) return (int)cudaErrorInvalidValue;
+  if (dw && (d_groups < 0 || d_groups > NORM_MAX_GROUPS || (d_groups && hidden % d_groups))) return (int)cudaErrorInvalidValue;
   const size_t smem = (size_t)(2 * hidden + 32 + 2 * NORM_MAX_GROUPS) * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   if (smem > 48 * 1024) {
@@ -349,7 +351,7 @@ static int add_norm_groups(float* x, const void* delta, const float* dw, float d
   }
   // four values at a time when every group (of the stream's norm and of the update's) is a multiple of
   // four wide and every row starts on a 16-byte boundary
-  const bool vec = hidden % 4 == 0 && (hidden / groups) % 4 == 0 && (!dw || (hidden / d_groups) % 4 == 0) &&
+  const bool vec = hidden % 4 == 0 && (hidden / groups) % 4 == 0 && (!dw || !d_groups || (hidden / d_groups) % 4 == 0) &&
                    !(((uintptr_t)x | (uintptr_t)delta | (uintptr_t)dw | (uintptr_t)w | (uintptr_t)out) & 15);
   const dim3 block(hidden >= 1024 ? 256 : 128);
   if (vec) launch(add_norm_groups_kernel<T, EXACT, true>, dim3(n_out), block, smem, (cudaStream_t)stream, x, (const T*)delta, dw, d_eps,

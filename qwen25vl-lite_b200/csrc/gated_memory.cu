@@ -375,7 +375,7 @@ __global__ void __launch_bounds__(256) memory_fold_kernel(MemoryArgs p, const in
 // A warp per (token, head).  act: 0 = silu of the gate channel, 1 = sigmoid.
 template <typename T>
 __global__ void memory_output_kernel(const float* __restrict__ o_raw, const float* __restrict__ m_exp, const T* __restrict__ x,
-                                     int x_stride, int g_off, const float* __restrict__ weight, T* __restrict__ out, int n_tokens,
+                                     int x_stride, int g_off, const float* __restrict__ weight, T* __restrict__ out, int out_stride, int n_tokens,
                                      int H, int Dv, int extra, float eps, int act) {
   pdl_trigger();
   pdl_wait();
@@ -391,7 +391,7 @@ __global__ void memory_output_kernel(const float* __restrict__ o_raw, const floa
   sq = warp_sum(sq);
   const float inv = inv_den / sqrtf(sq / (float)Dv + eps);
   const T* gate = x + (size_t)n * x_stride + g_off + head * Dv;
-  T* dst = out + ((size_t)n * H + head) * Dv;
+  T* dst = out + (size_t)n * out_stride + (size_t)head * Dv;
   for (int c = lane; c < Dv; c += 32) {
     const float z = to_f32(gate[c]);
     const float s = 1.0f / (1.0f + expf(-z));
@@ -552,22 +552,22 @@ Q25_EXPORT int q25_memory_scan_bf16(const void* x, int xs, int qo, int ko, int v
 }
 
 template <typename T>
-static int memory_output(const float* o_raw, const float* m_exp, const void* x, int x_stride, int g_off, const float* weight, void* out,
+static int memory_output(const float* o_raw, const float* m_exp, const void* x, int x_stride, int g_off, const float* weight, void* out, int out_stride,
                          int n_tokens, int H, int Dv, int extra, float eps, int act, void* stream) {
   if (n_tokens <= 0) return 0;
   if (extra && !m_exp) return (int)cudaErrorInvalidValue;
   const long long items = (long long)n_tokens * H;
   launch(memory_output_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, (cudaStream_t)stream, o_raw, m_exp, (const T*)x, x_stride,
-         g_off, weight, (T*)out, n_tokens, H, Dv, extra, eps, act);
+         g_off, weight, (T*)out, out_stride, n_tokens, H, Dv, extra, eps, act);
   return launch_status();
 }
-Q25_EXPORT int q25_memory_output_f32(const float* o, const float* me, const void* x, int xs, int go, const float* w, void* out, int n, int H, int Dv,
+Q25_EXPORT int q25_memory_output_f32(const float* o, const float* me, const void* x, int xs, int go, const float* w, void* out, int os, int n, int H, int Dv,
                                      int extra, float eps, int act, void* s) {
-  return memory_output<float>(o, me, x, xs, go, w, out, n, H, Dv, extra, eps, act, s);
+  return memory_output<float>(o, me, x, xs, go, w, out, os, n, H, Dv, extra, eps, act, s);
 }
-Q25_EXPORT int q25_memory_output_bf16(const float* o, const float* me, const void* x, int xs, int go, const float* w, void* out, int n, int H, int Dv,
+Q25_EXPORT int q25_memory_output_bf16(const float* o, const float* me, const void* x, int xs, int go, const float* w, void* out, int os, int n, int H, int Dv,
                                       int extra, float eps, int act, void* s) {
-  return memory_output<bf16>(o, me, x, xs, go, w, out, n, H, Dv, extra, eps, act, s);
+  return memory_output<bf16>(o, me, x, xs, go, w, out, os, n, H, Dv, extra, eps, act, s);
 }
 
 // The state space of Mamba-2 by the same walk: x holds the values (heads side by side at v_off) and, per group of heads, k

@@ -57,8 +57,9 @@
 
 // EPI_GLU: the clamped gated unit g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit), in the
 // layout of EPI_SWIGLU; its two constants (limit, alpha) are read where EPI_BIAS reads its bias.
-// EPI_RELU2: the square of relu, max(y, 0)^2, stored in bfloat16.
-enum { EPI_STORE = 0, EPI_BIAS = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_RESIDUAL = 4, EPI_GLU = 5, EPI_RELU2 = 6 };
+// EPI_RELU2: the square of relu, max(y, 0)^2, stored in bfloat16.  EPI_RESIDUAL_SCALED: out += bias[n] * y, a scale per output
+// channel on the way into the float residual.
+enum { EPI_STORE = 0, EPI_BIAS = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_RESIDUAL = 4, EPI_GLU = 5, EPI_RELU2 = 6, EPI_RESIDUAL_SCALED = 7 };
 
 #define GC_ROWS 16
 #define GC_MAX_M 8                               // rows of x: one 8-column tile of the MMA (MT = 1).  A second tile
@@ -195,6 +196,9 @@ __device__ __forceinline__ void gc_store_group(const float (&acc)[MT][4], int gr
         else if (op.epi == EPI_RESIDUAL) {
           float* dst = reinterpret_cast<float*>(op.out) + (size_t)m * op.ldo + n;
           *dst = has_old ? v : __ldcg(dst) + v;       // has_old: the old value is in v already
+        } else if (op.epi == EPI_RESIDUAL_SCALED) {
+          float* dst = reinterpret_cast<float*>(op.out) + (size_t)m * op.ldo + n;
+          *dst = fmaf(op.bias[n], v, __ldcg(dst));
         }
         else reinterpret_cast<bf16*>(op.out)[(size_t)m * op.ldo + n] = __float2bfloat16_rn(v);
       }
@@ -745,8 +749,8 @@ static bool chain_cut(const ChainOpDesc& d, ChainOp& op, int sms, int limit, int
   if (d.M <= 0 || d.M > GC_MAX_M || d.N <= 0 || d.K <= 0 || d.K % 32) return false;
   if (((unsigned long long)d.W & 15) || ((unsigned long long)d.X & 15)) return false;
   if (d.norm ? (d.ldx % 4 || !d.norm_w) : (d.ldx % 8 != 0)) return false;
-  if (((d.epi == EPI_SWIGLU || d.epi == EPI_GLU) && d.N % 16) || ((d.epi == EPI_BIAS || d.epi == EPI_GLU) && !d.bias) || d.epi < 0 ||
-      d.epi > EPI_RELU2)
+  if (((d.epi == EPI_SWIGLU || d.epi == EPI_GLU) && d.N % 16) || ((d.epi == EPI_BIAS || d.epi == EPI_GLU || d.epi == EPI_RESIDUAL_SCALED) && !d.bias) || d.epi < 0 ||
+      d.epi > EPI_RESIDUAL_SCALED)
     return false;
   op.W = (const bf16*)d.W; op.X = d.X; op.norm_w = d.norm_w; op.bias = d.bias; op.out = d.out;
   op.ldx = d.ldx; op.ldo = d.ldo; op.M = d.M; op.N = d.N; op.K = d.K; op.epi = d.epi; op.norm = d.norm; op.eps = d.eps;

@@ -632,7 +632,7 @@ Q25_EXPORT int q25_gemm_tcgen05_bf16(const void* W, const void* X, int ldx, cons
 
 // The grouped product: x [M, K] are rows sorted by expert in tiles of 128 (M the most rows there can be),
 // W [experts, N, K] the experts' matrices, plan as the kernel says (on the device).  out [M, N]:
-// bfloat16 (epi 0) or float (epi 2).  The tiles are counted on the device, so nothing is read back.
+// bfloat16 (epi 0; 6: the square of relu) or float (epi 2).  The tiles are counted on the device, so nothing is read back.
 Q25_EXPORT int q25_gemm_tcgen05_grouped_bf16(const void* W, const void* X, int ldx, void* out, int ldo, int M, int N, int K,
                                              int experts, const int* plan, int epi, int* err, void* stream) {
   if (M <= 0 || N <= 0) return 0;
@@ -647,5 +647,6 @@ Q25_EXPORT int q25_gemm_tcgen05_grouped_bf16(const void* W, const void* X, int l
   cudaStream_t s = (cudaStream_t)stream;
   if (epi == T5_STORE) return launch_t5<T5_STORE>(mx, mw, nullptr, out, ldo, M, N, K, bn, err, s, plan, experts);
   if (epi == T5_F32) return launch_t5<T5_F32>(mx, mw, nullptr, out, ldo, M, N, K, bn, err, s, plan, experts);
+  if (epi == T5_RELU2) return launch_t5<T5_RELU2>(mx, mw, nullptr, out, ldo, M, N, K, bn, err, s, plan, experts);
   return (int)cudaErrorInvalidValue;
 }

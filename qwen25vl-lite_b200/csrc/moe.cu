@@ -69,10 +69,10 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   }
 }
 
-// The router of a mixture whose scores are a softmax over all `outputs` router rows, the last `outputs - experts` of
-// which stand for experts without matrices (a choice among them takes no row of the grouped products).  The choice looks
-// at score + correction[e]; the rows form `groups` equal runs of neighbours, a run's mark is its largest such number, and
-// only the `keep` runs with the largest marks can be chosen from (the others count as minus infinity).  The `top`
+// The router of a mixture whose scores are a softmax over all `outputs` router rows (sigmoid != 0: each row's sigmoid), the
+// last `outputs - experts` of which stand for experts without matrices (a choice among them takes no row of the grouped products).  The choice looks
+// at score + correction[e]; the rows form `groups` equal runs of neighbours, a run's mark is its largest such number
+// (mark_two != 0: the sum of its two largest), and only the `keep` runs with the largest marks can be chosen from (the others count as minus infinity).  The `top`
 // largest are chosen (ties to the lower index, among runs too); a choice weighs in with its plain score: as it is, or
 // with renorm divided by the sum of the token's chosen scores (+ 1e-20); either way times weight_scale.  counts: one per
 // expert with matrices.  One block of 8 warps per TOK tokens as above, then a warp per token.
@@ -80,7 +80,8 @@ template <typename T, int TOK>
 __global__ void __launch_bounds__(256)
 moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
                          int* __restrict__ topk_idx, float* __restrict__ topk_w, int* __restrict__ counts, int n_tokens, int hidden,
-                         int experts, int outputs, int top, int groups, int keep, int renorm, float weight_scale) {
+                         int experts, int outputs, int top, int groups, int keep, int renorm, float weight_scale,
+                         int sigmoid, int mark_two) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) float route_smem[];       // TOK rows of hidden floats, then TOK x 3 x (MOE_MAX_EXPERTS + 1) numbers
@@ -94,15 +95,16 @@ moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ rout
   float* score = zs + warp * (MOE_MAX_EXPERTS + 1);                          // logits, then scores
   float* choice = zs + (TOK + 2 * warp) * (MOE_MAX_EXPERTS + 1);             // score + correction
   float* mark = choice + (MOE_MAX_EXPERTS + 1);                              // a run's mark
-  float top_z = -INFINITY;
-  for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, score[e]);
-  top_z = warp_max(top_z);
-  float sum = 0.f;
-  for (int e = lane; e < outputs; e += 32) { const float p = expf(score[e] - top_z); score[e] = p; sum += p; }
-  sum = warp_sum(sum);
-  __syncwarp();
+  float top_z = -INFINITY, sum = 0.f;
+  if (!sigmoid) {
+    for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, score[e]);
+    top_z = warp_max(top_z);
+    for (int e = lane; e < outputs; e += 32) { const float p = expf(score[e] - top_z); score[e] = p; sum += p; }
+    sum = warp_sum(sum);
+    __syncwarp();
+  }
   for (int e = lane; e < outputs; e += 32) {
-    const float s = score[e] / sum;
+    const float s = sigmoid ? 1.0f / (1.0f + expf(-score[e])) : score[e] / sum;
     score[e] = s;
     choice[e] = s + (correction ? correction[e] : 0.f);
   }
@@ -110,9 +112,13 @@ moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ rout
   if (groups > 1) {
     const int per = outputs / groups;
     for (int g = lane; g < groups; g += 32) {
-      float best = -INFINITY;
-      for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, choice[e]);
-      mark[g] = best;
+      float best = -INFINITY, next = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float c = choice[e];
+        if (c > best) { next = best; best = c; }
+        else next = fmaxf(next, c);
+      }
+      mark[g] = mark_two && per > 1 ? best + next : best;
     }
     __syncwarp();
     // the kept runs one after the other; every lane holds the same set: bit g % 32 of word g / 32
@@ -217,16 +223,23 @@ __global__ void moe_scatter_kernel(const int* __restrict__ topk_idx, const int* 
   pair_row[pair] = r;
 }
 
-// Grouped product on the CUDA cores.  GATE_UP: rows are the tile's pairs, a = weight * h[token];
-// two chains per element (gate, up), activation in the epilogue, out = act [rows, N] in T.
-// Otherwise: rows are act rows, one chain, out = y [rows, N] in float.  W* are [experts, N, K].
-template <typename T, bool GATE_UP, int BM, int BN, int BK, int TM, int TN>
+// What a grouped product does: down; gate and up with the gated unit; up alone with the square of relu.
+#define MOE_DOWN 0
+#define MOE_GATE_UP 1
+#define MOE_UP_RELU2 2
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
+
+// Grouped product on the CUDA cores.  MOE_GATE_UP: rows are the tile's pairs, a = weight * h[token];
+// two chains per element (gate, up), activation in the epilogue, out = act [rows, N] in T.  MOE_UP_RELU2: the same rows,
+// one chain.  MOE_DOWN: rows are act rows, one chain, out = y [rows, N] in float.  W* are [experts, N, K].
+template <typename T, int MODE, int BM, int BN, int BK, int TM, int TN>
 __global__ void __launch_bounds__((BM / TM) * (BN / TN))
 moe_grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ W0, const T* __restrict__ W1, void* __restrict__ out_,
                        const int* __restrict__ plan, const int* __restrict__ row_pair, const float* __restrict__ topk_w,
                        int experts, int top, int N, int K, long long w_stride, float limit, float alpha, float shift) {
   pdl_trigger();
   pdl_wait();
+  constexpr bool GATE_UP = MODE == MOE_GATE_UP, GATHER = MODE != MOE_DOWN;
   constexpr int THREADS = (BM / TM) * (BN / TN);
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
@@ -239,7 +252,7 @@ moe_grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ W0, const 
   const int m0 = tile * BM, n0 = blockIdx.x * BN;
   for (int r = threadIdx.x; r < BM; r += THREADS) {
     const int pair = row_pair[m0 + r];
-    if (GATE_UP) {
+    if (GATHER) {
       src_row[r] = pair < 0 ? -1 : pair / top;
       src_w[r] = pair < 0 ? 0.f : (topk_w ? topk_w[pair] : 1.f);      // no weights: the rows as they are
     } else {
@@ -262,7 +275,7 @@ moe_grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ W0, const 
       const int gk = k0 + c, src = src_row[r];
       float v = 0.f;
       if (src >= 0 && gk < K) v = to_f32(A[(size_t)src * K + gk]);
-      As[c][r] = GATE_UP ? v * src_w[r] : v;
+      As[c][r] = GATHER ? v * src_w[r] : v;
     }
     for (int x = threadIdx.x; x < BN * BK; x += THREADS) {
       const int r = x / BK, c = x % BK;
@@ -304,6 +317,8 @@ moe_grouped_fma_kernel(const T* __restrict__ A, const T* __restrict__ W0, const 
         const float g = fminf(acc0[i][j], limit);
         const float u = fminf(fmaxf(acc1[i][j], -limit), limit);
         reinterpret_cast<T*>(out_)[(size_t)(m0 + r) * N + gn] = from_f32<T>(g / (1.0f + expf(-alpha * g)) * (u + shift));
+      } else if (MODE == MOE_UP_RELU2) {
+        reinterpret_cast<T*>(out_)[(size_t)(m0 + r) * N + gn] = from_f32<T>(relu2_f(acc0[i][j]));
       } else {
         reinterpret_cast<float*>(out_)[(size_t)(m0 + r) * N + gn] = acc0[i][j];
       }
@@ -344,13 +359,14 @@ __global__ void moe_gather_kernel(const bf16* __restrict__ h, const int* __restr
 // steps of 64 through a ring of STAGES stages filled by 16-byte cp.async (the rows of A and of the
 // weights alike), so that a CTA always has several stages in flight.  Every element's sum runs over
 // K in the same order whatever tile the row is in.
-template <bool GATE_UP, int BM, int WARPS_M, int STAGES>
+template <int MODE, int BM, int WARPS_M, int STAGES>
 __global__ void __launch_bounds__(128)
 moe_grouped_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W0, const bf16* __restrict__ W1, void* __restrict__ out_,
                        const int* __restrict__ plan, const int* __restrict__ row_pair, int experts, int N, int K, long long w_stride,
                        float limit, float alpha, float shift) {
   pdl_trigger();
   pdl_wait();
+  constexpr bool GATE_UP = MODE == MOE_GATE_UP;
   constexpr int BN = 64, BK = 64, P = BK * 2 + 16;            // pitch in bytes: an odd number of 16-byte chunks
   constexpr int WARPS_N = 4 / WARPS_M, WM = BM / WARPS_M, WN = BN / WARPS_N;
   constexpr int MI = WM / 16, NJ = WN / 8;
@@ -459,6 +475,10 @@ moe_grouped_mma_kernel(const bf16* __restrict__ A, const bf16* __restrict__ W0, 
           bf16* o = reinterpret_cast<bf16*>(out_) + (size_t)(m0 + r) * N + gn;
           if (gn + 1 < N && N % 2 == 0) *reinterpret_cast<unsigned*>(o) = pack_bf16(y0, y1);
           else { o[0] = __float2bfloat16_rn(y0); if (gn + 1 < N) o[1] = __float2bfloat16_rn(y1); }
+        } else if (MODE == MOE_UP_RELU2) {
+          bf16* o = reinterpret_cast<bf16*>(out_) + (size_t)(m0 + r) * N + gn;
+          if (gn + 1 < N && N % 2 == 0) *reinterpret_cast<unsigned*>(o) = pack_bf16(relu2_f(v0), relu2_f(v1));
+          else { o[0] = __float2bfloat16_rn(relu2_f(v0)); if (gn + 1 < N) o[1] = __float2bfloat16_rn(relu2_f(v1)); }
         } else {
           float* o = reinterpret_cast<float*>(out_) + (size_t)(m0 + r) * N + gn;
           o[0] = v0;
@@ -510,11 +530,12 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 // out[n, :] = sum over the token's choices, in their order, of w[pair] * (y[row of the pair, :], or the token's own
 // input h[n, :] when the pair has no row: a choice that stands for an expert without matrices), plus shared[n, :] when
-// given (an expert that every token uses, unweighted), in T.
-template <typename T>
+// given (an expert that every token uses, unweighted), in T.  With x: x[n, :] += x_scale * the sum instead (the float
+// residual stream, a scale per channel or nullptr), and out is not written.
+template <typename T, int V>
 __global__ void moe_combine_weighted_kernel(const float* __restrict__ y, const int* __restrict__ pair_row, const float* __restrict__ topk_w,
-                                            const T* __restrict__ h, const T* __restrict__ shared, T* __restrict__ out, int n_tokens,
-                                            int hidden, int top) {
+                                            const T* __restrict__ h, const T* __restrict__ shared, T* __restrict__ out, float* __restrict__ x,
+                                            const float* __restrict__ x_scale, int n_tokens, int hidden, int top) {
   pdl_trigger();
   pdl_wait();
   const int n = blockIdx.x;
@@ -525,14 +546,45 @@ __global__ void moe_combine_weighted_kernel(const float* __restrict__ y, const i
     ws[threadIdx.x] = topk_w[(size_t)n * top + threadIdx.x];
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-    float acc = 0.f;
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    const size_t at = (size_t)n * hidden + c;
+    float acc[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) acc[i] = 0.f;
     for (int k = 0; k < top; ++k) {
-      const float v = rows[k] >= 0 ? y[(size_t)rows[k] * hidden + c] : to_f32(h[(size_t)n * hidden + c]);
-      acc = fmaf(ws[k], v, acc);
+      if (rows[k] >= 0) {
+        const float* src = y + (size_t)rows[k] * hidden + c;
+        if constexpr (V == 4) {
+          const float4 v = *reinterpret_cast<const float4*>(src);
+          acc[0] = fmaf(ws[k], v.x, acc[0]); acc[1] = fmaf(ws[k], v.y, acc[1]); acc[2] = fmaf(ws[k], v.z, acc[2]); acc[3] = fmaf(ws[k], v.w, acc[3]);
+        } else {
+          acc[0] = fmaf(ws[k], src[0], acc[0]);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = fmaf(ws[k], to_f32(h[at + i]), acc[i]);
+      }
     }
-    if (shared) acc += to_f32(shared[(size_t)n * hidden + c]);
-    out[(size_t)n * hidden + c] = from_f32<T>(acc);
+    if (shared) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] += to_f32(shared[at + i]);
+    }
+    if (x) {
+      float f[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] = x_scale ? x_scale[c + i] : 1.f;
+      if constexpr (V == 4) {
+        float4 v = *reinterpret_cast<float4*>(x + at);
+        v.x = fmaf(f[0], acc[0], v.x); v.y = fmaf(f[1], acc[1], v.y); v.z = fmaf(f[2], acc[2], v.z); v.w = fmaf(f[3], acc[3], v.w);
+        *reinterpret_cast<float4*>(x + at) = v;
+      } else {
+        x[at] = fmaf(f[0], acc[0], x[at]);
+      }
+    } else if constexpr (V == 4) {
+      store4<T>(out + at, make_float4(acc[0], acc[1], acc[2], acc[3]));
+    } else {
+      out[at] = from_f32<T>(acc[0]);
+    }
   }
 }
 
@@ -588,28 +640,28 @@ Q25_EXPORT int q25_moe_sort(const int* topk_idx, const int* counts, int* cursor,
   return launch_status();
 }
 
-template <bool GATE_UP, int BM, int WARPS_M, int STAGES>
+template <int MODE, int BM, int WARPS_M, int STAGES>
 static int moe_grouped_mma_shape(const void* A, const void* W0, const void* W1, void* out, const int* plan, const int* row_pair,
                                  int tiles, int experts, int N, int K, long long w_stride, float limit, float alpha, float shift, cudaStream_t s) {
-  constexpr int SMEM = STAGES * (BM + (GATE_UP ? 128 : 64)) * (64 * 2 + 16);
-  const cudaError_t e = cudaFuncSetAttribute(moe_grouped_mma_kernel<GATE_UP, BM, WARPS_M, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+  constexpr int SMEM = STAGES * (BM + (MODE == MOE_GATE_UP ? 128 : 64)) * (64 * 2 + 16);
+  const cudaError_t e = cudaFuncSetAttribute(moe_grouped_mma_kernel<MODE, BM, WARPS_M, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
   if (e != cudaSuccess) return (int)e;
-  launch(moe_grouped_mma_kernel<GATE_UP, BM, WARPS_M, STAGES>, dim3((N + 63) / 64, tiles), dim3(128), SMEM, s, (const bf16*)A, (const bf16*)W0,
+  launch(moe_grouped_mma_kernel<MODE, BM, WARPS_M, STAGES>, dim3((N + 63) / 64, tiles), dim3(128), SMEM, s, (const bf16*)A, (const bf16*)W0,
          (const bf16*)W1, out, plan, row_pair, experts, N, K, w_stride, limit, alpha, shift);
   return launch_status();
 }
 
 // A: the rows in the sorted order, [rows, K] bfloat16.
-template <bool GATE_UP>
+template <int MODE>
 static int moe_grouped_mma(const void* A, const void* W0, const void* W1, void* out, const int* plan, const int* row_pair,
                            int n_pairs, int experts, int N, int K, long long w_stride, float limit, float alpha, float shift, int tile, void* stream) {
   const int tiles = q25_moe_max_rows(n_pairs, experts, tile) / tile;
   cudaStream_t s = (cudaStream_t)stream;
-  if (tile == 16) return moe_grouped_mma_shape<GATE_UP, 16, 1, 4>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
+  if (tile == 16) return moe_grouped_mma_shape<MODE, 16, 1, 4>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
   // two stages for the large tiles: three or four CTAs then share an SM (12 to 16 warps), which hides the fixed latencies between
   // a fragment's load and its products better than a third stage does (gate and up at 4,096 rows: 268 us with three stages)
-  if (tile == 64) return moe_grouped_mma_shape<GATE_UP, 64, 2, 2>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
-  if (tile == 128) return moe_grouped_mma_shape<GATE_UP, 128, 4, 2>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
+  if (tile == 64) return moe_grouped_mma_shape<MODE, 64, 2, 2>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
+  if (tile == 128) return moe_grouped_mma_shape<MODE, 128, 4, 2>(A, W0, W1, out, plan, row_pair, tiles, experts, N, K, w_stride, limit, alpha, shift, s);
   return (int)cudaErrorInvalidValue;
 }
 
@@ -617,20 +669,20 @@ static bool moe_mma_takes(const void* A, const void* W0, const void* W1, const v
   return K % 8 == 0 && !(((uintptr_t)A | (uintptr_t)W0 | (uintptr_t)W1 | (uintptr_t)extra) & 15);
 }
 
-template <typename T, bool GATE_UP>
+template <typename T, int MODE>
 static int moe_grouped_fma(const void* A, const void* W0, const void* W1, void* out, const int* plan, const int* row_pair,
                            const float* topk_w, int n_pairs, int experts, int top, int N, int K, long long w_stride, float limit,
                            float alpha, float shift, int tile, void* stream) {
   if (n_pairs <= 0) return 0;
   const int tiles = q25_moe_max_rows(n_pairs, experts, tile) / tile;
   if (tile == 16) {
-    launch(moe_grouped_fma_kernel<T, GATE_UP, 16, 64, 16, 1, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
+    launch(moe_grouped_fma_kernel<T, MODE, 16, 64, 16, 1, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
            (const T*)A, (const T*)W0, (const T*)W1, out, plan, row_pair, topk_w, experts, top, N, K, w_stride, limit, alpha, shift);
   } else if (tile == 64) {
-    launch(moe_grouped_fma_kernel<T, GATE_UP, 64, 64, 16, 4, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
+    launch(moe_grouped_fma_kernel<T, MODE, 64, 64, 16, 4, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
            (const T*)A, (const T*)W0, (const T*)W1, out, plan, row_pair, topk_w, experts, top, N, K, w_stride, limit, alpha, shift);
   } else if (tile == 128) {     // the rows were laid out for the tensor-core product, which then did not take the operands
-    launch(moe_grouped_fma_kernel<T, GATE_UP, 128, 64, 16, 8, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
+    launch(moe_grouped_fma_kernel<T, MODE, 128, 64, 16, 8, 4>, dim3((N + 63) / 64, tiles), dim3(256), 0, (cudaStream_t)stream,
            (const T*)A, (const T*)W0, (const T*)W1, out, plan, row_pair, topk_w, experts, top, N, K, w_stride, limit, alpha, shift);
   } else {
     return (int)cudaErrorInvalidValue;
@@ -639,14 +691,18 @@ static int moe_grouped_fma(const void* A, const void* W0, const void* W1, void* 
 }
 
 // wgu: the experts' gate and up matrices, [experts, 2 * ff, hidden]: an expert's ff gate rows, then its
-// ff up rows.  sorted: [max rows, hidden] of scratch in the activation dtype for the rows in the sorted
-// order (bfloat16: the tensor-core product reads them; nullptr or float: the product gathers by itself).
+// ff up rows (gated 0: its ff up rows alone, and the square of relu).  sorted: [max rows, hidden] of scratch in the
+// activation dtype for the rows in the sorted order (bfloat16: the tensor-core product reads them; nullptr or float:
+// the product gathers by itself).
 Q25_EXPORT int q25_moe_gate_up_f32(const void* h, const void* wgu, void* act, const int* plan, const int* row_pair,
                                    const float* topk_w, int n_pairs, int experts, int top, int ff, int hidden, float limit,
-                                   float alpha, float shift, int tile, void* sorted, void* s) {
+                                   float alpha, float shift, int tile, void* sorted, int gated, void* s) {
   const float* w = (const float*)wgu;
-  return moe_grouped_fma<float, true>(h, w, w + (size_t)ff * hidden, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden,
-                                      2LL * ff * hidden, limit, alpha, shift, tile, s);
+  if (!gated)
+    return moe_grouped_fma<float, MOE_UP_RELU2>(h, w, nullptr, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden, (long long)ff * hidden,
+                                                limit, alpha, shift, tile, s);
+  return moe_grouped_fma<float, MOE_GATE_UP>(h, w, w + (size_t)ff * hidden, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden,
+                                             2LL * ff * hidden, limit, alpha, shift, tile, s);
 }
 Q25_EXPORT int q25_moe_gather_bf16(const void* h, const int* row_pair, const float* topk_w, void* sorted, int rows, int top, int hidden,
                                    void* s) {
@@ -657,29 +713,32 @@ Q25_EXPORT int q25_moe_gather_bf16(const void* h, const int* row_pair, const flo
 }
 Q25_EXPORT int q25_moe_gate_up_bf16(const void* h, const void* wgu, void* act, const int* plan, const int* row_pair,
                                     const float* topk_w, int n_pairs, int experts, int top, int ff, int hidden, float limit,
-                                    float alpha, float shift, int tile, void* sorted, void* s) {
+                                    float alpha, float shift, int tile, void* sorted, int gated, void* s) {
   if (n_pairs <= 0) return 0;
   const bf16* w = (const bf16*)wgu;
-  const bf16* wu = w + (size_t)ff * hidden;
+  const bf16* wu = gated ? w + (size_t)ff * hidden : nullptr;
+  const long long w_stride = (gated ? 2LL : 1LL) * ff * hidden;
   if (sorted && moe_mma_takes(h, w, wu, sorted, hidden)) {
     launch(moe_gather_kernel, dim3(q25_moe_max_rows(n_pairs, experts, tile)), dim3(128), 0, (cudaStream_t)s, (const bf16*)h, row_pair, topk_w,
            (bf16*)sorted, top, hidden);
-    return moe_grouped_mma<true>(sorted, w, wu, act, plan, row_pair, n_pairs, experts, ff, hidden, 2LL * ff * hidden, limit, alpha, shift, tile, s);
+    if (!gated) return moe_grouped_mma<MOE_UP_RELU2>(sorted, w, wu, act, plan, row_pair, n_pairs, experts, ff, hidden, w_stride, limit, alpha, shift, tile, s);
+    return moe_grouped_mma<MOE_GATE_UP>(sorted, w, wu, act, plan, row_pair, n_pairs, experts, ff, hidden, w_stride, limit, alpha, shift, tile, s);
   }
-  return moe_grouped_fma<bf16, true>(h, w, wu, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden, 2LL * ff * hidden, limit, alpha, shift,
-                                     tile, s);
+  if (!gated)
+    return moe_grouped_fma<bf16, MOE_UP_RELU2>(h, w, wu, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden, w_stride, limit, alpha, shift, tile, s);
+  return moe_grouped_fma<bf16, MOE_GATE_UP>(h, w, wu, act, plan, row_pair, topk_w, n_pairs, experts, top, ff, hidden, w_stride, limit, alpha, shift, tile, s);
 }
 Q25_EXPORT int q25_moe_down_f32(const void* act, const void* wd, void* y, const int* plan, const int* row_pair, int n_pairs,
                                 int experts, int top, int hidden, int ff, int tile, void* s) {
-  return moe_grouped_fma<float, false>(act, wd, nullptr, y, plan, row_pair, nullptr, n_pairs, experts, top, hidden, ff, (long long)hidden * ff,
+  return moe_grouped_fma<float, MOE_DOWN>(act, wd, nullptr, y, plan, row_pair, nullptr, n_pairs, experts, top, hidden, ff, (long long)hidden * ff,
                                        0.f, 0.f, 0.f, tile, s);
 }
 Q25_EXPORT int q25_moe_down_bf16(const void* act, const void* wd, void* y, const int* plan, const int* row_pair, int n_pairs,
                                  int experts, int top, int hidden, int ff, int tile, void* s) {
   if (n_pairs <= 0) return 0;
   if (moe_mma_takes(act, wd, nullptr, nullptr, ff))
-    return moe_grouped_mma<false>(act, wd, nullptr, y, plan, row_pair, n_pairs, experts, hidden, ff, (long long)hidden * ff, 0.f, 0.f, 0.f, tile, s);
-  return moe_grouped_fma<bf16, false>(act, wd, nullptr, y, plan, row_pair, nullptr, n_pairs, experts, top, hidden, ff, (long long)hidden * ff,
+    return moe_grouped_mma<MOE_DOWN>(act, wd, nullptr, y, plan, row_pair, n_pairs, experts, hidden, ff, (long long)hidden * ff, 0.f, 0.f, 0.f, tile, s);
+  return moe_grouped_fma<bf16, MOE_DOWN>(act, wd, nullptr, y, plan, row_pair, nullptr, n_pairs, experts, top, hidden, ff, (long long)hidden * ff,
                                       0.f, 0.f, 0.f, tile, s);
 }
 
@@ -701,7 +760,7 @@ Q25_EXPORT int q25_moe_combine_bf16(const float* y, const int* pr, const float* 
 template <typename T, int TOK>
 static int moe_route_softmax_shape(const void* h, const float* router, const float* correction, int* topk_idx, float* topk_w, int* counts,
                                    int n_tokens, int hidden, int experts, int outputs, int top, int groups, int keep, int renorm,
-                                   float weight_scale, cudaStream_t stream) {
+                                   float weight_scale, int sigmoid, int mark_two, cudaStream_t stream) {
   const size_t smem = (size_t)TOK * (((hidden + 3) & ~3) + 3 * (MOE_MAX_EXPERTS + 1)) * sizeof(float);
   if (smem > 200 * 1024) return -1;
   if (smem > 48 * 1024) {
@@ -709,45 +768,50 @@ static int moe_route_softmax_shape(const void* h, const float* router, const flo
     if (e != cudaSuccess) return (int)e;
   }
   launch(moe_route_softmax_kernel<T, TOK>, dim3((n_tokens + TOK - 1) / TOK), dim3(256), smem, stream, (const T*)h, router, correction,
-         topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale);
+         topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale, sigmoid, mark_two);
   return launch_status();
 }
 
 template <typename T>
 static int moe_route_softmax(const void* h, const float* router, const float* correction, int* topk_idx, float* topk_w, int* counts,
                              int n_tokens, int hidden, int experts, int outputs, int top, int groups, int keep, int renorm,
-                             float weight_scale, void* stream) {
+                             float weight_scale, int sigmoid, int mark_two, void* stream) {
   if (n_tokens <= 0) return 0;
   if (experts <= 0 || outputs < experts || outputs > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP || groups < 1 || outputs % groups ||
       keep < 1 || keep > groups || top > keep * (outputs / groups))
     return (int)cudaErrorInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   int rc = -1;
-  if (n_tokens >= 512) rc = moe_route_softmax_shape<T, 4>(h, router, correction, topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale, s);
-  if (rc == -1) rc = moe_route_softmax_shape<T, 1>(h, router, correction, topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale, s);
+  if (n_tokens >= 512) rc = moe_route_softmax_shape<T, 4>(h, router, correction, topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale, sigmoid, mark_two, s);
+  if (rc == -1) rc = moe_route_softmax_shape<T, 1>(h, router, correction, topk_idx, topk_w, counts, n_tokens, hidden, experts, outputs, top, groups, keep, renorm, weight_scale, sigmoid, mark_two, s);
   return rc == -1 ? (int)cudaErrorInvalidValue : rc;
 }
 Q25_EXPORT int q25_moe_route_softmax_f32(const void* h, const float* r, const float* corr, int* ti, float* tw, int* counts, int n, int hidden,
-                                         int experts, int outputs, int top, int groups, int keep, int renorm, float wscale, void* s) {
-  return moe_route_softmax<float>(h, r, corr, ti, tw, counts, n, hidden, experts, outputs, top, groups, keep, renorm, wscale, s);
+                                         int experts, int outputs, int top, int groups, int keep, int renorm, float wscale, int sig, int two, void* s) {
+  return moe_route_softmax<float>(h, r, corr, ti, tw, counts, n, hidden, experts, outputs, top, groups, keep, renorm, wscale, sig, two, s);
 }
 Q25_EXPORT int q25_moe_route_softmax_bf16(const void* h, const float* r, const float* corr, int* ti, float* tw, int* counts, int n, int hidden,
-                                          int experts, int outputs, int top, int groups, int keep, int renorm, float wscale, void* s) {
-  return moe_route_softmax<bf16>(h, r, corr, ti, tw, counts, n, hidden, experts, outputs, top, groups, keep, renorm, wscale, s);
+                                          int experts, int outputs, int top, int groups, int keep, int renorm, float wscale, int sig, int two, void* s) {
+  return moe_route_softmax<bf16>(h, r, corr, ti, tw, counts, n, hidden, experts, outputs, top, groups, keep, renorm, wscale, sig, two, s);
 }
 
 template <typename T>
-static int moe_combine_weighted(const float* y, const int* pair_row, const float* topk_w, const void* h, const void* shared, void* out,
-                                int n_tokens, int hidden, int top, void* stream) {
+static int moe_combine_weighted(const float* y, const int* pair_row, const float* topk_w, const void* h, const void* shared, void* out, float* x,
+                                const float* x_scale, int n_tokens, int hidden, int top, void* stream) {
   if (n_tokens <= 0) return 0;
-  if (top > MOE_MAX_TOP) return (int)cudaErrorInvalidValue;
-  launch(moe_combine_weighted_kernel<T>, dim3(n_tokens), dim3(hidden >= 2048 ? 256 : 128), 0, (cudaStream_t)stream, y, pair_row, topk_w,
-         (const T*)h, (const T*)shared, (T*)out, n_tokens, hidden, top);
+  if (top > MOE_MAX_TOP || (!x && !out)) return (int)cudaErrorInvalidValue;
+  const size_t row = 4 * sizeof(T);
+  const bool four = hidden % 4 == 0 && !(((uintptr_t)y | (uintptr_t)x) & 15) && !((uintptr_t)h % row) && !((uintptr_t)shared % row) && !((uintptr_t)out % row);
+  const int threads = hidden >= 2048 ? 256 : 128;
+  if (four) launch(moe_combine_weighted_kernel<T, 4>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream, y, pair_row, topk_w,
+                   (const T*)h, (const T*)shared, (T*)out, x, x_scale, n_tokens, hidden, top);
+  else launch(moe_combine_weighted_kernel<T, 1>, dim3(n_tokens), dim3(threads), 0, (cudaStream_t)stream, y, pair_row, topk_w,
+              (const T*)h, (const T*)shared, (T*)out, x, x_scale, n_tokens, hidden, top);
   return launch_status();
 }
-Q25_EXPORT int q25_moe_combine_weighted_f32(const float* y, const int* pr, const float* tw, const void* h, const void* sh, void* out, int n, int hd, int top, void* s) {
-  return moe_combine_weighted<float>(y, pr, tw, h, sh, out, n, hd, top, s);
+Q25_EXPORT int q25_moe_combine_weighted_f32(const float* y, const int* pr, const float* tw, const void* h, const void* sh, void* out, float* x, const float* xs, int n, int hd, int top, void* s) {
+  return moe_combine_weighted<float>(y, pr, tw, h, sh, out, x, xs, n, hd, top, s);
 }
-Q25_EXPORT int q25_moe_combine_weighted_bf16(const float* y, const int* pr, const float* tw, const void* h, const void* sh, void* out, int n, int hd, int top, void* s) {
-  return moe_combine_weighted<bf16>(y, pr, tw, h, sh, out, n, hd, top, s);
+Q25_EXPORT int q25_moe_combine_weighted_bf16(const float* y, const int* pr, const float* tw, const void* h, const void* sh, void* out, float* x, const float* xs, int n, int hd, int top, void* s) {
+  return moe_combine_weighted<bf16>(y, pr, tw, h, sh, out, x, xs, n, hd, top, s);
 }

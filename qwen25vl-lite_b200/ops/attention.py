@@ -318,20 +318,21 @@ def _plan_biased(host, group: int, window: int, keep_first: int) -> Dict[str, np
 
 
 def attend_biased(ctx, plan, qkv, kv, nq: int, nkv: int, dk: int, dv: int, window, keep_first: int, scale: float,
-                  r1, r2, sink=None, v_row: int = 0, softcap: float = 0.0, dist_bias=None, gate_off: int = -1) -> torch.Tensor:
+                  r1, r2, sink=None, v_row: int = 0, softcap: float = 0.0, dist_bias=None, gate_off: int = -1, out=None) -> torch.Tensor:
     """qkv: [N, nq*dk (+ ...)] rows that begin with the queries, this step's keys and values already in
     the pages.  ``sink``: float32 [nq] joining each head's denominator; ``v_row``: the values lie inside
     the key rows, that many channels apart; ``softcap`` c > 0: scaled scores become c * tanh(score / c);
     ``dist_bias``: float32 [rows, nq] added to the score by distance (the last row for every distance beyond);
     ``gate_off`` >= 0: the rows of ``qkv`` hold nq * dv gate channels there, whose sigmoid multiplies the result.
-    Returns [N, nq * dv]."""
-    out = torch.empty((qkv.shape[0], nq * dv), dtype=qkv.dtype, device=qkv.device)
+    Returns [N, nq * dv]; ``out``: rows (possibly strided) that take the result."""
+    if out is None:
+        out = torch.empty((qkv.shape[0], nq * dv), dtype=qkv.dtype, device=qkv.device)
     window, keep_first = int(window or 0), int(keep_first or 0)
     if kernels.biased_attention_mma_supports(qkv.dtype, dk, dv) and (v_row or dv) % 8 == 0 and (gate_off < 0 or gate_off % 2 == 0):
         items, tiles = plan.get("decode_items"), _pairs(plan.get("tiles64"))
         tiles128 = _pairs(plan.get("tiles128"), 3)
         if (tiles128 is not None and tcgen05_runs(dk, dv, nq // nkv, window, keep_first, r1, v_row, softcap)
-                and (gate_off < 0 or gate_off % 8 == 0) and kernels.attention_tcgen05_supports(qkv.dtype, dk, kv.page_size, qkv)):
+                and (gate_off < 0 or gate_off % 8 == 0) and out.is_contiguous() and kernels.attention_tcgen05_supports(qkv.dtype, dk, kv.page_size, qkv)):
             # the runs on the tcgen05 kernel (whose rows take a table by distance in their scores, and a sink and a gate
             # where they become results); the single tokens stay with the kernel below
             merge128 = _pairs(plan.get("merge128"), 4)
@@ -355,4 +356,31 @@ def attend_biased(ctx, plan, qkv, kv, nq: int, nkv: int, dk: int, dv: int, windo
     kernels.biased_attention_generic(qkv, out, kv.k_pages, kv.v_pages, kv.block_table, ctx.token_seq, ctx.cu_q,
                                      ctx.q_start_pos, nq, nkv, dk, dv, kv.page_size, int(window or 0), int(keep_first or 0),
                                      scale, r1, r2, sink, v_row, softcap, dist_bias, gate_off)
+    return out
+
+
+# ---- differential attention: two maps of every head over one value -------------------------------------------
+
+
+def attend_differential(ctx, plan, qkv, gate, kv, heads: int, kv_heads: int, dk: int, dv: int, window, scale: float, lam: float, gain: float,
+                        eps: float) -> torch.Tensor:
+    """qkv: rows that begin with the queries, ordered by (kv head, map, head of the group), ``dk`` channels each; the step's
+    keys (rows of both maps, 2 * dk channels) and values already in the pages; ``gate``: rows of heads * dv channels.
+    Returns [N, heads * dv]: per head the first map's result minus ``lam`` times the second's, divided by its root mean
+    square, times ``gain`` and the gate's sigmoid.  ``plan``: ``plan_biased`` for groups of 2 * heads / kv_heads rows (a
+    token's heads on both maps); a tile of 64 such rows is 32 (token, head) pairs."""
+    out = torch.empty((qkv.shape[0], heads * dv), dtype=qkv.dtype, device=qkv.device)
+    window = int(window or 0)
+    if kernels.differential_attention_mma_supports(qkv, gate, dk, dv):
+        items, tiles = plan.get("decode_items"), _pairs(plan.get("tiles64"))
+        splits, scratch = 1, None
+        if items is not None:
+            splits = decode_splits(items.shape[0], kv_heads, min(ctx.max_kv_len, window) if window else ctx.max_kv_len)
+            if splits > 1:
+                scratch = _scratch_floats(items.shape[0] * 2 * heads * splits * (dv + 2), qkv.device, "biased")
+        kernels.differential_attention_mma(qkv, gate, out, kv.k_pages, kv.v_pages, kv.block_table, ctx.cu_q, ctx.q_start_pos, tiles, items,
+                                           heads, kv_heads, dk, dv, kv.page_size, window, scale, lam, gain, eps, splits, scratch)
+    else:
+        kernels.differential_attention_generic(qkv, gate, out, kv.k_pages, kv.v_pages, kv.block_table, ctx.token_seq, ctx.cu_q, ctx.q_start_pos,
+                                               heads, kv_heads, dk, dv, kv.page_size, window, scale, lam, gain, eps)
     return out

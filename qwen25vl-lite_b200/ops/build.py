@@ -34,7 +34,8 @@ NVCC_FLAGS = [
 # of attention with a distance bias, kept first tokens or a sink, and of the routed feed-forward; "rotary" a
 # rotation of part of a head in either pairing, "latent" the compressed cache row of latent attention,
 # "retention" the decayed linear attention, "memory" the matrix memories whose gates depend on the token, "hyper" a
-# residual stream of several rows per token, "state_space" the tensor-core runs of the state space.  A library is compiled when a model first asks for one of its kernels, so a run compiles only what
+# residual stream of several rows per token, "state_space" the tensor-core runs of the state space, "differential" attention whose heads subtract one map from another,
+# "delta" the gated delta rule.  A library is compiled when a model first asks for one of its kernels, so a run compiles only what
 # its model and dtype need.
 LIBRARIES: Dict[str, List[str]] = {
     "core": ["elementwise.cu", "rope_cache.cu", "attention_generic.cu", "gemm_f32.cu", "sampling.cu"],
@@ -50,6 +51,8 @@ LIBRARIES: Dict[str, List[str]] = {
     "memory": ["gated_memory.cu"],
     "hyper": ["hyper.cu"],
     "state_space": ["state_space.cu"],
+    "differential": ["attention_differential.cu"],
+    "delta": ["delta_rule.cu"],
 }
 
 

@@ -30,19 +30,19 @@ _SIGNATURES = {
     "q25_add_norm_groups": [_P, _P, _P, _F, _I, _P, _F, _I, _P, _P, _I, _I, _P],
     "q25_glu_clamped": [_P, _P, _I, _I, _F, _F, _F, _I, _P],
     "q25_rglru_scan": [_P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _P, _I, _I, _P],
-    "q25_biased_attention_generic": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _I, _F, _P, _I, _I, _P],
-    "q25_biased_attention_qk_norm_store": [_P, _I, _P, _P, _F, _I, _P, _I, _I, _P, _F, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "q25_biased_attention_generic": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _I, _F, _P, _I, _I, _I, _P],
+    "q25_biased_attention_qk_norm_store": [_P, _I, _P, _P, _F, _I, _P, _I, _I, _P, _F, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "q25_add_dyt": [_P, _P, _P, _P, _F, _P, _P, _I, _I, _P],
     "q25_rotary_apply": [_P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "q25_latent_store": [_P, _I, _I, _I, _P, _F, _P, _I, _I, _P, _P, _I, _P, _I, _I, _P, _P, _P],
     "q25_retention": [_P, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _F, _P, _I, _P, _I, _P, _I, _I, _P],
     "q25_kv_store_mix": [_P, _I, _P, _I, _F, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "q25_moe_route": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "q25_moe_gate_up": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P, _P],
+    "q25_moe_gate_up": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P, _I, _P],
     "q25_moe_down": [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "q25_moe_combine": [_P, _P, _P, _P, _P, _I, _I, _I, _P],
-    "q25_moe_route_softmax": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P],
-    "q25_moe_combine_weighted": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _P],
+    "q25_moe_route_softmax": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P],
+    "q25_moe_combine_weighted": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _P],
     "q25_activation": [_P, _P, _LL, _I, _P],
     "q25_add_layernorm": [_P, _P, _P, _P, _P, _F, _P, _P, _F, _P, _P, _I, _I, _P],
     "q25_branch_mean_norm": [_P, _P, _I, _P, _I, _I, _F, _P],
@@ -57,7 +57,9 @@ _SIGNATURES = {
     "q25_latent_gate": [_P, _P, _I, _I, _I, _P],
     "q25_hyper_norm": [_P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P],
     "q25_hyper_embed": [_P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _LL, _LL, _LL, _I, _P],
-    "q25_memory_output": [_P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P],
+    "q25_memory_output": [_P, _P, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
+    "q25_differential_attention_generic": [_P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P],
+    "q25_delta_walk": [_P, _I, _I, _I, _P, _P, _P, _P, _LL, _P, _P, _P, _I, _P, _P, _I, _P, _F, _P, _I, _I, _I, _I, _I, _F, _F, _P],
 }
 _UNTYPED = {
     "q25_attention_decode_bf16": [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
@@ -96,7 +98,7 @@ _SYMBOL_LIBRARY = (("q25_gemm_chain", "chain"), ("q25_attention_decode", "bf16")
                    ("q25_gemm_tcgen05", "tcgen05"), ("q25_rope_angles", "bf16"), ("q25_rglru", "recurrent"),
                    ("q25_biased_attention", "biased"), ("q25_kv_store_mix", "biased"), ("q25_moe", "routed"),
                    ("q25_rotary", "rotary"), ("q25_latent", "latent"), ("q25_retention", "retention"), ("q25_memory", "memory"),
-                   ("q25_hyper", "hyper"), ("q25_state_space", "state_space"))
+                   ("q25_hyper", "hyper"), ("q25_state_space", "state_space"), ("q25_differential", "differential"), ("q25_delta", "delta"))
 
 
 def _library_of(symbol: str) -> str:
@@ -431,7 +433,7 @@ def gemm_f32(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out
         _stream()), "gemm_f32")
 
 
-SKINNY_STORE, SKINNY_BIAS, SKINNY_F32, SKINNY_SWIGLU, SKINNY_RESIDUAL, SKINNY_GLU, SKINNY_RELU2 = 0, 1, 2, 3, 4, 5, 6
+SKINNY_STORE, SKINNY_BIAS, SKINNY_F32, SKINNY_SWIGLU, SKINNY_RESIDUAL, SKINNY_GLU, SKINNY_RELU2, SKINNY_RESIDUAL_SCALED = 0, 1, 2, 3, 4, 5, 6, 7
 # Rows the weight-streaming kernel takes: the 8 batch columns of one m16n8k16 MMA.  A variant with two
 # column tiles ran 9 to 16 rows; measured against the library path on B200 it lost at every size (a
 # decode step of 9 / 12 / 16 requests at the 3B sizes 2.64 / 2.66 / 2.65 ms against 2.43 / 2.55 / 2.59,
@@ -459,8 +461,8 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
     ``epilogue``: SKINNY_STORE, SKINNY_BIAS (float32 bias), SKINNY_F32 (float32 out),
     SKINNY_SWIGLU (w rows are groups of 8 gate + 8 up features; out has half as many columns),
     SKINNY_GLU (the same layout with the clamped gated unit; ``bias`` then holds its two constants,
-    float32 [limit, alpha]), SKINNY_RELU2 (the square of relu of the product) or SKINNY_RESIDUAL (out is float32 and
-    the product is added into it).  Runs as an operation
+    float32 [limit, alpha]), SKINNY_RELU2 (the square of relu of the product), SKINNY_RESIDUAL (out is float32 and
+    the product is added into it) or SKINNY_RESIDUAL_SCALED (the same, times ``bias``: a float32 scale per column).  Runs as an operation
     of the chain kernel (``csrc/gemm_chain.cu``): at once and alone, or, between ``chain_begin``
     and ``chain_end``, together with the products around it."""
     m, k = x.shape
@@ -473,7 +475,7 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], 
 
 def _skinny_out(out: torch.Tensor, m: int, n: int, epilogue: int, what: str) -> None:
     cols = n // 2 if epilogue in (SKINNY_SWIGLU, SKINNY_GLU) else n
-    want = torch.float32 if epilogue in (SKINNY_F32, SKINNY_RESIDUAL) else torch.bfloat16
+    want = torch.float32 if epilogue in (SKINNY_F32, SKINNY_RESIDUAL, SKINNY_RESIDUAL_SCALED) else torch.bfloat16
     if out.shape != (m, cols) or out.dtype != want or out.stride(1) != 1:
         raise KernelError(f"{what}: output must be [{m}, {cols}] {want}")
     if epilogue in (SKINNY_SWIGLU, SKINNY_GLU) and n % 16:
@@ -690,7 +692,8 @@ def embed_position_norm(table: torch.Tensor, pos_table: torch.Tensor, ids: torch
 def add_norm_groups(x: torch.Tensor, delta: Optional[torch.Tensor], delta_weight: Optional[torch.Tensor], delta_eps: float,
                     delta_groups: int, weight: Optional[torch.Tensor], eps: float, groups: int,
                     out: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None, dtype: Optional[torch.dtype] = None) -> None:
-    """x += d with d = delta, or norm_in_groups(delta) * delta_weight when a weight is given; then
+    """x += d with d = delta, or norm_in_groups(delta) * delta_weight when a weight is given (``delta_groups`` 0: delta *
+    delta_weight, no norm); then
     out = norm_in_groups(x) * weight (out None: only the addition; weight None: out = x as it is, in out's dtype).
     ``rows`` as for ``add_rmsnorm``."""
     hidden = x.shape[-1]
@@ -814,7 +817,7 @@ def biased_attention_generic(qkv: torch.Tensor, out: torch.Tensor, k_pages: torc
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), cu_q.data_ptr(), q_start_pos.data_ptr(), qkv.shape[0], nq, nkv, dk, dv,
         page_size, int(window or 0), int(keep_first or 0), float(scale), _ptr(r1), _ptr(r2), _ptr(sink), int(v_row or 0), float(softcap or 0.0),
-        _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], int(gate_off), _stream()), "biased_attention_generic")
+        _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], int(gate_off), out.stride(0), _stream()), "biased_attention_generic")
 
 
 def _check_dist_bias(dist_bias: Optional[torch.Tensor], nq: int) -> None:
@@ -855,12 +858,12 @@ def biased_attention_mma(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Te
     if not biased_attention_mma_supports(qkv.dtype, dk, dv) or (n_items and nq // nkv > 16):
         raise KernelError(f"biased_attention_mma: unsupported sizes {dk}/{dv} or more than 16 heads per kv head for single tokens")
     _check(_fn("q25_biased_attention_mma_bf16",
-               [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _F, _P, _I, _I, _P])(
+               [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _F, _P, _I, _I, _I, _P])(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], cu_q.data_ptr(), q_start_pos.data_ptr(), _ptr(tiles), n_tiles, _ptr(items), n_items, nq, nkv, dk, dv,
         page_size, int(window or 0), int(keep_first or 0), float(scale), _ptr(r1), _ptr(r2), _ptr(sink), int(v_row or 0), int(n_splits),
         part_o, part_ml, float(softcap or 0.0), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], int(gate_off),
-        _stream()), "biased_attention_mma")
+        out.stride(0), _stream()), "biased_attention_mma")
     count_replayed((1 if n_tiles and n_items else 0) + (1 if n_items and n_splits > 1 else 0))
 
 
@@ -1024,20 +1027,21 @@ def moe_sort(topk_idx: torch.Tensor, counts: torch.Tensor, cursor: torch.Tensor,
 
 def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, plan: torch.Tensor, row_pair: torch.Tensor,
                 topk_w: Optional[torch.Tensor], top: int, limit: float, alpha: float, tile: int, shift: float = 1.0,
-                n_pairs: Optional[int] = None) -> None:
+                n_pairs: Optional[int] = None, gated: bool = True) -> None:
     """act[row] = glu(expert of the row's tile applied to weight * h[token of the row]) for the sorted
     rows.  ``w_gate_up``: [experts, 2 * ff, hidden], an expert's gate rows and then its up rows.  Without
     ``topk_w`` the rows go in as they are (``n_pairs`` then says how many pairs the step has); ``shift`` as for
-    ``glu_clamped``."""
+    ``glu_clamped``.  ``gated`` False: ``w_gate_up`` is [experts, ff, hidden], up rows alone, and act their square of relu."""
     n_pairs = topk_w.numel() if n_pairs is None else int(n_pairs)
     experts, ff2, hidden = w_gate_up.shape
+    ff = ff2 // 2 if gated else ff2
     _dev(h, act.dtype, "moe_gate_up input")
     _dev(w_gate_up, h.dtype, "moe_gate_up weights"); _dev(act, h.dtype, "moe_gate_up act")
     # bfloat16: the rows are first written out in the sorted order, weighted, for the tensor-core product
     sorted_rows = torch.empty((act.shape[0], hidden), dtype=h.dtype, device=h.device) if h.dtype == torch.bfloat16 else None
     _check(_typed("q25_moe_gate_up", h.dtype)(h.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), plan.data_ptr(),
-                                              row_pair.data_ptr(), _ptr(topk_w), n_pairs, experts, int(top), ff2 // 2, hidden,
-                                              float(limit), float(alpha), float(shift), int(tile), _ptr(sorted_rows), _stream()), "moe_gate_up")
+                                              row_pair.data_ptr(), _ptr(topk_w), n_pairs, experts, int(top), ff, hidden,
+                                              float(limit), float(alpha), float(shift), int(tile), _ptr(sorted_rows), int(bool(gated)), _stream()), "moe_gate_up")
     if sorted_rows is not None:
         count_replayed(1)
 
@@ -1058,18 +1062,21 @@ def gemm_tcgen05_grouped_supports(x_dtype: torch.dtype, hidden: int, ff: int) ->
     return x_dtype == torch.bfloat16 and hidden % 8 == 0 and ff % 8 == 0
 
 
-def gemm_tcgen05_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.Tensor) -> None:
+def gemm_tcgen05_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: torch.Tensor, epilogue: int = SKINNY_STORE) -> None:
     """out[row] = x[row] . w[expert of the row's tile]^T on the tcgen05 tensor cores: ``x`` [rows, K] sorted by
     expert in tiles of ``GROUPED_TILE`` rows (rows: the most there can be), ``w`` [experts, N, K], ``plan`` as
-    ``moe_sort`` leaves it on the device; ``out`` [rows, N] bfloat16 or float32."""
+    ``moe_sort`` leaves it on the device; ``out`` [rows, N] bfloat16 or float32.  ``epilogue`` SKINNY_RELU2: the square of relu of
+    the product (bfloat16)."""
     rows, k = x.shape
     experts, n, k2 = w.shape
+    if epilogue not in (SKINNY_STORE, SKINNY_RELU2) or (epilogue == SKINNY_RELU2 and out.dtype != torch.bfloat16):
+        raise KernelError(f"gemm_tcgen05_grouped: unsupported epilogue {epilogue} into {out.dtype}")
     if (k2 != k or rows % GROUPED_TILE or out.shape != (rows, n) or out.dtype not in (torch.bfloat16, torch.float32)
             or not gemm_tcgen05_supports(x, w.view(experts * n, k))):
         raise KernelError(f"gemm_tcgen05_grouped: unsupported operands {tuple(x.shape)} x {tuple(w.shape)} -> {tuple(out.shape)}")
     _check(_fn("q25_gemm_tcgen05_grouped_bf16", [_P, _P, _I, _P, _I, _I, _I, _I, _I, _P, _I, _P, _P])(
         w.data_ptr(), x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), rows, n, k, experts, plan.data_ptr(),
-        SKINNY_F32 if out.dtype == torch.float32 else SKINNY_STORE, error_flag(x.device).data_ptr(), _stream()), "gemm_tcgen05_grouped")
+        SKINNY_F32 if out.dtype == torch.float32 else epilogue, error_flag(x.device).data_ptr(), _stream()), "gemm_tcgen05_grouped")
 
 
 def moe_down(act: torch.Tensor, w_down: torch.Tensor, y: torch.Tensor, plan: torch.Tensor, row_pair: torch.Tensor, n_pairs: int,
@@ -1091,10 +1098,11 @@ def moe_combine(y: torch.Tensor, pair_row: torch.Tensor, sg: Optional[torch.Tens
 
 def moe_route_softmax(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], experts: int, top: int, groups: int,
                       keep: int, topk_idx: torch.Tensor, topk_w: torch.Tensor, counts: torch.Tensor, renorm: bool = False,
-                      weight_scale: float = 1.0) -> None:
+                      weight_scale: float = 1.0, scores: str = "softmax", mark: str = "largest") -> None:
     """Router logits in float32 over all rows of ``router`` (the last ``rows - experts`` stand for experts without
-    matrices), scores = softmax; the ``top`` largest of score + correction inside the ``keep`` best of ``groups``
-    equal runs of rows are chosen and weigh in with their plain scores (``renorm``: divided by their sum + 1e-20), times
+    matrices), scores = softmax, or with ``scores`` "sigmoid" each row's own sigmoid; the ``top`` largest of score + correction inside the ``keep`` best of ``groups``
+    equal runs of rows (the best by their largest such number, or with ``mark`` "two_largest" by the sum of their two largest)
+    are chosen and weigh in with their plain scores (``renorm``: divided by their sum + 1e-20), times
     ``weight_scale``; ``counts`` (one per expert with matrices) takes how many tokens chose each."""
     n, hidden = h.shape
     outputs = router.shape[0]
@@ -1104,21 +1112,32 @@ def moe_route_softmax(h: torch.Tensor, router: torch.Tensor, correction: Optiona
         _dev(correction, torch.float32, "moe_route_softmax correction")
     _check(_typed("q25_moe_route_softmax", h.dtype)(h.data_ptr(), router.data_ptr(), _ptr(correction), topk_idx.data_ptr(), topk_w.data_ptr(),
                                                     counts.data_ptr(), n, hidden, int(experts), outputs, int(top), int(groups), int(keep),
-                                                    int(bool(renorm)), float(weight_scale), _stream()), "moe_route_softmax")
+                                                    int(bool(renorm)), float(weight_scale), int(scores == "sigmoid"), int(mark == "two_largest"),
+                                                    _stream()), "moe_route_softmax")
 
 
-def moe_combine_weighted(y: torch.Tensor, pair_row: torch.Tensor, topk_w: torch.Tensor, h: torch.Tensor, out: torch.Tensor, top: int,
-                         shared: Optional[torch.Tensor] = None) -> None:
+def moe_combine_weighted(y: torch.Tensor, pair_row: torch.Tensor, topk_w: torch.Tensor, h: torch.Tensor, out: Optional[torch.Tensor], top: int,
+                         shared: Optional[torch.Tensor] = None, residual: Optional[torch.Tensor] = None,
+                         residual_scale: Optional[torch.Tensor] = None) -> None:
     """out[n] = sum over the token's choices of weight * (the row of ``y`` the choice has, or h[n] itself when it has none),
-    plus ``shared[n]`` when given (the result of an expert that every token uses)."""
-    n, hidden = out.shape
-    _dev(y, torch.float32, "moe_combine_weighted rows"); _dev(h, out.dtype, "moe_combine_weighted input")
+    plus ``shared[n]`` when given (the result of an expert that every token uses).  With ``residual`` (float32) the sum,
+    times ``residual_scale`` (float32 per channel) when given, is added there instead and ``out`` is None."""
+    n, hidden = h.shape
+    _dev(y, torch.float32, "moe_combine_weighted rows"); _dev(h, h.dtype, "moe_combine_weighted input")
+    if residual is not None:
+        _dev(residual, torch.float32, "moe_combine_weighted residual")
+        if residual_scale is not None:
+            _dev(residual_scale, torch.float32, "moe_combine_weighted residual scale")
+        if residual.shape != h.shape or (residual_scale is not None and residual_scale.numel() != hidden):
+            raise KernelError("moe_combine_weighted: the residual has the input's shape, its scale a number per channel")
+    else:
+        _dev(out, h.dtype, "moe_combine_weighted out")
     if shared is not None:
-        _dev(shared, out.dtype, "moe_combine_weighted shared")
-        if shared.shape != out.shape or not shared.is_contiguous():
+        _dev(shared, h.dtype, "moe_combine_weighted shared")
+        if shared.shape != h.shape or not shared.is_contiguous():
             raise KernelError("moe_combine_weighted: the shared expert's result has the output's shape")
-    _check(_typed("q25_moe_combine_weighted", out.dtype)(y.data_ptr(), pair_row.data_ptr(), topk_w.data_ptr(), h.data_ptr(), _ptr(shared),
-                                                         out.data_ptr(), n, hidden, int(top), _stream()), "moe_combine_weighted")
+    _check(_typed("q25_moe_combine_weighted", h.dtype)(y.data_ptr(), pair_row.data_ptr(), topk_w.data_ptr(), h.data_ptr(), _ptr(shared),
+                                                       _ptr(out), _ptr(residual), _ptr(residual_scale), n, hidden, int(top), _stream()), "moe_combine_weighted")
 
 
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1}
@@ -1196,12 +1215,13 @@ def qk_norm_store(qk: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: 
                   angles: Optional[torch.Tensor], layout: str, k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor],
                   kv_slot: Optional[torch.Tensor], nq: int, nkv: int, dk: int, page_size: int, keys_as_values: bool,
                   unit_norm: bool = False, positions: Optional[torch.Tensor] = None, temp_coef: float = 0.0, temp_every: int = 0,
-                  dv: int = 0) -> None:
+                  dv: int = 0, pack: int = 1) -> None:
     """Rows [nq query heads | nkv key heads] of ``dk`` channels: every head divided by its root mean square and
     multiplied by its weight (dk numbers, shared by the heads; without weights only divided when ``unit_norm``, else
     left alone), then turned by ``angles``; queries are written back, keys go to the pages at ``kv_slot``; with
     ``keys_as_values`` the keys as they came go to the value pages, with ``dv`` > 0 the nkv value heads of ``dv``
-    channels that follow the keys in a row.  ``temp_every`` > 0: the queries of a token at position p (``positions``,
+    channels that follow the keys in a row.  ``pack``: that many neighbouring key heads lie side by side in one wide key row
+    of the cache, which has nkv / pack key/value heads.  ``temp_every`` > 0: the queries of a token at position p (``positions``,
     int32 [N]) are multiplied by ``1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)``."""
     half = 0 if angles is None else angles.shape[1]
     if qk.stride(1) != 1:
@@ -1211,7 +1231,7 @@ def qk_norm_store(qk: torch.Tensor, q_weight: Optional[torch.Tensor], k_weight: 
     _check(_typed("q25_biased_attention_qk_norm_store", qk.dtype)(
         qk.data_ptr(), qk.stride(0), _ptr(q_weight), _ptr(k_weight), float(eps), int(bool(unit_norm)), _ptr(angles), half,
         ROTARY_LAYOUTS[layout], _ptr(positions) if temp_every else 0, float(temp_coef), int(temp_every or 0), _ptr(k_pages), _ptr(v_pages),
-        _ptr(kv_slot), qk.shape[0], int(nq), int(nkv), int(dk), int(dv or 0), int(page_size), int(keys_as_values), _stream()), "qk_norm_store")
+        _ptr(kv_slot), qk.shape[0], int(nq), int(nkv), int(dk), int(dv or 0), int(page_size), int(keys_as_values), int(pack), _stream()), "qk_norm_store")
 
 
 # ---- matrix memories with gates that depend on the token -------------------------------------------------
@@ -1319,10 +1339,10 @@ def memory_output(o_raw: torch.Tensor, m_exp: Optional[torch.Tensor], x: torch.T
     when ``m_exp`` is given (``o_raw`` then has one more column), else 1."""
     extra = 0 if m_exp is None else 1
     _dev(weight, torch.float32, "memory_output weight")
-    if weight.numel() != heads * vdim or out.shape != (x.shape[0], heads * vdim) or out.dtype != x.dtype or not out.is_contiguous():
+    if weight.numel() != heads * vdim or out.shape != (x.shape[0], heads * vdim) or out.dtype != x.dtype or out.stride(1) != 1:
         raise KernelError("memory_output: a weight per channel of every head")
     _check(_typed("q25_memory_output", x.dtype)(o_raw.data_ptr(), _ptr(m_exp), x.data_ptr(), x.stride(0), int(g_off), weight.data_ptr(),
-                                                out.data_ptr(), x.shape[0], heads, vdim, extra, float(eps), MEMORY_GATES[gate], _stream()),
+                                                out.data_ptr(), out.stride(0), x.shape[0], heads, vdim, extra, float(eps), MEMORY_GATES[gate], _stream()),
            "memory_output")
 
 
@@ -1435,3 +1455,133 @@ def hyper_embed(table: torch.Tensor, pairs: Optional[torch.Tensor], ids: torch.T
     _check(_typed("q25_hyper_embed", table.dtype)(
         table.data_ptr(), _ptr(pairs), ids.data_ptr(), token_seq.data_ptr(), cu_q.data_ptr(), q_start_pos.data_ptr(), slot_ids.data_ptr(),
         _ptr(last_token), x.data_ptr(), n, width, table.shape[0], int(buckets), int(mul_prev), int(mul_cur), streams, _stream()), "hyper_embed")
+
+
+# ---- differential attention ---------------------------------------------------------------------------------
+
+
+def differential_attention_mma_supports(qkv: torch.Tensor, gate: torch.Tensor, dk: int, dv: int) -> bool:
+    """Sizes and rows the tensor-core kernels of differential attention take; the rest goes to the general kernel."""
+    return (qkv.dtype == torch.bfloat16 and dk in (32, 64, 128) and dv in (32, 64, 128) and (qkv.stride(0) | gate.stride(0)) % 2 == 0
+            and (qkv.data_ptr() | gate.data_ptr()) % 4 == 0)
+
+
+def _check_differential(qkv, gate, out, heads: int, kv_heads: int, dk: int, dv: int) -> None:
+    n = qkv.shape[0]
+    if (heads % kv_heads or qkv.stride(1) != 1 or qkv.shape[1] < 2 * heads * dk or gate.shape != (n, heads * dv) or gate.stride(1) != 1
+            or tuple(out.shape) != (n, heads * dv) or not out.is_contiguous() or gate.dtype != qkv.dtype or out.dtype != qkv.dtype):
+        raise KernelError(f"differential_attention: rows of {2 * heads} queries of {dk} channels and {heads} gates of {dv}, of one dtype")
+
+
+def differential_attention_mma(qkv: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                               block_table: torch.Tensor, cu_q: torch.Tensor, q_start_pos: torch.Tensor, tiles: Optional[torch.Tensor],
+                               items: Optional[torch.Tensor], heads: int, kv_heads: int, dk: int, dv: int, page_size: int, window: int, scale: float,
+                               lam: float, gain: float, eps: float, n_splits: int = 1, scratch: Optional[torch.Tensor] = None) -> None:
+    """Differential attention on tensor cores (bfloat16).  ``qkv``: rows that begin with the queries, by (kv head, map, head
+    of the group); key rows of the pages hold both maps, 2 * dk channels.  ``tiles`` int32 [n, 2] are (entry, tile of 32
+    (token, head of the group) pairs) of the runs, ``items`` the entries that bring one token, whose keys are cut into
+    ``n_splits`` ranges (``scratch`` float32, len(items) * 2 * heads * n_splits * (dv + 2))."""
+    _check_differential(qkv, gate, out, heads, kv_heads, dk, dv)
+    n_items = 0 if items is None else items.shape[0]
+    n_tiles = 0 if tiles is None else tiles.shape[0]
+    part_o = part_ml = 0
+    if n_items and n_splits > 1:
+        rows = n_items * 2 * heads * n_splits
+        if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < rows * (dv + 2):
+            raise KernelError(f"differential_attention_mma: {n_splits} key ranges need {rows * (dv + 2)} float32 of scratch memory")
+        part_o = scratch.data_ptr()
+        part_ml = part_o + 4 * rows * dv
+    if not differential_attention_mma_supports(qkv, gate, dk, dv) or (n_items and heads // kv_heads > 8):
+        raise KernelError(f"differential_attention_mma: unsupported sizes {dk}/{dv} or more than 8 heads per kv head for single tokens")
+    _check(_fn("q25_differential_attention_mma_bf16",
+               [_P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _P, _P, _P])(
+        qkv.data_ptr(), qkv.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], cu_q.data_ptr(), q_start_pos.data_ptr(), _ptr(tiles), n_tiles, _ptr(items), n_items, int(heads), int(kv_heads), int(dk),
+        int(dv), int(page_size), int(window or 0), float(scale), float(lam), float(gain), float(eps), int(n_splits), part_o, part_ml, _stream()),
+        "differential_attention_mma")
+    count_replayed((1 if n_tiles and n_items else 0) + (1 if n_items and n_splits > 1 else 0))
+
+
+def differential_attention_generic(qkv: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                                   block_table: torch.Tensor, token_seq: torch.Tensor, cu_q: torch.Tensor, q_start_pos: torch.Tensor, heads: int,
+                                   kv_heads: int, dk: int, dv: int, page_size: int, window: int, scale: float, lam: float, gain: float,
+                                   eps: float) -> None:
+    """The same for any sizes (values of up to 512 channels), float32 or bfloat16."""
+    _check_differential(qkv, gate, out, heads, kv_heads, dk, dv)
+    if dv > 512:
+        raise KernelError(f"differential_attention: value size {dv} is beyond 512")
+    _check(_typed("q25_differential_attention_generic", qkv.dtype)(
+        qkv.data_ptr(), qkv.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], token_seq.data_ptr(), cu_q.data_ptr(), q_start_pos.data_ptr(), qkv.shape[0], int(heads), int(kv_heads), int(dk), int(dv),
+        int(page_size), int(window or 0), float(scale), float(lam), float(gain), float(eps), _stream()), "differential_attention_generic")
+
+
+# ---- the gated delta rule -------------------------------------------------------------------------------------
+
+
+def delta_walk_finishes(vdim: int, dim: int) -> bool:
+    """Whether the walk can finish the heads itself (a CTA has all of a head's columns)."""
+    return vdim <= (128 if vdim % 4 == 0 and dim <= 256 else 32)
+
+
+def _check_delta(qkv, gates, step_bias, rate_log, state, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+    for t in (gates, step_bias, rate_log, state):
+        _dev(t, torch.float32, "delta rule")
+    if (heads % kv_heads or qkv.shape[1] != 2 * kv_heads * dim + heads * vdim or qkv.stride(1) != 1 or tuple(gates.shape) != (qkv.shape[0], 2 * heads)
+            or step_bias.numel() != heads or rate_log.numel() != heads or state.dim() != 2 or state.shape[1] < heads * dim * vdim):
+        raise KernelError(f"delta rule: rows of {kv_heads} queries and keys of {dim} and {heads} values of {vdim} channels, gates [N, {2 * heads}], slots "
+                          f"that begin with [{heads}, {dim}, {vdim}]")
+
+
+def delta_walk(qkv: torch.Tensor, gates: torch.Tensor, step_bias: torch.Tensor, rate_log: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+               slot_ids: torch.Tensor, n_seqs: int, walked: Optional[torch.Tensor], o_raw: Optional[torch.Tensor], heads: int, kv_heads: int, dim: int,
+               vdim: int, q_scale: float, unit_eps: float, out_gate: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None,
+               norm_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """Tokens in order through the gated delta rule, from and to the requests' states: all entries, or the spans in ``walked``
+    (int32, (first row, end, entry) each).  ``qkv``: rows q | k | v behind the convolution; ``gates`` float32 [N, 2 * heads]: what
+    becomes the decays (softplus(. + step_bias) times -exp(rate_log)), then what becomes the write strengths (sigmoid).  Results
+    go to ``o_raw`` (float32), or, with ``o_raw`` None, to ``out`` as o / rms(o) * norm_weight * silu(out_gate) per head."""
+    _check_delta(qkv, gates, step_bias, rate_log, state, heads, kv_heads, dim, vdim)
+    n = qkv.shape[0]
+    if o_raw is not None:
+        _dev(o_raw, torch.float32, "delta_walk out")
+        if o_raw.numel() != n * heads * vdim:
+            raise KernelError("delta_walk: a result per value channel")
+    elif (not delta_walk_finishes(vdim, dim) or out_gate.shape != (n, heads * vdim) or out.shape != out_gate.shape or out_gate.stride(1) != 1
+          or out.stride(1) != 1 or out.dtype != qkv.dtype or out_gate.dtype != qkv.dtype or norm_weight.numel() != heads * vdim
+          or (vdim > 32 and (state.shape[1] % 4 or state.data_ptr() % 16))):
+        raise KernelError("delta_walk: gate and result are rows of heads * vdim channels of the rows' dtype")
+    n_items = int(n_seqs) if walked is None else walked.numel() // 3
+    _check(_typed("q25_delta_walk", qkv.dtype)(
+        qkv.data_ptr(), qkv.stride(0), kv_heads * dim, 2 * kv_heads * dim, gates.data_ptr(), step_bias.data_ptr(), rate_log.data_ptr(), state.data_ptr(),
+        state.shape[1], cu_q.data_ptr(), slot_ids.data_ptr(), _ptr(walked), n_items, _ptr(o_raw), _ptr(out_gate), 0 if out_gate is None else out_gate.stride(0),
+        _ptr(norm_weight), float(norm_eps), _ptr(out), 0 if out is None else out.stride(0), int(heads), int(kv_heads), int(dim), int(vdim), float(q_scale),
+        float(unit_eps), _stream()), "delta_walk")
+
+
+def delta_mma_supports(dtype: torch.dtype, heads: int, kv_heads: int, dim: int, vdim: int) -> bool:
+    """Sizes of ``delta_runs_mma`` for contiguous rows (every offset a multiple of 8 channels)."""
+    return dtype == torch.bfloat16 and dim in (32, 64, 128) and vdim % 8 == 0 and heads % kv_heads == 0
+
+
+def delta_runs_mma(qkv: torch.Tensor, gates: torch.Tensor, step_bias: torch.Tensor, rate_log: torch.Tensor, state: torch.Tensor, slot_ids: torch.Tensor,
+                   o_raw: torch.Tensor, chunks: torch.Tensor, runs: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, q_scale: float,
+                   unit_eps: float) -> None:
+    """``delta_walk`` on tensor cores for the runs in ``runs`` (int32, (first row, end, entry, first chunk) each), cut into
+    ``chunks`` ((first row, end) each, at most 64 tokens): bfloat16 rows; states, gates and everything made of them float32,
+    operands that are float by nature as sums of two bfloat16 numbers."""
+    _check_delta(qkv, gates, step_bias, rate_log, state, heads, kv_heads, dim, vdim)
+    _dev(o_raw, torch.float32, "delta_runs_mma out")
+    for t in (chunks, runs):
+        _dev(t, torch.int32, "delta_runs_mma work list")
+    if not delta_mma_supports(qkv.dtype, heads, kv_heads, dim, vdim) or qkv.stride(0) % 8 or qkv.data_ptr() % 16 or o_raw.numel() != qkv.shape[0] * heads * vdim:
+        raise KernelError(f"delta_runs_mma: unsupported sizes: {heads} heads, {dim} x {vdim}")
+    n_chunks = chunks.numel() // 2
+    floats = _fn("q25_delta_scratch_floats", [_I, _I, _I, _I])
+    floats.restype = _LL
+    scratch = torch.empty(floats(n_chunks, heads, dim, vdim), dtype=torch.float32, device=qkv.device)
+    _check(_fn("q25_delta_runs_bf16", [_P, _I, _I, _I, _P, _P, _P, _P, _LL, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P])(
+        qkv.data_ptr(), qkv.stride(0), kv_heads * dim, 2 * kv_heads * dim, gates.data_ptr(), step_bias.data_ptr(), rate_log.data_ptr(), state.data_ptr(),
+        state.shape[1], slot_ids.data_ptr(), chunks.data_ptr(), n_chunks, runs.data_ptr(), runs.numel() // 4, scratch.data_ptr(), o_raw.data_ptr(),
+        int(heads), int(kv_heads), int(dim), int(vdim), float(q_scale), float(unit_eps), _stream()), "delta_runs_mma")
+    count_replayed(1)                          # two kernels in one call

@@ -82,23 +82,25 @@ class Linear:
         # the library path adds the bias in the activation dtype
         self._bias_lib = None if bias is None or weight.dtype == torch.float32 else bias.to(weight.dtype)
 
-    def __call__(self, x, out_dtype: Optional[torch.dtype] = None, residual: Optional[torch.Tensor] = None):
+    def __call__(self, x, out_dtype: Optional[torch.dtype] = None, residual: Optional[torch.Tensor] = None,
+                 residual_scale: Optional[torch.Tensor] = None):
         """``x``: activations [M, K] or a ``DeferredNorm``.  With ``residual`` (float32 [M, N])
         the product is added into it and None is returned when the kernel at hand can do
-        that; otherwise the product is returned and the caller adds it later."""
+        that; otherwise the product is returned and the caller adds it later.  ``residual_scale`` (float32
+        [N]): the product is multiplied by it on its way into the residual (a returned one is not)."""
         w = self.weight
         if x.shape[-1] != self.in_features:
             raise ValueError(f"linear: input width {x.shape[-1]} does not match weight {tuple(w.shape)}")
         deferred = isinstance(x, DeferredNorm)
         if w.dtype == torch.bfloat16 and x.shape[0] <= kernels.SKINNY_MAX_ROWS:
-            y = self._skinny(x, deferred, out_dtype, residual)
+            y = self._skinny(x, deferred, out_dtype, residual, residual_scale)
             if y is not NotImplemented:
                 return y
         kernels.chain_flush()           # what follows is no chain product; products that wait come first
         if deferred:
             x = x.materialize()
         if w.dtype == torch.bfloat16 and use_tcgen05(x, w):
-            return self._tcgen05(x, out_dtype, residual)
+            return self._tcgen05(x, out_dtype, residual if residual_scale is None else None)
         if w.dtype == torch.float32:
             out = torch.empty((x.shape[0], self.out_features), dtype=torch.float32, device=x.device)
             kernels.gemm_f32(x, w, self.bias, out)
@@ -128,7 +130,7 @@ class Linear:
         kernels.gemm_tcgen05(x, w, self.bias, out, kernels.SKINNY_BIAS if self.bias is not None else kernels.SKINNY_STORE)
         return out
 
-    def _skinny(self, x, deferred: bool, out_dtype, residual):
+    def _skinny(self, x, deferred: bool, out_dtype, residual, residual_scale=None):
         """The weight-streaming kernel with the epilogue the call asks for, or NotImplemented."""
         w = self.weight
         if deferred:
@@ -137,8 +139,10 @@ class Linear:
         elif not kernels.gemm_skinny_supports(x, w):
             return NotImplemented
         m = x.shape[0]
+        bias = self.bias
         if residual is not None and self.bias is None:
-            epilogue, out, result = kernels.SKINNY_RESIDUAL, residual, None
+            bias = residual_scale
+            epilogue, out, result = (kernels.SKINNY_RESIDUAL if residual_scale is None else kernels.SKINNY_RESIDUAL_SCALED), residual, None
         elif out_dtype == torch.float32:
             if self.bias is not None:
                 return NotImplemented
@@ -148,7 +152,7 @@ class Linear:
             out = torch.empty((m, self.out_features), dtype=w.dtype, device=x.device)
             epilogue, result = (kernels.SKINNY_BIAS if self.bias is not None else kernels.SKINNY_STORE), out
         if deferred:
-            kernels.gemm_skinny_norm(x.x, x.weight, x.eps, w, self.bias, out, epilogue)
+            kernels.gemm_skinny_norm(x.x, x.weight, x.eps, w, bias, out, epilogue)
         else:
-            kernels.gemm_skinny(x, w, self.bias, out, epilogue)
+            kernels.gemm_skinny(x, w, bias, out, epilogue)
         return result

@@ -18,7 +18,7 @@ import torch
 from ..ops import attention as attention_ops
 from ..ops import kernels
 from ..ops.linear import Linear
-from .base import KVCacheNeed, Mixer, TensorSpec, register_mixer
+from .base import KVCacheNeed, Mixer, StateNeed, TensorSpec, register_mixer
 
 
 @register_mixer("gqa_attention")
@@ -222,6 +222,8 @@ class SinkAttention(Mixer):
     the same input as the projections) before ``o``; the gate's product rides with q, k, v and the sigmoid is the
     attention kernels' epilogue.
 
+    ``keep_first``: beside a window the first tokens of the request stay visible, at their true positions.
+
     Three more options.  ``softcap`` c > 0: the scaled score becomes ``c * tanh(score / c)``.
     ``qk_norm_eps`` (a number): before the rotation every query and key head is divided by its root mean
     square (eps inside the root) and multiplied by the weight ``q.norm`` / ``k.norm`` (``head_dim`` numbers,
@@ -235,7 +237,7 @@ class SinkAttention(Mixer):
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: Optional[int] = None,
                  scale: Optional[float] = None, window: Optional[int] = None, sink: Optional[str] = None, position=None,
                  softcap: float = 0.0, qk_norm_eps: Optional[float] = None, values_from_keys: bool = False, qkv_bias: bool = False,
-                 qk_norm_weight: bool = True, q_temp=None, distance_bias=None, out_gate: bool = False):
+                 qk_norm_weight: bool = True, q_temp=None, distance_bias=None, out_gate: bool = False, keep_first: int = 0):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot share {num_kv_heads} kv heads")
         self.qkv_bias, self.qk_norm_weight, self.out_gate = bool(qkv_bias), bool(qk_norm_weight), bool(out_gate)
@@ -256,6 +258,7 @@ class SinkAttention(Mixer):
             raise ValueError(f"values that are the keys have the keys' size {self.head_dim}, not {self.value_dim}")
         self.scale = float(head_dim) ** -0.5 if scale is None else float(scale)
         self.window = None if not window else int(window)
+        self.keep_first = int(keep_first) if self.window else 0
         self.softcap = float(softcap or 0.0)
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
         # an encoding that turns no channel (positions that enter at the embedding or as a bias) is none to this mixer
@@ -266,7 +269,7 @@ class SinkAttention(Mixer):
 
     @property
     def _fused_store(self) -> bool:
-        return self.values_from_keys or self.qk_norm_eps is not None or self.q_temp is not None
+        return self.values_from_keys or self.qk_norm_eps is not None or self.q_temp is not None or (self.keep_first > 0 and self.position is not None)
 
     @property
     def _gate_off(self) -> int:
@@ -297,7 +300,7 @@ class SinkAttention(Mixer):
         return tuple(specs)
 
     def cache_need(self):
-        return KVCacheNeed(self.num_kv_heads, self.head_dim, self.window, self.value_dim)
+        return KVCacheNeed(self.num_kv_heads, self.head_dim, self.window, self.value_dim, self.keep_first)
 
     def load(self, tensors, device, dtype):
         names = ["q", "k"] + ([] if self.values_from_keys else ["v"])
@@ -323,17 +326,17 @@ class SinkAttention(Mixer):
     @property
     def _tcgen05_runs(self) -> bool:
         """Whether this mixer's runs of tokens can go to the tcgen05 prefill kernel (bfloat16 permitting)."""
-        return attention_ops.tcgen05_runs(self.head_dim, self.value_dim, self.num_heads // self.num_kv_heads, self.window, 0, None, 0,
+        return attention_ops.tcgen05_runs(self.head_dim, self.value_dim, self.num_heads // self.num_kv_heads, self.window, self.keep_first, None, 0,
                                           self.softcap)
 
     def plan_key(self):
         if self._tcgen05_runs:
             return ("sink_attention_tcgen05", self.num_heads // self.num_kv_heads, self.num_kv_heads)
-        return ("biased_window_attention", self.num_heads // self.num_kv_heads, self.window or 0, 0)
+        return ("biased_window_attention", self.num_heads // self.num_kv_heads, self.window or 0, self.keep_first)
 
     def plan_step(self, host):
         group = self.num_heads // self.num_kv_heads
-        plan = attention_ops.plan_biased(host, group, self.window or 0, 0)
+        plan = attention_ops.plan_biased(host, group, self.window or 0, self.keep_first)
         if self._tcgen05_runs:
             places = 2 * kernels.sm_count() // self.num_kv_heads           # two CTAs of the tcgen05 kernel fit an SM
             wide = attention_ops.plan_step(host, group, 0, places)
@@ -341,8 +344,16 @@ class SinkAttention(Mixer):
         return plan
 
     def forward(self, ctx, h, stop, residual=None):
+        return self.o_proj(self.between(ctx, self.qkv_proj(h), stop), residual=residual)
+
+    def products(self):
+        return self.qkv_proj, self.o_proj
+
+    def drop_products(self):
+        self.qkv_proj = self.o_proj = None
+
+    def between(self, ctx, qkv, stop, side=None, out=None):
         nq, nkv, dk, dv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim
-        qkv = self.qkv_proj(h)
         kv = ctx.kv(stop)
         if self._fused_store:
             angles = self.position.angles(ctx) if self.position is not None else None
@@ -359,9 +370,107 @@ class SinkAttention(Mixer):
                 self.position.rotate(ctx, qk, qk, dk)
             if stop.owns_cache:
                 kernels.kv_store_mix(qkv, None, 0.0, kv.k_pages, kv.v_pages, kv.kv_slot, nq, nkv, dk, dv, kv.page_size)
-        out = attention_ops.attend_biased(ctx, ctx.plan(self), qkv, kv, nq, nkv, dk, dv, self.window, 0, self.scale, None, None,
-                                          self.sink, softcap=self.softcap, dist_bias=self.dist_table, gate_off=self._gate_off)
-        return self.o_proj(out, residual=residual)
+        return attention_ops.attend_biased(ctx, ctx.plan(self), qkv, kv, nq, nkv, dk, dv, self.window, self.keep_first, self.scale, None, None,
+                                           self.sink, softcap=self.softcap, dist_bias=self.dist_table, gate_off=self._gate_off, out=out)
+
+
+@register_mixer("differential_attention")
+class DifferentialAttention(Mixer):
+    """Differential attention (Ye, Dong, Xia, Sun, Zhu, Huang, Wei, "Differential Transformer"): every head has two maps,
+    each a softmax attention of its own over the same values, and the second is subtracted from the first,
+
+        o = a1 - lambda a2,   lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + diff   (one number per layer),
+
+    then each head's o is divided by its root mean square (no weight) and multiplied by ``1 - diff``.  Query head h reads
+    key/value head ``h // (num_heads / num_kv_heads)``; a query or key head has 2 * ``head_dim`` channels, map 1 then map 2, a
+    value ``value_dim``.  ``conv``: a causal convolution of that many taps over time on every channel of q, k and v, right
+    behind the projections (tensors ``q.conv``, ``k.conv``, ``v.conv``, no bias); its last inputs are per-request state.
+    Then query/key norm per head and map (weights ``q.norm``, ``k.norm`` of ``head_dim`` numbers shared by heads and maps) and
+    the layer's rotation.  A sliding ``window`` (None: causal).  The concatenated heads are multiplied channel by channel
+    with ``sigmoid(Wg h)`` (tensor ``g``) before ``o``.
+
+    The gate's product rides with q, k and v.  In the cache a key row holds both maps side by side over one value row, so
+    a key tile is fetched once for both.  Queries are kept ordered by (key/value head, map, head of the group).  Two
+    softmaxes, the difference, its norm and the gate are one kernel (``csrc/attention_differential.cu``); scores,
+    softmax, both maps' results and everything behind them are float32 in both dtypes."""
+
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+    accepts_residual = True          # the output projection can add into the residual stream itself
+    accepts_scaled_residual = True
+    accepts_deferred_norm = True     # one product reads the mixer's input
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, scale: float, diff: float, norm_eps: float,
+                 window: Optional[int] = None, conv: int = 1, position=None):
+        if num_heads % num_kv_heads:
+            raise ValueError(f"{num_heads} query heads cannot share {num_kv_heads} kv heads")
+        self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.head_dim, self.value_dim, self.scale, self.diff, self.norm_eps = int(head_dim), int(value_dim), float(scale), float(diff), float(norm_eps)
+        if not 0 < self.value_dim <= 512 or self.head_dim <= 0:
+            raise ValueError(f"key size {head_dim} / value size {value_dim} is not supported: values take up to 512 channels")
+        self.window, self.conv = None if not window else int(window), int(conv)
+        if not 1 <= self.conv <= 16:
+            raise ValueError(f"the convolution takes 1 to 16 taps, got {conv}")
+        self.position = position if getattr(position, "dims", 0) > 0 else None
+        if self.position is not None and position.dims > self.head_dim:
+            raise ValueError(f"the position encoding turns {position.dims} channels, a map of a head has {head_dim}")
+        self.group = self.num_heads // self.num_kv_heads
+        self.channels = 2 * (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim     # q | k | v
+        self.in_proj = self.o_proj = None
+
+    def tensor_specs(self):
+        h, D = self.hidden_size, self.head_dim
+        q, k, v, o = 2 * self.num_heads * D, 2 * self.num_kv_heads * D, self.num_kv_heads * self.value_dim, self.num_heads * self.value_dim
+        specs = [TensorSpec("q", (q, h)), TensorSpec("k", (k, h)), TensorSpec("v", (v, h)), TensorSpec("q.norm", (D,), "norm"), TensorSpec("k.norm", (D,), "norm")]
+        specs += [TensorSpec(f"{n}.conv", (rows, self.conv), "matrix_wide", optional=self.conv == 1) for n, rows in (("q", q), ("k", k), ("v", v))]
+        specs += [TensorSpec(n, (D,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
+        return tuple(specs + [TensorSpec("g", (o, h)), TensorSpec("o", (h, o))])
+
+    def cache_need(self):
+        return KVCacheNeed(self.num_kv_heads, 2 * self.head_dim, self.window, self.value_dim)
+
+    def state_need(self):
+        return StateNeed(((self.conv - 1) * self.channels,), "float32") if self.conv > 1 else None
+
+    def load(self, tensors, device, dtype):
+        G, D = self.num_kv_heads, self.head_dim
+        by_map = lambda t: t.reshape(G, self.group, 2, D, -1).transpose(1, 2).reshape(2 * self.num_heads * D, -1)
+        w = torch.cat([by_map(tensors["q"]), tensors["k"], tensors["v"], tensors["g"]], dim=0)
+        self.in_proj = Linear(w.to(device=device, dtype=dtype).contiguous())
+        self.o_proj = Linear(tensors["o"].to(device=device, dtype=dtype).contiguous())
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        self.q_norm, self.k_norm = f32(tensors["q.norm"]), f32(tensors["k.norm"])
+        self.conv_w = None
+        if "q.conv" in tensors:
+            self.conv_w = f32(torch.cat([by_map(tensors["q.conv"]), tensors["k.conv"], tensors["v.conv"]], dim=0).t())        # [taps, channels]
+            self.conv_b = torch.zeros(self.channels, dtype=torch.float32, device=device)
+            self.no_state = torch.zeros((1, 0), dtype=torch.float32, device=device)             # what one tap carries from step to step
+        l = {n: tensors[n].double() for n in ("lq1", "lk1", "lq2", "lk2")}
+        self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + self.diff
+
+    def plan_key(self):
+        return ("biased_window_attention", 2 * self.group, self.window or 0, 0)
+
+    def plan_step(self, host):
+        return attention_ops.plan_biased(host, 2 * self.group, self.window or 0, 0)
+
+    def forward(self, ctx, h, stop, residual=None, residual_scale=None):
+        """Returns the update of the residual stream, or None after adding it into ``residual``."""
+        nq, nkv, D, Dv = 2 * self.num_heads, 2 * self.num_kv_heads, self.head_dim, self.value_dim
+        x = self.in_proj(h)                                             # [N, q | k | v | gate]
+        n, ch = x.shape[0], self.channels
+        qkv = x
+        if self.conv_w is not None:
+            qkv = torch.empty((n, ch), dtype=x.dtype, device=x.device)
+            state = self.no_state if self.conv == 1 else stop.state
+            kernels.causal_conv(x[:, :ch], self.conv_w, self.conv_b, state, 0, ctx.cu_q, ctx.slot_ids, qkv, ctx.n_seqs, ctx.max_q_len, silu=False)
+        kv, own = ctx.kv(stop), stop.owns_cache
+        angles = self.position.angles(ctx) if self.position is not None else None
+        layout = self.position.layout if self.position is not None else "halves"
+        kernels.qk_norm_store(qkv, self.q_norm, self.k_norm, self.norm_eps, angles, layout, kv.k_pages if own else None, kv.v_pages if own else None,
+                              kv.kv_slot if own else None, nq, nkv, D, kv.page_size, False, unit_norm=True, dv=Dv, pack=2)
+        out = attention_ops.attend_differential(ctx, ctx.plan(self), qkv, x[:, ch:], kv, self.num_heads, self.num_kv_heads, D, Dv, self.window,
+                                                self.scale, self.lam, 1.0 - self.diff, self.norm_eps)
+        return self.o_proj(out, residual=residual, residual_scale=residual_scale)
 
 
 @register_mixer("latent_attention")

@@ -85,6 +85,7 @@ class Part:
     # What a part may declare about itself (class attributes); the defaults promise nothing.
     graph_safe = False              # forward is a fixed sequence of this engine's kernels: a step may be captured
     accepts_residual = False        # forward takes ``residual=`` and may add its result into the float32 stream
+    accepts_scaled_residual = False  # the same with ``residual_scale=``: a float32 factor per channel on the result's way into the stream
     accepts_deferred_norm = False   # forward takes an ``ops.linear.DeferredNorm`` to normalise inside its first product
 
     def tensor_specs(self) -> Sequence[TensorSpec]:
@@ -197,6 +198,12 @@ class Mixer(Part):
     ``ctx.slot_ids``.  A mixer with state must process a request's tokens in order and must
     give the same result wherever the run of tokens is cut.
 
+    A mixer whose forward is a product, what lies between, and a product may offer the three apart, so that mixers side by
+    side run as one product each way (``parts.composite.SummedMixers``): ``products() -> (Linear in, Linear out)``,
+    ``between(ctx, x, stop, side=None, out=None) -> [N, K]`` on the first product's rows ``x`` (possibly a strided view), the
+    result in ``out`` when given (rows, possibly strided); ``side_products(ctx, h)``, whatever else reads the mixer's
+    input, which ``between`` gets as ``side``; and ``drop_products()`` once others hold the products.
+
     A part whose kernels read per-step work lists may define ``plan_step(host) -> {name: int32
     array}`` (``host.q_lens``, ``host.starts``, ``host.n_tokens``, ``host.n_seqs`` describe the
     step) and ``plan_key()`` (parts with equal keys share one plan).  The step function packs the
@@ -209,6 +216,9 @@ class Mixer(Part):
         return None
 
     def state_need(self) -> Optional[StateNeed]:
+        return None
+
+    def side_products(self, ctx, h):
         return None
 
     def forward(self, ctx, h, stop):

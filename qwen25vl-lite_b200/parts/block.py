@@ -46,6 +46,30 @@ class SandwichResidualBlock(Block):
         return PendingUpdate(self.feed_forward.forward(ctx, h), self.norms[3])
 
 
+@register_block("scaled_residual")
+class ScaledResidualBlock(Block):
+    """Pre-norm sublayers whose results are scaled per channel on their way into the stream: ``x += s1 * mixer(norm1(x))``,
+    then ``x += s2 * ffn(norm2(x))``; the norms come in that order (norm1, s1, norm2, s2, the scales being
+    ``channel_scale`` parts).  A part that says ``accepts_scaled_residual`` is handed the stream and the scale and may add
+    its result itself; otherwise the result is a ``PendingUpdate`` that the next norm's kernel scales and adds."""
+
+    @staticmethod
+    def _update(part, scale, x, *args):
+        if not part.accepts_scaled_residual:
+            return PendingUpdate(part.forward(*args), scale)
+        value = part.forward(*args, residual=x, residual_scale=scale.weight)
+        return None if value is None else PendingUpdate(value, scale)
+
+    def forward(self, ctx, x, pending, stop):
+        mixer, ffn = self.mixer, self.feed_forward
+        h = self.norms[0].forward(ctx, x, pending, defer=mixer.accepts_deferred_norm)
+        mixed = self._update(mixer, self.norms[1], x, ctx, h, stop)
+        if ffn is None:
+            return mixed
+        h = self.norms[2].forward(ctx, x, mixed, defer=ffn.accepts_deferred_norm)
+        return self._update(ffn, self.norms[3], x, ctx, h)
+
+
 @register_block("hyper_residual")
 class HyperResidualBlock(Block):
     """Pre-norm sublayers over a stream of several rows per token (``parts.norm.HyperRMSNorm``): each sublayer's norm reads

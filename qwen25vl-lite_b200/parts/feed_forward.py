@@ -174,16 +174,16 @@ class RoutedGLU(FeedForward):
         return out
 
 
-def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, limit: float, alpha: float, shift: float):
+def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, limit: float, alpha: float, shift: float, gated: bool = True):
     """The grouped products of a routed feed-forward.  ``route(topk_idx, topk_w, counts)`` launches the router, which
     writes every token's ``top`` choices (int32 [N, top]; a choice beyond the experts that have matrices takes no row),
     their weights (float32) and how many tokens chose each expert.  The pairs are sorted by expert on the device and
     two grouped products walk them: ``act = g * sigmoid(alpha g) * (u + shift)`` with ``g = min(Wg a, limit)``,
     ``u = clamp(Wu a, -limit, limit)``, then ``Wd act``; ``a`` is the token's row times the pair's weight
-    (``weigh_input``) or the row as it is.  Returns (float32 rows in the sorted order, the row of every pair or -1,
+    (``weigh_input``) or the row as it is.  ``gated`` False: the experts have up rows alone, ``act = max(Wu a, 0)^2``.  Returns (float32 rows in the sorted order, the row of every pair or -1,
     the weights)."""
     experts, ff2, hidden = w_gate_up.shape
-    expert_size = ff2 // 2
+    expert_size = ff2 // 2 if gated else ff2
     n, dev = h.shape[0], h.device
     pairs = n * top
     # rows of a tile of the grouped products, from the step's shape alone: 16 while an expert gets up to 16
@@ -214,12 +214,15 @@ def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, 
         # (which finds its tiles in the plan on the device), the activation, and down the same way
         sorted_rows = torch.empty((rows, hidden), dtype=ctx.dtype, device=dev)
         kernels.moe_gather(h, row_pair, in_w, top, sorted_rows)
-        gate_up = torch.empty((rows, 2 * expert_size), dtype=ctx.dtype, device=dev)
-        kernels.gemm_tcgen05_grouped(sorted_rows, w_gate_up, gate_up, plan)
-        kernels.glu_clamped(gate_up, act, limit, alpha, shift=shift)
+        if gated:
+            gate_up = torch.empty((rows, 2 * expert_size), dtype=ctx.dtype, device=dev)
+            kernels.gemm_tcgen05_grouped(sorted_rows, w_gate_up, gate_up, plan)
+            kernels.glu_clamped(gate_up, act, limit, alpha, shift=shift)
+        else:
+            kernels.gemm_tcgen05_grouped(sorted_rows, w_gate_up, act, plan, kernels.SKINNY_RELU2)
         kernels.gemm_tcgen05_grouped(act, w_down, y, plan)
     else:
-        kernels.moe_gate_up(h, w_gate_up, act, plan, row_pair, in_w, top, limit, alpha, tile, shift=shift, n_pairs=pairs)
+        kernels.moe_gate_up(h, w_gate_up, act, plan, row_pair, in_w, top, limit, alpha, tile, shift=shift, n_pairs=pairs, gated=gated)
         kernels.moe_down(act, w_down, y, plan, row_pair, pairs, top, tile)
     return y, pair_row, topk_w
 
@@ -291,6 +294,60 @@ class GroupedRoutedGLU(FeedForward):
         y, pair_row, topk_w = _run_experts(ctx, h, self.w_gate_up, self.w_down, self.top, route, False, float("inf"), 1.0, 0.0)
         out = torch.empty((h.shape[0], self.hidden_size), dtype=ctx.dtype, device=h.device)
         kernels.moe_combine_weighted(y, pair_row, topk_w, h, out, self.top, shared)
+        return out
+
+
+@register_feed_forward("grouped_routed_mlp")
+class GroupedRoutedMLP(FeedForward):
+    """A mixture of ``experts`` small feed-forwards without a gate and without biases, ``Wd max(Wu h, 0)^2``, of which each
+    token uses ``top``, with a router that scores every expert by itself and chooses inside groups.
+
+    Router: ``z = Wr h`` in float32, scores ``s = sigmoid(z)``.  The choice looks at ``s + correction`` (a learned vector);
+    the experts form ``groups`` equal runs of neighbours, a run's mark is the sum of its two largest such numbers, and only
+    experts of the ``keep`` runs with the largest marks can be chosen (the others count as minus infinity).  The ``top``
+    largest are chosen; their outputs weigh in with their plain scores ``s``, not renormalised.  Tensors: ``router``,
+    ``correction``, ``e<i>.up|down``.
+
+    Router, sort by expert and grouped products are those of the other mixtures (``csrc/moe.cu``, and the grouped mode of
+    ``csrc/gemm_tcgen05.cu`` with the square of relu as its epilogue); the kernel that sums a token's choices can add the
+    sum, scaled per channel, into the residual stream."""
+
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+    accepts_scaled_residual = True
+
+    def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, groups: int = 1, keep: int = 1, correction: bool = True):
+        self.hidden_size, self.experts, self.top, self.expert_size = int(hidden_size), int(experts), int(top), int(expert_size)
+        self.groups, self.keep, self.has_correction = max(int(groups), 1), max(int(keep), 1), bool(correction)
+        if not 1 <= self.experts <= 256 or not 1 <= self.top <= 16:
+            raise ValueError(f"the router takes up to 256 experts and chooses 1 to 16 of them, got {experts} and {top}")
+        if self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError(f"{experts} experts do not form {groups} equal groups of which {keep} are kept")
+        if self.top > self.keep * (self.experts // self.groups):
+            raise ValueError(f"{top} choices cannot come from {keep} groups of {self.experts // self.groups}")
+
+    def tensor_specs(self):
+        h, f = self.hidden_size, self.expert_size
+        specs = []
+        for e in range(self.experts):
+            specs += [TensorSpec(f"e{e}.up", (f, h)), TensorSpec(f"e{e}.down", (h, f))]
+        specs.append(TensorSpec("router", (self.experts, h), "matrix_wide"))
+        if self.has_correction:
+            specs.append(TensorSpec("correction", (self.experts,), "bias"))
+        return tuple(specs)
+
+    def load(self, tensors, device, dtype):
+        stack = lambda name: torch.stack([tensors[f"e{e}.{name}"] for e in range(self.experts)]).to(device=device, dtype=dtype).contiguous()
+        self.w_up, self.w_down = stack("up"), stack("down")
+        self.router = tensors["router"].to(device=device, dtype=torch.float32).contiguous()
+        self.correction = tensors["correction"].to(device=device, dtype=torch.float32).contiguous() if self.has_correction else None
+
+    def forward(self, ctx, h, residual=None, residual_scale=None):
+        """Returns the update of the residual stream, or None after adding it (scaled) into ``residual``."""
+        route = lambda idx, w, counts: kernels.moe_route_softmax(h, self.router, self.correction, self.experts, self.top, self.groups,
+                                                                 self.keep, idx, w, counts, scores="sigmoid", mark="two_largest")
+        y, pair_row, topk_w = _run_experts(ctx, h, self.w_up, self.w_down, self.top, route, False, 0.0, 0.0, 0.0, gated=False)
+        out = None if residual is not None else torch.empty((h.shape[0], self.hidden_size), dtype=ctx.dtype, device=h.device)
+        kernels.moe_combine_weighted(y, pair_row, topk_w, h, out, self.top, residual=residual, residual_scale=residual_scale)
         return out
 
 

@@ -21,6 +21,12 @@ and request, a float32 state ``S`` [dim, value_dim] from token to token: ``S_t =
   shared by groups of consecutive heads, v = x; ``y_t = o_t + D x_t``, the heads are concatenated, multiplied by
   ``silu(z)``, RMS-normed in equal parts with a weight over all channels, and projected by ``Wo``.  The state keeps the
   convolution's last inputs beside S.
+* ``gated_delta_rule`` (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule"): q, k and v pass
+  a short causal convolution and silu, q and k become unit vectors per head; per head a decay
+  ``a_t = exp(-exp(A_log) softplus(Wa h + dt_bias))`` and a write strength ``beta_t = sigmoid(Wb h)``; the memory is told the
+  difference between a value and what it would answer, ``S <- a_t S``, ``S <- S + k_t (beta_t (v_t - S^T k_t))^T``,
+  ``o_t = S^T q_t``; each head's o is RMS-normed with one weight shared by the heads, multiplied by ``silu(Wg h)`` and
+  projected by ``Wo``.
 
 Float32 in both dtypes: the decays and gates from their pre-activations on (the gate rows of ``mlstm`` and the second
 factor of the decay's projection are float32 products in a fixed order; the steps of ``mamba2`` leave their product in
@@ -35,8 +41,8 @@ from __future__ import annotations
 import numpy as np
 import torch
 
-from ..ops import kernels, state_space
-from ..ops.linear import Linear
+from ..ops import delta_rule, kernels, state_space
+from ..ops.linear import DeferredNorm, Linear
 from .base import Mixer, StateNeed, TensorSpec, register_mixer
 
 
@@ -233,3 +239,99 @@ class Mamba2(Mixer):
         out = torch.empty((n, inner), dtype=zx.dtype, device=zx.device)
         kernels.ssd_output(o_raw, xbc[:, :inner], zx[:, :inner], self.skip, self.norm_weight, self.norm_groups, self.norm_eps, out, self.value_dim)
         return self.out_proj(out, residual=residual)
+
+
+@register_mixer("gated_delta_rule")
+class GatedDeltaRule(Mixer):
+    """``num_heads`` heads of ``value_dim`` channels over ``num_kv_heads`` query and key heads of ``head_dim`` (head h reads
+    number ``h // (num_heads / num_kv_heads)``); ``conv`` taps.  Tensors: ``q``, ``k``, ``v`` with ``.conv`` (no biases), ``a``,
+    ``dt_bias``, ``A_log``, ``b``, ``g``, ``norm``, ``o``.  The rows of a and b are a product of their own, whose result stays in
+    float32.  A slot's state: S [heads, head_dim, value_dim], then the convolution's last inputs over q | k | v."""
+
+    graph_safe = True                # forward is a fixed sequence of this engine's kernels
+    accepts_residual = True          # the output projection can add into the residual stream itself
+    accepts_scaled_residual = True
+    accepts_deferred_norm = True
+    UNIT_EPS = 1e-6                  # inside the root when q and k become unit vectors
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, conv: int, norm_eps: float, position=None):
+        self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
+        self.head_dim, self.value_dim, self.conv, self.norm_eps = int(head_dim), int(value_dim), int(conv), float(norm_eps)
+        if self.num_kv_heads < 1 or self.num_heads % self.num_kv_heads:
+            raise ValueError(f"{num_heads} heads cannot share {num_kv_heads} query and key heads")
+        if not 0 < self.head_dim <= 512:
+            raise ValueError(f"a memory's key size is 1 to 512, got {head_dim}")
+        if not 1 <= self.conv <= 16:
+            raise ValueError(f"the convolution takes 1 to 16 taps, got {conv}")
+        self.channels = 2 * self.num_kv_heads * self.head_dim + self.num_heads * self.value_dim
+        self.in_proj = self.o_proj = self.gate_proj = None
+
+    def tensor_specs(self):
+        h, H, qk, v = self.hidden_size, self.num_heads, self.num_kv_heads * self.head_dim, self.num_heads * self.value_dim
+        return (TensorSpec("q", (qk, h)), TensorSpec("q.conv", (qk, self.conv), "matrix_wide"), TensorSpec("k", (qk, h)),
+                TensorSpec("k.conv", (qk, self.conv), "matrix_wide"), TensorSpec("v", (v, h)), TensorSpec("v.conv", (v, self.conv), "matrix_wide"),
+                TensorSpec("b", (H, h), "matrix_wide"), TensorSpec("A_log", (H,), "bias"), TensorSpec("norm", (self.value_dim,), "norm"),
+                TensorSpec("a", (H, h), "matrix_wide"), TensorSpec("dt_bias", (H,), "bias"), TensorSpec("g", (v, h)), TensorSpec("o", (h, v)))
+
+    @property
+    def _memory_floats(self) -> int:
+        return self.num_heads * self.head_dim * self.value_dim
+
+    def state_need(self):
+        floats = self._memory_floats + (self.conv - 1) * self.channels
+        return StateNeed((-(-floats // 4) * 4,), "float32")              # every slot starts on a 16-byte boundary
+
+    def load(self, tensors, device, dtype):
+        f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
+        rows = lambda *names: torch.cat([tensors[n] for n in names], dim=0).to(device=device, dtype=dtype).contiguous()
+        self.dtype = dtype
+        self.in_proj = Linear(rows("q", "k", "v", "g"))
+        self.gate_proj = Linear(rows("a", "b"))
+        self.o_proj = Linear(rows("o"))
+        self.conv_w = f32(torch.cat([tensors[n] for n in ("q.conv", "k.conv", "v.conv")], dim=0).t())              # [taps, channels]
+        self.conv_b = torch.zeros(self.channels, dtype=torch.float32, device=device)
+        self.rate_log, self.step_bias = f32(tensors["A_log"]), f32(tensors["dt_bias"])
+        self.norm_weight = f32(tensors["norm"]).repeat(self.num_heads).contiguous()                               # the same for every head
+
+    def products(self):
+        return self.in_proj, self.o_proj
+
+    def drop_products(self):
+        self.in_proj = self.o_proj = None
+
+    def scale_heads(self, factor: float):
+        """The heads times a constant: it rides in the output norm's float32 weight."""
+        self.norm_weight = (self.norm_weight * factor).contiguous()
+
+    @property
+    def _tensor_cores(self) -> bool:
+        """Whether this mixer's runs of tokens can go to the tensor-core kernels."""
+        return kernels.delta_mma_supports(getattr(self, "dtype", torch.float32), self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim)
+
+    def plan_key(self):
+        return ("delta_rule", self._tensor_cores)
+
+    def plan_step(self, host):
+        return delta_rule.plan(host.q_lens, self._tensor_cores)
+
+    def side_products(self, ctx, h):
+        return self.gate_proj(h, out_dtype=torch.float32)               # [N, a of every head | b of every head]
+
+    def between(self, ctx, x, stop, side=None, out=None):
+        """``x``: rows q | k | v | g as projected."""
+        H, G, D, Dv, n = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, x.shape[0]
+        state = stop.state
+        qkv = torch.empty((n, self.channels), dtype=x.dtype, device=x.device)
+        kernels.causal_conv(x[:, :self.channels], self.conv_w, self.conv_b, state, self._memory_floats, ctx.cu_q, ctx.slot_ids, qkv, ctx.n_seqs,
+                            ctx.max_q_len, silu=True)
+        if out is None:
+            out = torch.empty((n, H * Dv), dtype=x.dtype, device=x.device)
+        delta_rule.run(ctx.plan(self), ctx, qkv, side, self.step_bias, self.rate_log, state, x[:, self.channels:], self.norm_weight, self.norm_eps, out,
+                       H, G, D, Dv, float(D) ** -0.5, self.UNIT_EPS)
+        return out
+
+    def forward(self, ctx, h, stop, residual=None, residual_scale=None):
+        if isinstance(h, DeferredNorm) and not kernels.gemm_skinny_norm_supports(h.x, self.in_proj.weight):
+            h = h.materialize()
+        x = self.in_proj(h)
+        return self.o_proj(self.between(ctx, x, stop, side=self.side_products(ctx, h)), residual=residual, residual_scale=residual_scale)

@@ -1,5 +1,5 @@
 """Normalisations fused with the residual update: RMS norm (of one stream or of several), Dynamic Tanh, layer
-norm, and no norm at all.
+norm, no norm at all, and the scale per channel that may stand behind a sublayer in a norm's place.
 
 Formula (reference src/qwen25vl_lite/layers.py:27-31): ``x * rsqrt(mean(x^2) + eps) * w``,
 statistics in float32, plain (not 1 + w) weight.  With ``groups`` > 1 the vector is cut into
@@ -74,11 +74,38 @@ class RMSNorm(Norm):
         if plain:
             kernels.add_rmsnorm(x, delta, self.weight, self.eps, out, rows)
         else:
-            if post is not None and not isinstance(post, RMSNorm):
-                raise TypeError("a pending update can be normalised by an rmsnorm only")
+            if post is not None and not isinstance(post, (RMSNorm, ChannelScale)):
+                raise TypeError("a pending update can be normalised by an rmsnorm or scaled per channel only")
             kernels.add_norm_groups(x, delta, None if post is None else post.weight, 0.0 if post is None else post.eps,
                                     1 if post is None else post.groups, self.weight, self.eps, self.groups, out, rows)
         return out
+
+
+@register_norm("channel_scale")
+class ChannelScale(Norm):
+    """No norm but what stands in a norm's place behind a sublayer: the sublayer's result is multiplied channel by
+    channel with a learned vector (a layer scale) times the constant ``gain`` on its way into the stream,
+    ``x += gain * w * value``.  It is only ever the norm of a ``PendingUpdate``, or handed (``weight``) to a sublayer
+    that adds into the stream itself.  The product of the vector and the constant is float32."""
+
+    graph_safe = True
+    eps, groups = 0.0, 0             # what the kernel that adds a pending update reads: no groups, no norm
+
+    def __init__(self, dim: int, name: str = "weight", gain: float = 1.0, optional: bool = False):
+        self.dim, self.name, self.gain, self.optional = int(dim), name, float(gain), bool(optional)
+        self.weight = None
+
+    def tensor_specs(self):
+        return (TensorSpec(self.name, (self.dim,), init="fraction", optional=self.optional),)
+
+    def load(self, tensors, device, dtype):
+        if self.name in tensors:
+            self.weight = (tensors[self.name].to(device=device, dtype=torch.float32) * self.gain).contiguous()
+        elif not self.optional:
+            raise KeyError(self.name)
+
+    def add_only(self, ctx, x, value):
+        kernels.add_norm_groups(x, value, self.weight, 0.0, 0, None, 0.0, 1, None, None, dtype=ctx.dtype)
 
 
 @register_norm("hyper_rmsnorm")
