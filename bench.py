@@ -1,7 +1,7 @@
 #!/usr/bin/env python3
 """Decode and prefill throughput of the engine at Qwen2.5-VL sizes, random bfloat16 weights.
 
-    python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 3b|7b-trace|32b|rirulix|labolix|mozutar|fatilix|mezinex]
+    python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--config 3b|7b-trace|32b|rirulix|labolix|mozutar|fatilix|mezinex|sudilorn]
 
 One "step" is one decode step of the whole batch.  The default run (``--config 3b``) has the 3B
 layer sizes: the headline ``value`` is decoded tokens a second at batch 8 after 2,048-token
@@ -12,7 +12,7 @@ decode at batch 1 and 64, the clocks seen while timing, and the number of this e
 launches in the timed region.  ``--config 7b-trace`` runs a continuous-batching trace of 128
 requests at the 7B sizes, ``--config 32b`` decode at batch 1 / 8 / 32 after 8,192-token prompts and
 a 2,048-token prefill at the 32B sizes, ``--config rirulix`` / ``--config labolix`` / ``--config mozutar`` / ``--config fatilix`` / ``--config mezinex`` prefill and decode of the Rirulix / Labolix / Mozutar / Fatilix / Mezinex design
-at a few layer sizes beside this decoder at equal size; each prints one line of its own.
+at a few layer sizes beside this decoder at equal size, ``--config sudilorn`` the Sudilorn design beside the Mozutar design; each prints one line of its own.
 The engine is single-GPU: for --gpus N > 1 one line says so and the exit code is 2.
 """
 
@@ -589,6 +589,43 @@ def run_mezinex(args):
     return _run_design(args, "Mezinex", "mezinex", MEZINEX_SIZES)
 
 
+def _sudilorn_sizes(width, layers, heads, kv_heads, dim, window, keep, mem_heads, mem_kv, mem_dim, experts, groups, kept, top, ff, vocab):
+    """A Sudilorn model of ``layers`` layers (differential attention, then window attention beside a gated delta rule twice, and
+    so on; routed experts in each; a map of the differential attention has half a head's channels) and, as the closest
+    model the engine had, a Mozutar model of equal size beside it: the same width, layers, heads, memories, experts and
+    vocabulary (softmax beside gated linear attention twice, then an mLSTM, no stretch that runs twice)."""
+    router = {"experts": experts, "top": top, "groups": {"count": groups, "keep": kept}}
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": router}
+    diff = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "conv": 4, "diff": 0.5, "scale": (dim // 2) ** -0.5,
+                                           "mask": {"size": window}, "rot": {"dims": dim // 2, "base": 250000.0,
+                                                                             "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    par = {"type": "parallel", "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                  "mask": {"size": window, "keep_first": keep}, "rot": {"dims": dim // 2, "base": 10000.0}},
+                                         "right": {"heads": mem_heads, "kv_heads": mem_kv, "dim": mem_dim, "vdim": mem_dim, "conv": 4},
+                                         "left_scale": 0.8, "right_scale": 0.6}}
+    ours = {"architecture": "Sudilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "layers": [dict((diff, par, par)[i % 3], mlp=moe) for i in range(layers)]}
+    gla = {"type": "parallel", "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+                                                  "rot": {"dims": dim // 2, "base": 10000.0}},
+                                         "right": {"heads": mem_heads, "dim": mem_dim, "vdim": mem_dim, "tau": 16.0, "rank": 32}}}
+    mem = {"type": "mlstm", "mixer": {"heads": mem_heads, "dim": mem_dim, "vdim": mem_dim, "gate_cap": 15.0}}
+    closest = {"architecture": "Mozutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
+               "layers": [dict((gla, gla, mem)[i % 3], mlp=dict(moe, router=dict(router, identity=0))) for i in range(layers)]}
+    return ours, closest
+
+
+SUDILORN_SIZES = {
+    "w1024": _sudilorn_sizes(1024, 6, 8, 2, 128, 1024, 4, 8, 4, 128, 8, 4, 2, 2, 1408, 32000),
+    "w2048": _sudilorn_sizes(2048, 6, 16, 2, 128, 1024, 4, 16, 8, 128, 16, 4, 2, 2, 2816, 32000),
+    "w2560_d64": _sudilorn_sizes(2560, 6, 40, 8, 64, 1024, 4, 40, 40, 64, 32, 8, 4, 4, 1728, 32000),
+}
+
+
+def run_sudilorn(args):
+    """The same measurement for the Sudilorn design, beside the Mozutar design of equal size."""
+    return _run_design(args, "Sudilorn", "sudilorn", SUDILORN_SIZES)
+
+
 def run_rirulix(args):
     """Prefill and decode throughput of the Rirulix design at a few layer sizes, each beside the
     Qwen2.5-VL text decoder of equal size, random weights: a 2,048-token prompt in one step, and
@@ -668,10 +705,10 @@ def main(argv=None):
     ap.add_argument("--only-batch", type=int, default=0, help="time decode steps at this batch size only (for profilers)")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
                     help="float32 times the true 32-bit path of the 3b configuration (fewer --layers advised)")
-    ap.add_argument("--only-size", default="", help="with --config rirulix, labolix, mozutar, fatilix or mezinex: one of its sizes only (for profilers)")
-    ap.add_argument("--config", default="3b", choices=["3b", "7b-trace", "32b", "rirulix", "labolix", "mozutar", "fatilix", "mezinex"],
+    ap.add_argument("--only-size", default="", help="with --config rirulix, labolix, mozutar, fatilix, mezinex or sudilorn: one of its sizes only (for profilers)")
+    ap.add_argument("--config", default="3b", choices=["3b", "7b-trace", "32b", "rirulix", "labolix", "mozutar", "fatilix", "mezinex", "sudilorn"],
                     help="3b: the headline line (default); 7b-trace, 32b: the other workloads, one line each; rirulix, labolix, mozutar, fatilix, mezinex: "
-                         "that design at a few layer sizes beside the Qwen2.5-VL decoder of equal size")
+                         "that design at a few layer sizes beside the Qwen2.5-VL decoder of equal size; sudilorn: beside the Mozutar design")
     args = ap.parse_args(argv)
     if args.gpus != 1:
         print(f"bench.py: this engine runs on one GPU; --gpus {args.gpus} is not measured")
@@ -683,7 +720,7 @@ def main(argv=None):
             print(json.dumps({"impl": "reference", "unavailable": "the reference arm measures the 3b configuration only"}))
             return 0
         return run_reference(args)
-    return {"3b": run_ours, "7b-trace": run_7b_trace, "32b": run_32b, "rirulix": run_rirulix, "labolix": run_labolix, "mozutar": run_mozutar, "fatilix": run_fatilix, "mezinex": run_mezinex}[args.config](args)
+    return {"3b": run_ours, "7b-trace": run_7b_trace, "32b": run_32b, "rirulix": run_rirulix, "labolix": run_labolix, "mozutar": run_mozutar, "fatilix": run_fatilix, "mezinex": run_mezinex, "sudilorn": run_sudilorn}[args.config](args)
 
 
 if __name__ == "__main__":
