@@ -7,7 +7,7 @@ every constant that may differ between models of the design is read from the fil
 
     {"architecture": "Sudilorn", "vocab": V, "width": W, "norm": {"eps": e}, "residual_mult": m,
      "layers": [{"type": "attention",
-                 "mixer": {"heads", "kv_heads", "dim", "vdim", "conv", "diff", "scale", "mask": {"size"} | absent, "rot": ROT},
+                 "mixer": {"heads", "kv_heads", "dim", "vdim", "conv" | absent, "diff", "scale", "mask": {"size"} | absent, "rot": ROT},
                  "mlp": {"kind": "moe", "expert": {"ff"}, "router": {"experts", "top", "groups": {"count", "keep"}}} | null},
                 {"type": "parallel",
                  "mixer": {"left": {"heads", "kv_heads", "dim", "vdim", "scale", "mask": {"size", "keep_first"} | absent, "rot": ROT},
@@ -45,7 +45,7 @@ class SoftmaxMixerConfig:
     window: Optional[int]
     keep_first: int
     rot: Optional[SudilornRotary]
-    conv: int = 1               # the differential attention's convolution and constant
+    conv: int = 0               # the differential attention's convolution (0: none) and constant
     diff: float = 0.0
 
 
@@ -90,9 +90,9 @@ def _heads(m: Dict[str, Any], where: str) -> Tuple[int, int]:
     return heads, kv
 
 
-def _taps(m: Dict[str, Any], where: str) -> int:
-    taps = int(_need(m, "conv", where))
-    if not 1 <= taps <= 16:
+def _taps(m: Dict[str, Any], where: str, optional: bool = False) -> int:
+    taps = int(m.get("conv") or 0) if optional else int(_need(m, "conv", where))
+    if not (0 if optional else 1) <= taps <= 16:
         raise ConfigError(f"config.json: {where}.conv takes 1 to 16 taps, got {taps}")
     return taps
 
@@ -121,7 +121,7 @@ def _softmax(m: Dict[str, Any], where: str, differential: bool) -> SoftmaxMixerC
         raise ConfigError(f"config.json: {where}.mask.keep_first must not be negative, got {keep}")
     return SoftmaxMixerConfig(heads=heads, kv_heads=kv, dim=dim, vdim=int(m["vdim"]) if m.get("vdim") else dim, scale=float(_need(m, "scale", where)),
                               window=window, keep_first=keep if window else 0, rot=_rotary(m.get("rot"), dim, where + ".rot"),
-                              conv=_taps(m, where) if differential else 1, diff=float(_need(m, "diff", where)) if differential else 0.0)
+                              conv=_taps(m, where, optional=True) if differential else 0, diff=float(_need(m, "diff", where)) if differential else 0.0)
 
 
 def _delta(m: Dict[str, Any], where: str) -> DeltaMixerConfig:

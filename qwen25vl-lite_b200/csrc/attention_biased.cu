@@ -37,7 +37,7 @@ __global__ void biased_attention_generic_kernel(
   pdl_wait();
   extern __shared__ __align__(16) unsigned char att_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const size_t per_warp = (size_t)(dk + 32) * sizeof(float) + 32 * sizeof(size_t);
+  const size_t per_warp = (size_t)((dk + 33) & ~1) * sizeof(float) + 32 * sizeof(size_t);      // an even count: the next warp's offsets are whole
   unsigned char* base = att_smem + warp * per_warp;
   size_t* voff = reinterpret_cast<size_t*>(base);
   float* qs = reinterpret_cast<float*>(base + 32 * sizeof(size_t));
@@ -164,7 +164,7 @@ static int biased_attention_generic(const void* qkv, int qkv_stride, void* out, 
     return (int)cudaErrorInvalidValue;
   const long long items = (long long)n_tokens * nq;
   const unsigned blocks = (unsigned)((items + BATT_WARPS - 1) / BATT_WARPS);
-  const size_t smem = BATT_WARPS * ((size_t)(dk + 32) * sizeof(float) + 32 * sizeof(size_t));
+  const size_t smem = BATT_WARPS * ((size_t)((dk + 33) & ~1) * sizeof(float) + 32 * sizeof(size_t));
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(biased_attention_generic_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;

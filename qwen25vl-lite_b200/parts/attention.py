@@ -383,7 +383,7 @@ class DifferentialAttention(Mixer):
 
     then each head's o is divided by its root mean square (no weight) and multiplied by ``1 - diff``.  Query head h reads
     key/value head ``h // (num_heads / num_kv_heads)``; a query or key head has 2 * ``head_dim`` channels, map 1 then map 2, a
-    value ``value_dim``.  ``conv``: a causal convolution of that many taps over time on every channel of q, k and v, right
+    value ``value_dim``.  ``conv``: a causal convolution of that many taps (0: none) over time on every channel of q, k and v, right
     behind the projections (tensors ``q.conv``, ``k.conv``, ``v.conv``, no bias); its last inputs are per-request state.
     Then query/key norm per head and map (weights ``q.norm``, ``k.norm`` of ``head_dim`` numbers shared by heads and maps) and
     the layer's rotation.  A sliding ``window`` (None: causal).  The concatenated heads are multiplied channel by channel
@@ -400,7 +400,7 @@ class DifferentialAttention(Mixer):
     accepts_deferred_norm = True     # one product reads the mixer's input
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, scale: float, diff: float, norm_eps: float,
-                 window: Optional[int] = None, conv: int = 1, position=None):
+                 window: Optional[int] = None, conv: int = 0, position=None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot share {num_kv_heads} kv heads")
         self.hidden_size, self.num_heads, self.num_kv_heads = int(hidden_size), int(num_heads), int(num_kv_heads)
@@ -408,8 +408,8 @@ class DifferentialAttention(Mixer):
         if not 0 < self.value_dim <= 512 or self.head_dim <= 0:
             raise ValueError(f"key size {head_dim} / value size {value_dim} is not supported: values take up to 512 channels")
         self.window, self.conv = None if not window else int(window), int(conv)
-        if not 1 <= self.conv <= 16:
-            raise ValueError(f"the convolution takes 1 to 16 taps, got {conv}")
+        if not 0 <= self.conv <= 16:
+            raise ValueError(f"the convolution takes 1 to 16 taps (0: there is none), got {conv}")
         self.position = position if getattr(position, "dims", 0) > 0 else None
         if self.position is not None and position.dims > self.head_dim:
             raise ValueError(f"the position encoding turns {position.dims} channels, a map of a head has {head_dim}")
@@ -421,7 +421,8 @@ class DifferentialAttention(Mixer):
         h, D = self.hidden_size, self.head_dim
         q, k, v, o = 2 * self.num_heads * D, 2 * self.num_kv_heads * D, self.num_kv_heads * self.value_dim, self.num_heads * self.value_dim
         specs = [TensorSpec("q", (q, h)), TensorSpec("k", (k, h)), TensorSpec("v", (v, h)), TensorSpec("q.norm", (D,), "norm"), TensorSpec("k.norm", (D,), "norm")]
-        specs += [TensorSpec(f"{n}.conv", (rows, self.conv), "matrix_wide", optional=self.conv == 1) for n, rows in (("q", q), ("k", k), ("v", v))]
+        if self.conv:
+            specs += [TensorSpec(f"{n}.conv", (rows, self.conv), "matrix_wide") for n, rows in (("q", q), ("k", k), ("v", v))]
         specs += [TensorSpec(n, (D,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")]
         return tuple(specs + [TensorSpec("g", (o, h)), TensorSpec("o", (h, o))])
 
@@ -440,7 +441,7 @@ class DifferentialAttention(Mixer):
         f32 = lambda t: t.to(device=device, dtype=torch.float32).contiguous()
         self.q_norm, self.k_norm = f32(tensors["q.norm"]), f32(tensors["k.norm"])
         self.conv_w = None
-        if "q.conv" in tensors:
+        if self.conv:
             self.conv_w = f32(torch.cat([by_map(tensors["q.conv"]), tensors["k.conv"], tensors["v.conv"]], dim=0).t())        # [taps, channels]
             self.conv_b = torch.zeros(self.channels, dtype=torch.float32, device=device)
             self.no_state = torch.zeros((1, 0), dtype=torch.float32, device=device)             # what one tap carries from step to step
