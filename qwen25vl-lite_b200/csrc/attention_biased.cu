@@ -349,6 +349,79 @@ __global__ void qk_norm_store_flat_kernel(T* __restrict__ qk, int qk_stride, con
   }
 }
 
+// The same for heads of up to 128 channels that come in fours and are turned: 2 ^ log_lanes lanes a head (several heads to a
+// warp), four neighbouring channels a lane, in registers.  In halves a channel's partner lies half / 4 lanes on.
+template <typename T>
+__global__ void __launch_bounds__(256)
+qk_norm_store_turned_kernel(T* __restrict__ qk, int qk_stride, const float* __restrict__ wq, const float* __restrict__ wk, float eps, int unit_norm,
+                            const float* __restrict__ angles, int half, int layout, const int* __restrict__ positions, float temp_coef, int temp_every,
+                            T* __restrict__ kpages, T* __restrict__ vpages, const int* __restrict__ kv_slot, int n_tokens, int nq, int nkv, int dk, int dv,
+                            int page_size, int keys_as_values, int pack, int log_lanes) {
+  pdl_trigger();
+  pdl_wait();
+  typedef typename Raw4<T>::type R4;
+  const int lanes = 1 << log_lanes, lane = threadIdx.x & (lanes - 1);
+  const int kvs = nkv / pack, v_heads = dv > 0 && !keys_as_values ? kvs : 0, heads = nq + nkv + v_heads;
+  const long long item = ((long long)blockIdx.x * 256 + threadIdx.x) >> log_lanes;
+  const bool real = item < (long long)n_tokens * heads;       // every lane stays for the shuffles
+  const int n = real ? (int)(item / heads) : 0, head = real ? (int)(item % heads) : 0;
+  const int slot = kv_slot ? kv_slot[n] : -1;
+  const int page = slot / page_size, in_page = slot % page_size;
+  T* row = qk + (size_t)n * qk_stride;
+  const bool is_value = head >= nq + nkv, is_key = head >= nq && !is_value, turned = real && !is_value;
+  if (real && is_value && slot >= 0) {
+    const int vh = head - nq - nkv;
+    const T* src = row + (size_t)(nq + nkv) * dk + (size_t)vh * dv;
+    T* dst = vpages + (((size_t)page * kvs + vh) * page_size + in_page) * dv;
+    for (int c = lane * 4; c < dv; c += lanes * 4) *reinterpret_cast<R4*>(dst + c) = *reinterpret_cast<const R4*>(src + c);
+  }
+  T* src = row + (size_t)(turned ? head : 0) * dk;
+  const int c = lane * 4;
+  const bool in = turned && c < dk;
+  R4 raw = {};
+  if (in) raw = *reinterpret_cast<const R4*>(src + c);
+  float4 v = raw4_f32(raw);
+  float sq = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+  for (int o = lanes >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+  const float* w = is_key ? wk : wq;
+  if (w || unit_norm) {
+    const float inv = 1.0f / sqrtf(sq / (float)dk + eps);
+    v.x *= inv; v.y *= inv; v.z *= inv; v.w *= inv;
+    if (w && in) { const float4 ww = *reinterpret_cast<const float4*>(w + c); v.x *= ww.x; v.y *= ww.y; v.z *= ww.z; v.w *= ww.w; }
+  }
+  const float* ang = angles + (size_t)n * half * 2;
+  if (layout == ROTARY_INTERLEAVED) {
+    if (c < 2 * half) {
+      const float4 a = *reinterpret_cast<const float4*>(ang + c);                  // (cos, sin) of two pairs
+      v = make_float4(fmaf(v.x, a.x, -v.y * a.y), fmaf(v.y, a.x, v.x * a.y), fmaf(v.z, a.z, -v.w * a.w), fmaf(v.w, a.z, v.z * a.w));
+    }
+  } else {
+    const bool second = c >= half && c < 2 * half, first = c < half;
+    const int step = half >> 2, other = (threadIdx.x & 31) + (first ? step : second ? -step : 0);
+    const float4 u = make_float4(__shfl_sync(0xffffffffu, v.x, other), __shfl_sync(0xffffffffu, v.y, other), __shfl_sync(0xffffffffu, v.z, other),
+                                 __shfl_sync(0xffffffffu, v.w, other));
+    if (first || second) {
+      const float4 a = *reinterpret_cast<const float4*>(ang + 2 * (second ? c - half : c)), b = *reinterpret_cast<const float4*>(ang + 2 * (second ? c - half : c) + 4);
+      const float s = second ? 1.f : -1.f;
+      v = make_float4(fmaf(v.x, a.x, s * u.x * a.y), fmaf(v.y, a.z, s * u.y * a.w), fmaf(v.z, b.x, s * u.z * b.y), fmaf(v.w, b.z, s * u.w * b.w));
+    }
+  }
+  if (!in || (is_key && slot < 0)) return;
+  if (is_key) {
+    const size_t page_row = ((size_t)page * kvs + (head - nq) / pack) * page_size + in_page;
+    if (keys_as_values) *reinterpret_cast<R4*>(vpages + page_row * dk + c) = raw;
+    f32_raw4(v, raw);
+    *reinterpret_cast<R4*>(kpages + (page_row * pack + (head - nq) % pack) * dk + c) = raw;
+  } else {
+    if (temp_every > 0) {
+      const float temper = 1.0f + temp_coef * logf((float)((positions[n] + 1) / temp_every) + 1.0f);
+      v.x *= temper; v.y *= temper; v.z *= temper; v.w *= temper;
+    }
+    f32_raw4(v, raw);
+    *reinterpret_cast<R4*>(src + c) = raw;
+  }
+}
+
 template <typename T>
 static int qk_norm_store(void* qk, int qk_stride, const float* wq, const float* wk, float eps, int unit_norm, const float* angles, int half,
                          int layout, const int* positions, float temp_coef, int temp_every, void* kpages, void* vpages, const int* kv_slot,
@@ -366,6 +439,16 @@ static int qk_norm_store(void* qk, int qk_stride, const float* wq, const float* 
     const unsigned blocks = (unsigned)(((long long)n_tokens * heads + 7) / 8);
     launch(qk_norm_store_flat_kernel<T>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (T*)qk, qk_stride, wq, wk, eps, unit_norm, positions,
            temp_coef, temp_every, (T*)kpages, (T*)vpages, kv_slot, n_tokens, nq, nkv, dk, dv, page_size, keys_as_values, pack);
+    return launch_status();
+  }
+  if (half > 0 && dk % chunk == 0 && dk <= 128 && (layout == ROTARY_INTERLEAVED ? half % 2 == 0 : half % 4 == 0) && qk_stride % chunk == 0 && aligned &&
+      !((uintptr_t)angles & 15) && (keys_as_values || dv % chunk == 0)) {
+    int log_lanes = 0;
+    while ((4 << log_lanes) < dk) ++log_lanes;
+    const long long heads = nq + nkv + (dv > 0 && !keys_as_values ? nkv / pack : 0);
+    const unsigned blocks = (unsigned)((((long long)n_tokens * heads << log_lanes) + 255) / 256);
+    launch(qk_norm_store_turned_kernel<T>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (T*)qk, qk_stride, wq, wk, eps, unit_norm, angles, half, layout,
+           positions, temp_coef, temp_every, (T*)kpages, (T*)vpages, kv_slot, n_tokens, nq, nkv, dk, dv, page_size, keys_as_values, pack, log_lanes);
     return launch_status();
   }
   // as many blocks a token as its heads fill: a warp that walks several heads one after the other waits for each one's loads

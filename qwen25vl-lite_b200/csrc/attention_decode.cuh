@@ -34,6 +34,8 @@ struct AttnArgs {
   // (nullptr: none); only the tcgen05 prefill kernel's build for it reads it
   const float* dist_bias;
   int dist_rows;
+  // beside a window: first tokens that stay visible; values between the results of two tokens (the tcgen05 kernel again)
+  int keep_first, out_stride;
 };
 
 // Row pitch of a key/value tile in shared memory: D bf16 plus 16 bytes, an odd number of 16-byte
@@ -656,6 +658,6 @@ static int fill_args(AttnArgs& a, const void* qkv, int qkv_stride, void* out, co
   a.vpages = (const bf16*)vp; a.block_table = bt; a.table_width = tw; a.cu_q = cu_q; a.q_start_pos = q_start;
   a.items = items; a.nq = nq; a.nkv = nkv; a.page_shift = shift; a.window = window;
   a.scale_log2 = scale * 1.4426950408889634f; a.n_splits = 1; a.part_o = nullptr; a.part_ml = nullptr;
-  a.sink = nullptr; a.gate_off = -1; a.dist_bias = nullptr; a.dist_rows = 1;
+  a.sink = nullptr; a.gate_off = -1; a.dist_bias = nullptr; a.dist_rows = 1; a.keep_first = 0; a.out_stride = 0;
   return 0;
 }

@@ -4,7 +4,15 @@
 // 156-175, src/qwen25vl_lite/attention.py:143-148): S = Q K^T * D^-1/2, a query at position a sees
 // keys j <= a (and j > a - window), softmax over the keys in float, O = P V.  Two things more for models that have
 // them, both where a row's sums become its result: a sink per query head (a score without key or value that joins
-// the denominator) and an output gate (the result times the sigmoid of the row's gate channels).
+// the denominator) and an output gate (the result times the sigmoid of the row's gate channels).  Beside a window the
+// first keep_first tokens may stay visible (a build of its own, KEEP): a CTA whose window has left them behind walks their
+// tiles first, counting keys below keep_first alone there, then the window's.
+//
+// Differential attention (a build of its own, DIFF) for maps of 64 channels over values of 128: a key row holds both maps'
+// keys, a row of queries 64 channels of its map and zeros in place of the other's, so the products are those of plain
+// attention over rows of 128; the rows of a token are (map, head of the group), and when all keys are done the rows of the
+// second map go through shared memory to those of the first, which form a1 - lam a2, divide by its root mean square (a
+// thread has its whole row) and multiply by gain and the gate.
 //
 // A CTA takes 128 rows = (token, query head of one kv group) pairs of one entry, so one pass over a
 // kv head's keys serves the whole group, and walks the keys in tiles of 64.  Its threads have two
@@ -144,8 +152,14 @@ __device__ __forceinline__ void a5_gate32(float (&v)[32], const bf16* g) {
 // kernel carries none of it.  A row whose nearest key of a tile lies at the table's last row or beyond adds that row's
 // number to all its scores of the tile (into the exponent's offset, at no cost per score); in the two or three tiles at
 // the diagonal every score looks its distance up.
-template <bool TABLE>
-__global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kernel(AttnArgs a, int n_sms, int* __restrict__ err) {
+struct A5Diff {
+  const bf16* gate;         // [N, gate_stride]: nq / 2 heads of D channels
+  int gate_stride;
+  float lam, gain, eps;
+};
+
+template <bool TABLE, bool KEEP, bool DIFF>
+__global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kernel(AttnArgs a, A5Diff df, int n_sms, int* __restrict__ err) {
   constexpr int NROW = A5_NROW, ROWS = A5_ROWS;         // one thread per row; the warp after them issues the products
   constexpr int TMEM_COLS = 256, O_COL = 128;           // two score buffers of 64 columns, then the outputs
   pdl_trigger();
@@ -188,8 +202,11 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
   const int c_first = R0 / G, c_last = min(R0 + ROWS - 1, n_rows - 1) / G;
   int c_hi = start + c_last;                               // the last key anybody of the CTA sees: nothing is loaded past it
   const int c_lo = a.window > 0 ? max(0, start + c_first - a.window + 1) : 0;
-  int key_begin = c_lo & ~(A5_BN - 1);
-  int n_tiles = (c_hi - key_begin) / A5_BN + 1;
+  // kept first tokens that the window of every row has left behind: tiles of their own, in front; else one range
+  const int kept = KEEP && c_lo > a.keep_first ? a.keep_first : 0;
+  const int kept_tiles = KEEP ? (kept + A5_BN - 1) / A5_BN : 0;
+  int key_begin = (KEEP && c_lo <= a.keep_first ? 0 : c_lo) & ~(A5_BN - 1);
+  int n_tiles = kept_tiles + (c_hi - key_begin) / A5_BN + 1;
   if (n_parts > 1) {                                       // this CTA's part of the key tiles
     const int per = (n_tiles + n_parts - 1) / n_parts;
     const int t0 = part * per, t1 = min(n_tiles, t0 + per);
@@ -235,12 +252,13 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
   constexpr int N_COPIES = A5_BN * 16 / NROW;
   const int lane = tid & 31;
   const bool blocks = a.page_shift >= 4;
-  const int block_key = key_begin + 16 * (warp & 3);                          // first key of this warp's block in tile 0
+  auto tile_key = [&](int t) { return KEEP && t < kept_tiles ? t * A5_BN : key_begin + (t - kept_tiles) * A5_BN; };      // first key of a tile
+  const int block_off = 16 * (warp & 3);                                      // this warp's block in a tile
   auto block_row = [&](int page, int kfirst) { return ((page * a.nkv + kvh) << a.page_shift) + (kfirst & ((1 << a.page_shift) - 1)); };
   auto block_valid = [&](int kfirst) { return min(max(c_hi - kfirst + 1, 0), 16); };
   int rb0 = 0, rb1 = 0, rb2 = 0;
   if (blocks && tid < NROW) {
-    const int k0 = block_key, k1 = block_key + A5_BN, k2 = block_key + 2 * A5_BN;
+    const int k0 = tile_key(0) + block_off, k1 = tile_key(1) + block_off, k2 = tile_key(2) + block_off;
     const int p0 = k0 <= c_hi ? __ldg(table + (k0 >> a.page_shift)) : 0;
     const int p1 = k1 <= c_hi ? __ldg(table + (k1 >> a.page_shift)) : 0;
     const int p2 = k2 <= c_hi ? __ldg(table + (k2 >> a.page_shift)) : 0;
@@ -253,7 +271,7 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
   if (looks_up) {
 #pragma unroll
     for (int j = 0; j < 3; ++j)
-      if (j < n_tiles) key_rows[j * A5_BN + my_key] = a5_key_row(a, table, kvh, key_begin + j * A5_BN + my_key, c_hi);
+      if (j < n_tiles) key_rows[j * A5_BN + my_key] = a5_key_row(a, table, kvh, tile_key(j) + my_key, c_hi);
   }
   __syncwarp();
   // Up to here the kernel has read the step's work list, lengths and block tables only, which came
@@ -265,19 +283,21 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
   // nothing of its own is in flight.
   if (tid < NROW) {
     if (blocks) {
-      a5_load_block(k_s, a.kpages, rb0, block_valid(block_key), warp, lane);
-      if (n_tiles > 1) a5_load_block(k_s + A5_KV_BYTES, a.kpages, rb1, block_valid(block_key + A5_BN), warp, lane);
-      a5_load_block(v_s, a.vpages, rb0, block_valid(block_key), warp, lane);
+      a5_load_block(k_s, a.kpages, rb0, block_valid(tile_key(0) + block_off), warp, lane);
+      if (n_tiles > 1) a5_load_block(k_s + A5_KV_BYTES, a.kpages, rb1, block_valid(tile_key(1) + block_off), warp, lane);
+      a5_load_block(v_s, a.vpages, rb0, block_valid(tile_key(0) + block_off), warp, lane);
     } else {
       a5_load_tile(k_s, a.kpages, key_rows, tid);
       if (n_tiles > 1) a5_load_tile(k_s + A5_KV_BYTES, a.kpages, key_rows + A5_BN, tid);
       a5_load_tile(v_s, a.vpages, key_rows, tid);
     }
     cp_async_commit();
-    const uint4* src = reinterpret_cast<const uint4*>(a.qkv + (size_t)(q0 + tok) * a.qkv_stride + (size_t)(kvh * G + head) * A5_D);
+    const int map = DIFF && head >= (G >> 1) ? 1 : 0;
+    const uint4* src = reinterpret_cast<const uint4*>(a.qkv + (size_t)(q0 + tok) * a.qkv_stride + (size_t)(kvh * G + head) * (DIFF ? A5_D / 2 : A5_D));
 #pragma unroll
     for (int cc = 0; cc < 16; ++cc) {
-      const uint4 v = live ? __ldcg(src + cc) : make_uint4(0, 0, 0, 0);
+      const bool mine = live && (!DIFF || (cc >> 3) == map);             // a map's channels, zeros in place of the other's
+      const uint4 v = mine ? __ldcg(src + (DIFF ? cc & 7 : cc)) : make_uint4(0, 0, 0, 0);
       *reinterpret_cast<uint4*>(q_s + (cc >> 3) * (A5_ROWS * 128) + a5_swz(tid, cc & 7)) = v;
     }
     cp_async_wait<0>();
@@ -346,7 +366,7 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
 
     for (int tile = 0; tile < n_tiles; ++tile) {
       const int stage = tile & 1;
-      const int key0 = key_begin + tile * A5_BN;
+      const int key0 = tile_key(tile);
       if (ok && !mbar_wait(bars->s_full + stage, (unsigned)(tile >> 1) & 1)) {
         ok = false;
         atomicExch(err, 24);
@@ -354,20 +374,20 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
       tc5_fence_after();
       // K(t + 2) goes where K(t) was, which the scores are done with; V(t) where V(t - 2) was, whose
       // product was done before the scores of this tile were asked for
-      const int kb = block_key + tile * A5_BN;             // this warp's block in this tile
+      const int kb = key0 + block_off, kb2 = tile_key(tile + 2) + block_off, kb3 = tile_key(tile + 3) + block_off;      // this warp's block in this tile and further on
       int row_ahead = -1, page_ahead = 0;                  // asked for now, used when the tile ends
       if (blocks) {
         if (tile + 2 < n_tiles)
-          a5_load_block(k_s + (size_t)stage * A5_KV_BYTES, a.kpages, rb2, block_valid(kb + 2 * A5_BN), warp, lane);
+          a5_load_block(k_s + (size_t)stage * A5_KV_BYTES, a.kpages, rb2, block_valid(kb2), warp, lane);
         if (tile > 0) a5_load_block(v_s + (size_t)stage * A5_KV_BYTES, a.vpages, rb0, block_valid(kb), warp, lane);
         cp_async_commit();
-        if (kb + 3 * A5_BN <= c_hi) page_ahead = __ldg(table + ((kb + 3 * A5_BN) >> a.page_shift));
+        if (kb3 <= c_hi) page_ahead = __ldg(table + (kb3 >> a.page_shift));
       } else {
         if (tile + 2 < n_tiles)
           a5_load_tile(k_s + (size_t)stage * A5_KV_BYTES, a.kpages, key_rows + ((tile + 2) & 3) * A5_BN, tid);
         if (tile > 0) a5_load_tile(v_s + (size_t)stage * A5_KV_BYTES, a.vpages, key_rows + (tile & 3) * A5_BN, tid);
         cp_async_commit();
-        if (looks_up && tile + 3 < n_tiles) row_ahead = a5_key_row(a, table, kvh, key0 + 3 * A5_BN + my_key, c_hi);
+        if (looks_up && tile + 3 < n_tiles) row_ahead = a5_key_row(a, table, kvh, tile_key(tile + 3) + my_key, c_hi);
       }
 
       // this row's 64 scores
@@ -382,11 +402,16 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
         for (int j = 0; j < 32; ++j) s[32 + j] = part[j];
       }
       const bool need_mask = !all_live || key0 + A5_BN - 1 > min_hi || key0 < max_lo;      // the same for the whole CTA
-      if (need_mask) {
+      if (KEEP && tile < kept_tiles) {
+        const int end = live ? kept - key0 : 0;            // of the tile's keys, those that are kept (every row's window is past them)
+#pragma unroll
+        for (int j = 0; j < A5_BN; ++j) s[j] = j < end ? s[j] : -INFINITY;
+      } else if (need_mask) {
+        const int keep_end = KEEP && kept_tiles == 0 ? a.keep_first : 0;
 #pragma unroll
         for (int j = 0; j < A5_BN; ++j) {
           const int kidx = key0 + j;
-          s[j] = (kidx >= lo && kidx <= hi) ? s[j] : -INFINITY;
+          s[j] = ((kidx >= lo || (KEEP && kidx < keep_end)) && kidx <= hi) ? s[j] : -INFINITY;
         }
       }
       float sc = a.scale_log2, add = 0.f;                  // a score enters the exponent as s * sc + add
@@ -446,7 +471,7 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
       if (blocks) {
         rb0 = rb1;
         rb1 = rb2;
-        rb2 = kb + 3 * A5_BN <= c_hi ? block_row(page_ahead, kb + 3 * A5_BN) : 0;
+        rb2 = kb3 <= c_hi ? block_row(page_ahead, kb3) : 0;
       } else {
         if (looks_up && tile + 3 < n_tiles) key_rows[((tile + 3) & 3) * A5_BN + my_key] = row_ahead;
         __syncwarp();
@@ -466,7 +491,66 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
   }
 
   // ---- the results ----
-  if (pair && n_parts > 1) {
+  if (DIFF) {
+    // 128 rows are whole tokens: a row of the second map leaves its result in shared memory (the K and V tiles are done with:
+    // value quads of all rows side by side), its partner of the first map, G / 2 rows before it, finishes the head
+    if (tid < NROW) {
+      const int half = G >> 1;
+      const bool second = live && head >= half, firsts = live && head < half;
+      const float inv = live && l > 0.f ? 1.0f / l : 0.f;
+#pragma unroll
+      for (int c = 0; c < A5_D / 32; ++c) {
+        float part[32];
+        tc5_ld32(t_o + c * 32, part);
+        if (!second) continue;
+#pragma unroll
+        for (int q = 0; q < 8; ++q)
+          *reinterpret_cast<float4*>(k_s + (size_t)((c * 8 + q) * NROW + tid) * 16) =
+              make_float4(part[q * 4] * inv, part[q * 4 + 1] * inv, part[q * 4 + 2] * inv, part[q * 4 + 3] * inv);
+      }
+      asm volatile("bar.sync 1, 128;\n" ::: "memory");
+      const int partner = min(tid + half, NROW - 1);
+      auto combine = [&](int c, float (&part)[32]) {      // 32 channels of a1 - lam a2
+        tc5_ld32(t_o + c * 32, part);
+#pragma unroll
+        for (int q = 0; q < 8; ++q) {
+          const float4 b = *reinterpret_cast<const float4*>(k_s + (size_t)((c * 8 + q) * NROW + partner) * 16);
+          part[q * 4] = fmaf(-df.lam, b.x, part[q * 4] * inv); part[q * 4 + 1] = fmaf(-df.lam, b.y, part[q * 4 + 1] * inv);
+          part[q * 4 + 2] = fmaf(-df.lam, b.z, part[q * 4 + 2] * inv); part[q * 4 + 3] = fmaf(-df.lam, b.w, part[q * 4 + 3] * inv);
+        }
+      };
+      float sq = 0.f;
+#pragma unroll
+      for (int c = 0; c < A5_D / 32; ++c) {
+        float part[32];
+        combine(c, part);
+#pragma unroll
+        for (int j = 0; j < 32; ++j) sq = fmaf(part[j], part[j], sq);
+      }
+      const float f = df.gain / sqrtf(sq / (float)A5_D + df.eps);
+      const size_t channel = (size_t)(kvh * half + (firsts ? head : 0)) * A5_D;
+      bf16* dst = a.out + (size_t)(q0 + tok) * a.out_stride + channel;
+      const bf16* gate = df.gate + (size_t)(q0 + tok) * df.gate_stride + channel;
+#pragma unroll
+      for (int c = 0; c < A5_D / 32; ++c) {
+        float part[32];
+        combine(c, part);
+        if (!firsts) continue;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) part[j] *= f;
+        a5_gate32(part, gate + c * 32);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          uint4 o;
+          o.x = pack_bf16(part[q * 8], part[q * 8 + 1]);
+          o.y = pack_bf16(part[q * 8 + 2], part[q * 8 + 3]);
+          o.z = pack_bf16(part[q * 8 + 4], part[q * 8 + 5]);
+          o.w = pack_bf16(part[q * 8 + 6], part[q * 8 + 7]);
+          *reinterpret_cast<uint4*>(dst + c * 32 + q * 8) = o;
+        }
+      }
+    }
+  } else if (pair && n_parts > 1) {
     // Two CTAs of a cluster with half of the keys each.  The second leaves its rows as they are, with
     // their maxima and sums, in its own shared memory (the K and V tiles are done with: 64 KB, value
     // quads of all rows side by side; maxima and sums where Q was); the first adds them to its own:
@@ -493,7 +577,7 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
       const float L = l * w0 + l1 * w1 + (live ? a5_sink_weight(a, kvh * G + head, M) : 0.f);
       const float inv = live && L > 0.f ? 1.0f / L : 0.f;
       const float s0 = w0 * inv, s1 = w1 * inv;
-      bf16* dst = a.out + (size_t)(q0 + tok) * a.nq * A5_D + (size_t)(kvh * G + head) * A5_D;
+      bf16* dst = a.out + (size_t)(q0 + tok) * a.out_stride + (size_t)(kvh * G + head) * A5_D;
       const bf16* gate = a.gate_off >= 0 && live ? a.qkv + (size_t)(q0 + tok) * a.qkv_stride + a.gate_off + (size_t)(kvh * G + head) * A5_D : nullptr;
 #pragma unroll
       for (int c = 0; c < A5_D / 32; ++c) {
@@ -539,7 +623,7 @@ __global__ void __launch_bounds__(A5_THREADS, 2) attention_prefill_tcgen05_kerne
     } else {
     const float l_all = l + (live ? a5_sink_weight(a, kvh * G + head, m_used) : 0.f);
     const float inv = live && l_all > 0.f ? 1.0f / l_all : 0.f;
-    bf16* dst = a.out + (size_t)(q0 + tok) * a.nq * A5_D + (size_t)(kvh * G + head) * A5_D;
+    bf16* dst = a.out + (size_t)(q0 + tok) * a.out_stride + (size_t)(kvh * G + head) * A5_D;
     const bf16* gate = a.gate_off >= 0 && live ? a.qkv + (size_t)(q0 + tok) * a.qkv_stride + a.gate_off + (size_t)(kvh * G + head) * A5_D : nullptr;
 #pragma unroll
     for (int c = 0; c < A5_D / 32; ++c) {                 // tcgen05.ld is warp-wide: dead rows read too, and store nothing
@@ -627,7 +711,7 @@ __global__ void __launch_bounds__(A5_MERGE_WARPS * 32, 4) attention_prefill_merg
   uint2 packed;
   packed.x = pack_bf16(acc.x, acc.y);
   packed.y = pack_bf16(acc.z, acc.w);
-  *reinterpret_cast<uint2*>(a.out + (size_t)(q0 + tok) * a.nq * A5_D + (size_t)(kvh * G + head) * A5_D + lane * 4) = packed;
+  *reinterpret_cast<uint2*>(a.out + (size_t)(q0 + tok) * a.out_stride + (size_t)(kvh * G + head) * A5_D + lane * 4) = packed;
 }
 
 // tiles: (entry, row tile, code) triples with row tiles of 128 rows (code 1: the whole tile; else
@@ -635,23 +719,27 @@ __global__ void __launch_bounds__(A5_MERGE_WARPS * 32, 4) attention_prefill_merg
 // first part, parts) of the n_merges tiles that were cut, scratch: n_tiles * nkv * 128 * (D + 2)
 // floats when there are any.  pairs != 0: every piece of work goes to a cluster of two CTAs, and the
 // codes are 1 (the whole tile, one CTA) or 2 (half of the keys each).  Otherwise the arguments of
-// q25_attention_prefill_bf16.  Head size 128 only.  err: one int that receives a nonzero code if a
+// q25_attention_prefill_bf16.  keep: first tokens that stay visible beside a window; out_stride: values between the results
+// of two tokens.  Head size 128 only.  err: one int that receives a nonzero code if a
 // wait gave up.
 Q25_EXPORT int q25_attention_prefill_tcgen05_bf16(const void* qkv, int qkv_stride, void* out, const void* kp, const void* vp,
                                                   const int* bt, int tw, const int* cu_q, const int* q_start,
                                                   const int* tiles, int n_tiles, int nq, int nkv, int d, int page_size,
                                                   int window, float scale, const int* merges, int n_merges, float* scratch,
                                                   int pairs, const float* sink, int gate_off, const float* dist_bias, int dist_rows,
-                                                  int* err, void* stream) {
+                                                  int keep, int out_stride, int* err, void* stream) {
   if (n_tiles <= 0) return 0;
   if (d != A5_D || !err || (n_merges > 0 && (!merges || !scratch || window > 0 || pairs)) || (pairs && window > 0) ||
-      (gate_off >= 0 && gate_off % 8) || (dist_bias && dist_rows < 1))
+      (gate_off >= 0 && gate_off % 8) || (dist_bias && dist_rows < 1) || keep < 0 || (keep > 0 && (window <= 0 || dist_bias)) || out_stride % 8)
     return (int)cudaErrorInvalidValue;
   AttnArgs a;
   int e = fill_args(a, qkv, qkv_stride, out, kp, vp, bt, tw, cu_q, q_start, tiles, nq, nkv, page_size, window, scale);
   if (e) return e;
   if (((uintptr_t)qkv & 15) || (qkv_stride % 8) || ((uintptr_t)out & 15)) return (int)cudaErrorInvalidValue;
-  void (*kernel)(AttnArgs, int, int*) = dist_bias ? attention_prefill_tcgen05_kernel<true> : attention_prefill_tcgen05_kernel<false>;
+  void (*kernel)(AttnArgs, A5Diff, int, int*) = dist_bias  ? attention_prefill_tcgen05_kernel<true, false, false>
+                                                : keep > 0 ? attention_prefill_tcgen05_kernel<false, true, false>
+                                                           : attention_prefill_tcgen05_kernel<false, false, false>;
+  a.keep_first = keep; a.out_stride = out_stride;
   cudaError_t ce = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, A5_SMEM);
   if (ce != cudaSuccess) return (int)ce;
   a.dist_bias = dist_bias; a.dist_rows = dist_bias ? dist_rows : 1;
@@ -659,9 +747,33 @@ Q25_EXPORT int q25_attention_prefill_tcgen05_bf16(const void* qkv, int qkv_strid
   a.part_o = scratch;                                    // [part, kv head, row, D], then [part, kv head, row, (m, l)]
   a.part_ml = scratch ? scratch + (size_t)n_tiles * nkv * A5_ROWS * A5_D : nullptr;
   launch_clusters(pairs ? 2 : 1, kernel, dim3(n_tiles * nkv * (pairs ? 2 : 1)), dim3(A5_THREADS),
-                  (size_t)A5_SMEM, (cudaStream_t)stream, a, device_sm_count(), err);
+                  (size_t)A5_SMEM, (cudaStream_t)stream, a, A5Diff{}, device_sm_count(), err);
   if (n_merges > 0)
     launch(attention_prefill_merge_kernel, dim3(n_merges * nkv * (A5_ROWS / A5_MERGE_WARPS)), dim3(A5_MERGE_WARPS * 32), 0,
            (cudaStream_t)stream, a, merges);
+  return launch_status();
+}
+
+// Runs of a differential attention with maps of 64 channels over values of 128: qkv rows begin with the queries by (kv head,
+// map, head of the group); key rows hold both maps, [pages, nkv, page_size, 128].  tiles: (entry, row tile of 128 rows, 1)
+// triples over the rows (token, map, head of the group); 128 must be a multiple of 2 * heads / nkv.  gate: rows of heads * 128
+// channels.
+Q25_EXPORT int q25_attention_prefill_differential_bf16(const void* qkv, int qkv_stride, const void* gate, int gate_stride, void* out, const void* kp,
+                                                       const void* vp, const int* bt, int tw, const int* cu_q, const int* q_start, const int* tiles,
+                                                       int n_tiles, int heads, int nkv, int page_size, int window, float scale, float lam, float gain,
+                                                       float eps, int* err, void* stream) {
+  if (n_tiles <= 0) return 0;
+  if (heads <= 0 || nkv <= 0 || heads % nkv || A5_ROWS % (2 * (heads / nkv)) || !err || gate_stride % 8 || qkv_stride % 8 ||
+      (((uintptr_t)qkv | (uintptr_t)gate | (uintptr_t)out) & 15))
+    return (int)cudaErrorInvalidValue;
+  AttnArgs a;
+  const int e = fill_args(a, qkv, qkv_stride, out, kp, vp, bt, tw, cu_q, q_start, tiles, 2 * heads, nkv, page_size, window, scale);
+  if (e) return e;
+  a.out_stride = heads * A5_D;
+  void (*kernel)(AttnArgs, A5Diff, int, int*) = attention_prefill_tcgen05_kernel<false, false, true>;
+  const cudaError_t ce = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, A5_SMEM);
+  if (ce != cudaSuccess) return (int)ce;
+  const A5Diff df = {(const bf16*)gate, gate_stride, lam, gain, eps};
+  launch_clusters(1, kernel, dim3(n_tiles * nkv), dim3(A5_THREADS), (size_t)A5_SMEM, (cudaStream_t)stream, a, df, device_sm_count(), err);
   return launch_status();
 }

@@ -263,17 +263,15 @@ __device__ __forceinline__ void split_store(bf16* hi, bf16* lo, float a, float b
 
 // blockIdx.x = head, blockIdx.y = chunk.
 template <int D>
-__global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, const int* __restrict__ chunks, DeltaScratch out) {
-  constexpr int DP = D + 8, LP = DL + 8, FP = DL + 4, KT = D / 16;
+__global__ void __launch_bounds__(DL_THREADS, 3) delta_prepare_kernel(DeltaArgs p, const int* __restrict__ chunks, DeltaScratch out) {
+  constexpr int DP = D + 8, LP = DL + 8, FP = DL + 8, KT = D / 16;
   extern __shared__ __align__(16) unsigned char dp_smem[];
   bf16* Ks = reinterpret_cast<bf16*>(dp_smem);               // [DL][DP]
   bf16* Qs = Ks + DL * DP;                                   // [DL][DP]; then the values, 64 columns at a time
   float* A = reinterpret_cast<float*>(Qs + DL * (DP > LP ? DP : LP));        // [DL][FP]
   float* Ti = A + DL * FP;                                   // [DL][FP]: (I + A)^-1
   float* W = Ti + DL * FP;                                   // [3][16][17]: products on the way to a block below the diagonal
-  bf16* Tv = reinterpret_cast<bf16*>(W + 3 * 16 * 17 + 12);  // [2][DL][LP]: T, rounded and the rest
-  bf16* Tk = Tv + 2 * DL * LP;                               // [2][DL][LP]: T diag(e^c / |k'|)
-  float* num = reinterpret_cast<float*>(Tk + 2 * DL * LP);   // [6][DL]: c, beta, 1 / |k'|, q_scale / |q'|, e^c / |k'|, -
+  float* num = W + 3 * 16 * 17;                              // [5][DL]: c, beta, 1 / |k'|, q_scale / |q'|, beta e^c / |k'|
   pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2;
   const int head = blockIdx.x, begin = chunks[2 * blockIdx.y], end = chunks[2 * blockIdx.y + 1], n = end - begin;
@@ -321,7 +319,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, 
     kk = warp_sum(kk); qq = warp_sum(qq);
     if (lane == 0) {
       const float ik = 1.0f / sqrtf(kk + p.unit_eps), iq = p.q_scale / sqrtf(qq + p.unit_eps), ec = expf(num[r]);
-      num[2 * DL + r] = ik; num[3 * DL + r] = iq; num[4 * DL + r] = ec * ik;
+      num[2 * DL + r] = ik; num[3 * DL + r] = iq; num[4 * DL + r] = num[DL + r] * ec * ik;
       out.row[ch * 2 * DL + r] = ec * iq;
       out.row[(ch * 2 + 1) * DL + r] = expf(num[DL - 1] - num[r]) * ik;
       if (r == 0) out.keep[ch] = expf(num[DL - 1]);
@@ -411,16 +409,21 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, 
     }
     __syncthreads();
   }
-  for (int i = tid; i < DL * DL / 2; i += DL_THREADS) {
-    const int r = i / (DL / 2), c = (i % (DL / 2)) * 2;
-    const float2 v = *reinterpret_cast<const float2*>(Ti + r * FP + c);
-    const float a = v.x * num[DL + c], b = v.y * num[DL + c + 1];
-    split_store(Tv + r * LP + c, Tv + (DL + r) * LP + c, a, b);
-    split_store(Tk + r * LP + c, Tk + (DL + r) * LP + c, a * num[4 * DL + c], b * num[4 * DL + c + 1]);
-  }
+  // a 16 x 16 block of the inverse as an operand, its columns times factor: rounded, and what that left
+  auto inverse_block = [&](int ti, int j, const float* factor, unsigned (&hi)[4], unsigned (&lo)[4]) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = ti * 16 + g + (e & 1) * 8, c = j * 16 + t2 + (e >> 1) * 8;
+      const float2 v = *reinterpret_cast<const float2*>(Ti + r * FP + c), f = *reinterpret_cast<const float2*>(factor + c);
+      const float a = v.x * f.x, b = v.y * f.y;
+      const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+      hi[e] = *reinterpret_cast<const unsigned*>(&h);
+      lo[e] = pack_bf16(a - __low2float(h), b - __high2float(h));
+    }
+  };
   cp_async_wait<0>();
   __syncthreads();
-  // Y = Tk K': a warp has 16 tokens and half of the columns
+  // Y = T diag(e^c / |k'|) K': a warp has 16 tokens and half of the columns
   const int tile = warp & 3, half = warp >> 2;
   {
     constexpr int NT = D / 16;                               // 8-column tiles of a warp
@@ -431,8 +434,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, 
       for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
     for (int j = 0; j <= tile; ++j) {
       unsigned hi[4], lo[4];
-      ldmatrix_x4(hi, Tk + (tile * 16 + (lane & 15)) * LP + j * 16 + (lane >> 4) * 8);
-      ldmatrix_x4(lo, Tk + (DL + tile * 16 + (lane & 15)) * LP + j * 16 + (lane >> 4) * 8);
+      inverse_block(tile, j, num + 4 * DL, hi, lo);
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
         unsigned b[2];
@@ -450,7 +452,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, 
         split_store(y + at, y + (size_t)DL * D + at, acc[i][2 * e], acc[i][2 * e + 1]);
       }
   }
-  // Uv = Tv V, 64 columns at a time
+  // Uv = T V, 64 columns at a time
   for (int v0 = 0; v0 < p.V; v0 += 64) {
     if (v0 > 0) {
       __syncthreads();
@@ -465,8 +467,7 @@ __global__ void __launch_bounds__(DL_THREADS) delta_prepare_kernel(DeltaArgs p, 
       for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
     for (int j = 0; j <= tile; ++j) {
       unsigned hi[4], lo[4];
-      ldmatrix_x4(hi, Tv + (tile * 16 + (lane & 15)) * LP + j * 16 + (lane >> 4) * 8);
-      ldmatrix_x4(lo, Tv + (DL + tile * 16 + (lane & 15)) * LP + j * 16 + (lane >> 4) * 8);
+      inverse_block(tile, j, num + DL, hi, lo);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         unsigned b[2];
@@ -715,8 +716,8 @@ static int delta_run_shape(const DeltaArgs& p, const int* items, int n_runs, con
 
 template <int D>
 static int delta_prepare(const DeltaArgs& p, const int* chunks, int n_chunks, const DeltaScratch& sc, cudaStream_t s) {
-  constexpr int DP = D + 8, LP = DL + 8, FP = DL + 4;
-  const size_t smem = (size_t)(DL * DP + DL * (DP > LP ? DP : LP) + 4 * DL * LP) * sizeof(bf16) + (size_t)(2 * DL * FP + 3 * 16 * 17 + 12 + 6 * DL) * sizeof(float);
+  constexpr int DP = D + 8, LP = DL + 8, FP = DL + 8;
+  const size_t smem = (size_t)(DL * DP + DL * (DP > LP ? DP : LP)) * sizeof(bf16) + (size_t)(2 * DL * FP + 3 * 16 * 17 + 5 * DL) * sizeof(float);
   const cudaError_t e = cudaFuncSetAttribute(delta_prepare_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   launch(delta_prepare_kernel<D>, dim3(p.H, n_chunks), dim3(DL_THREADS), smem, s, p, chunks, sc);

@@ -399,6 +399,32 @@ __global__ void memory_output_kernel(const float* __restrict__ o_raw, const floa
   }
 }
 
+// The same for memories without a normaliser whose heads come in fours of channels: four channels a load and a store.
+template <typename T>
+__global__ void memory_output_four_kernel(const float* __restrict__ o_raw, const T* __restrict__ x, int x_stride, int g_off, const float* __restrict__ weight,
+                                          T* __restrict__ out, int out_stride, int n_tokens, int H, int Dv, float eps, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
+  if (item >= (long long)n_tokens * H) return;
+  const int n = (int)(item / H), head = (int)(item % H);
+  const float* o = o_raw + (size_t)item * Dv;
+  float sq = 0.f;
+  for (int c = lane * 4; c < Dv; c += 128) {
+    const float4 v = *reinterpret_cast<const float4*>(o + c);
+    sq = fmaf(v.x, v.x, sq); sq = fmaf(v.y, v.y, sq); sq = fmaf(v.z, v.z, sq); sq = fmaf(v.w, v.w, sq);
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)Dv + eps);
+  const T* gate = x + (size_t)n * x_stride + g_off + head * Dv;
+  T* dst = out + (size_t)n * out_stride + (size_t)head * Dv;
+  auto gated = [&](float z) { const float s = 1.0f / (1.0f + expf(-z)); return act == 0 ? z * s : s; };
+  for (int c = lane * 4; c < Dv; c += 128) {
+    const float4 v = *reinterpret_cast<const float4*>(o + c), w = *reinterpret_cast<const float4*>(weight + head * Dv + c), z = load4<T>(gate + c);
+    store4<T>(dst + c, make_float4(v.x * inv * w.x * gated(z.x), v.y * inv * w.y * gated(z.y), v.z * inv * w.z * gated(z.z), v.w * inv * w.w * gated(z.w)));
+  }
+}
+
 template <typename T>
 static int gla_decay(const void* x, int x_stride, int low_off, int rank, const float* a2t, const float* bias, float tau, float* decay,
                      int n_tokens, int channels, void* stream) {
@@ -557,6 +583,13 @@ static int memory_output(const float* o_raw, const float* m_exp, const void* x, 
   if (n_tokens <= 0) return 0;
   if (extra && !m_exp) return (int)cudaErrorInvalidValue;
   const long long items = (long long)n_tokens * H;
+  const size_t row = 4 * sizeof(T);
+  if (!extra && Dv % 4 == 0 && x_stride % 4 == 0 && g_off % 4 == 0 && out_stride % 4 == 0 && !((uintptr_t)x % row) && !((uintptr_t)out % row) &&
+      !(((uintptr_t)o_raw | (uintptr_t)weight) & 15)) {
+    launch(memory_output_four_kernel<T>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, o_raw, (const T*)x, x_stride, g_off, weight,
+           (T*)out, out_stride, n_tokens, H, Dv, eps, act);
+    return launch_status();
+  }
   launch(memory_output_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, (cudaStream_t)stream, o_raw, m_exp, (const T*)x, x_stride,
          g_off, weight, (T*)out, out_stride, n_tokens, H, Dv, extra, eps, act);
   return launch_status();

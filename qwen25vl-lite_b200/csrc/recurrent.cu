@@ -405,11 +405,12 @@ causal_conv_kernel(const T* __restrict__ in, int in_stride, const float* __restr
   float wt[WIN][V], b[V];
   if (c < channels) {                          // weights: no kernel ever writes them
 #pragma unroll
-    for (int j = 0; j < WIN; ++j)
+    for (int j = 0; j < WIN; ++j) {
 #pragma unroll
-      for (int v = 0; v < V; ++v) wt[j][v] = j >= WIN - taps ? w[(size_t)(j - (WIN - taps)) * channels + c + v] : 0.f;
-#pragma unroll
-    for (int v = 0; v < V; ++v) b[v] = bias[c + v];
+      for (int v = 0; v < V; ++v) wt[j][v] = 0.f;
+      if (j >= WIN - taps) conv_load<float, V>(w + (size_t)(j - (WIN - taps)) * channels + c, wt[j]);
+    }
+    conv_load<float, V>(bias + c, b);
   }
   pdl_wait();
   const int seq = blockIdx.y, piece = blockIdx.z;
@@ -500,7 +501,7 @@ static int causal_conv(const void* in, int in_stride, const float* w, const floa
   if (taps < 1 || taps > RG_MAX_TAPS || max_q_len < 1 || (taps > 1 && !state)) return (int)cudaErrorInvalidValue;
   const int pieces = (max_q_len + CONV_TOKENS - 1) / CONV_TOKENS;
   if (pieces > 65535 || n_seqs > 65535) return (int)cudaErrorInvalidValue;
-  const bool four = channels % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && !((uintptr_t)in % (4 * sizeof(T))) && !((uintptr_t)out % (4 * sizeof(TO)));
+  const bool four = channels % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && !(((uintptr_t)w | (uintptr_t)bias) & 15) && !((uintptr_t)in % (4 * sizeof(T))) && !((uintptr_t)out % (4 * sizeof(TO)));
   const int threads_c = four ? channels / 4 : channels;
   const dim3 grid((threads_c + 127) / 128, n_seqs, pieces);
   void (*kernel)(const T*, int, const float*, const float*, float*, size_t, const int*, const int*, TO*, int, int, int, int) =

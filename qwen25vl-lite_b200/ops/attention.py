@@ -282,10 +282,9 @@ def paged_attention(ctx, plan, qkv, kv, nq: int, nkv: int, head_dim: int, window
 
 def tcgen05_runs(dk: int, dv: int, group: int, window, keep_first, r1, v_row, softcap) -> bool:
     """Whether the runs of an attention of this family can go to the tcgen05 prefill kernel: heads of 128 for keys and
-    values alike, every earlier key visible, and nothing between the scaled score and the softmax but a table by
-    distance and a sink."""
-    return (dk == 128 and dv == 128 and group <= 16 and not window and not keep_first and r1 is None and not v_row
-            and not softcap)
+    values alike, all earlier keys visible or a window's beside kept first tokens, and nothing between the scaled score and
+    the softmax but a table by distance and a sink."""
+    return dk == 128 and dv == 128 and group <= 16 and r1 is None and not v_row and not softcap
 
 
 def plan_biased(host, group: int, window: int, keep_first: int) -> Dict[str, np.ndarray]:
@@ -332,14 +331,15 @@ def attend_biased(ctx, plan, qkv, kv, nq: int, nkv: int, dk: int, dv: int, windo
         items, tiles = plan.get("decode_items"), _pairs(plan.get("tiles64"))
         tiles128 = _pairs(plan.get("tiles128"), 3)
         if (tiles128 is not None and tcgen05_runs(dk, dv, nq // nkv, window, keep_first, r1, v_row, softcap)
-                and (gate_off < 0 or gate_off % 8 == 0) and out.is_contiguous() and kernels.attention_tcgen05_supports(qkv.dtype, dk, kv.page_size, qkv)):
+                and (gate_off < 0 or gate_off % 8 == 0) and not (dist_bias is not None and keep_first) and kernels.attention_tcgen05_rows(out)
+                and kernels.attention_tcgen05_supports(qkv.dtype, dk, kv.page_size, qkv)):
             # the runs on the tcgen05 kernel (whose rows take a table by distance in their scores, and a sink and a gate
             # where they become results); the single tokens stay with the kernel below
             merge128 = _pairs(plan.get("merge128"), 4)
             parts = None if merge128 is None else _scratch_floats(tiles128.shape[0] * nkv * 128 * (dk + 2), qkv.device, "parts")
             kernels.attention_prefill_tcgen05(qkv, out, kv.k_pages, kv.v_pages, kv.block_table, ctx.cu_q, ctx.q_start_pos, tiles128,
-                                              nq, nkv, dk, kv.page_size, 0, scale, merge128, parts, pairs=plan.get("pairs128") is not None,
-                                              sink=sink, gate_off=gate_off, dist_bias=dist_bias)
+                                              nq, nkv, dk, kv.page_size, window, scale, merge128, parts, pairs=plan.get("pairs128") is not None,
+                                              sink=sink, gate_off=gate_off, dist_bias=dist_bias, keep_first=keep_first)
             tiles = None
             if items is None:
                 return out
@@ -368,11 +368,19 @@ def attend_differential(ctx, plan, qkv, gate, kv, heads: int, kv_heads: int, dk:
     keys (rows of both maps, 2 * dk channels) and values already in the pages; ``gate``: rows of heads * dv channels.
     Returns [N, heads * dv]: per head the first map's result minus ``lam`` times the second's, divided by its root mean
     square, times ``gain`` and the gate's sigmoid.  ``plan``: ``plan_biased`` for groups of 2 * heads / kv_heads rows (a
-    token's heads on both maps); a tile of 64 such rows is 32 (token, head) pairs."""
+    token's heads on both maps; a tile of 64 such rows is 32 (token, head) pairs), and with ``tiles128`` for maps of 64 channels
+    over values of 128, whose runs then go to the tcgen05 kernel."""
     out = torch.empty((qkv.shape[0], heads * dv), dtype=qkv.dtype, device=qkv.device)
     window = int(window or 0)
     if kernels.differential_attention_mma_supports(qkv, gate, dk, dv):
         items, tiles = plan.get("decode_items"), _pairs(plan.get("tiles64"))
+        tiles128 = _pairs(plan.get("tiles128"), 3)
+        if tiles128 is not None and kernels.differential_attention_tcgen05_supports(qkv, gate, heads, kv_heads, dk, dv, kv.page_size):
+            kernels.differential_attention_tcgen05(qkv, gate, out, kv.k_pages, kv.v_pages, kv.block_table, ctx.cu_q, ctx.q_start_pos, tiles128, heads,
+                                                   kv_heads, dk, dv, kv.page_size, window, scale, lam, gain, eps)
+            tiles = None
+            if items is None:
+                return out
         splits, scratch = 1, None
         if items is not None:
             splits = decode_splits(items.shape[0], kv_heads, min(ctx.max_kv_len, window) if window else ctx.max_kv_len)

@@ -376,13 +376,18 @@ def attention_tcgen05_supports(dtype: torch.dtype, head_dim: int, page_size: int
     return qkv is None or (qkv.data_ptr() % 16 == 0 and qkv.stride(0) % 8 == 0 and qkv.stride(1) == 1)
 
 
+def attention_tcgen05_rows(out: torch.Tensor) -> bool:
+    """Whether the tcgen05 attention can store its results into these rows."""
+    return out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+
+
 def attention_prefill_tcgen05(qkv: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                               block_table: torch.Tensor, cu_q: torch.Tensor, q_start_pos: torch.Tensor,
                               tiles: torch.Tensor, nq: int, nkv: int, head_dim: int, page_size: int, window: int,
                               scale: float, merges: Optional[torch.Tensor] = None,
                               scratch: Optional[torch.Tensor] = None, pairs: bool = False,
                               sink: Optional[torch.Tensor] = None, gate_off: int = -1,
-                              dist_bias: Optional[torch.Tensor] = None) -> None:
+                              dist_bias: Optional[torch.Tensor] = None, keep_first: int = 0) -> None:
     """``attention_prefill`` on the tcgen05 tensor cores (scores, P and the outputs in tensor memory).
     ``tiles`` is int32 [n, 3]: (entry, row tile, code) with row tiles of 128 rows; code 1 is a whole
     tile, else first part << 8 | part << 4 | parts: one of the parts its keys are cut into, which
@@ -392,10 +397,13 @@ def attention_prefill_tcgen05(qkv: torch.Tensor, out: torch.Tensor, k_pages: tor
     means half of the keys for each, added up through the cluster's shared memory, code 1 the whole
     tile for one of them.  ``sink`` (float32 [nq]) joins each head's denominator; ``gate_off`` >= 0 (a multiple of 8):
     the rows of ``qkv`` hold nq * head_dim gate channels there, whose sigmoid multiplies the result.  ``dist_bias``
-    (float32 [rows, nq]): ``dist_bias[min(i - j, rows - 1), head]`` is added to the scaled score."""
+    (float32 [rows, nq]): ``dist_bias[min(i - j, rows - 1), head]`` is added to the scaled score.  ``keep_first``: beside a window,
+    that many first tokens stay visible.  ``out`` may be columns of wider rows (16-byte aligned)."""
     if sink is not None:
         _dev(sink, torch.float32, "attention sink")
     _check_dist_bias(dist_bias, nq)
+    if not attention_tcgen05_rows(out) or (keep_first and (not window or dist_bias is not None)):
+        raise KernelError("attention_prefill_tcgen05: results in rows on 16-byte boundaries; kept tokens stand beside a window and no table")
     if gate_off >= 0 and gate_off % 8:
         raise KernelError("attention_prefill_tcgen05: the gate channels must start on a 16-byte boundary")
     if not attention_tcgen05_supports(qkv.dtype, head_dim, page_size, qkv):
@@ -409,11 +417,11 @@ def attention_prefill_tcgen05(qkv: torch.Tensor, out: torch.Tensor, k_pages: tor
     if pairs and window:
         raise KernelError("attention_prefill_tcgen05: keys behind a window are not cut")
     _check(_fn("q25_attention_prefill_tcgen05_bf16",
-               [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P])(
+               [_P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _P, _P])(
         qkv.data_ptr(), qkv.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], cu_q.data_ptr(), q_start_pos.data_ptr(), tiles.data_ptr(), tiles.shape[0], nq, nkv,
         head_dim, page_size, int(window or 0), float(scale), _ptr(merges), n_merge, _ptr(scratch), int(bool(pairs)),
-        _ptr(sink), int(gate_off), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0],
+        _ptr(sink), int(gate_off), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0], int(keep_first), out.stride(0),
         error_flag(qkv.device).data_ptr(), _stream()), "attention_prefill_tcgen05")
     if n_merge:
         count_replayed(1)                      # the merge kernel, launched by the same call
@@ -1514,6 +1522,30 @@ def differential_attention_generic(qkv: torch.Tensor, gate: torch.Tensor, out: t
         qkv.data_ptr(), qkv.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), cu_q.data_ptr(), q_start_pos.data_ptr(), qkv.shape[0], int(heads), int(kv_heads), int(dk), int(dv),
         int(page_size), int(window or 0), float(scale), float(lam), float(gain), float(eps), _stream()), "differential_attention_generic")
+
+
+def differential_attention_tcgen05_supports(qkv: torch.Tensor, gate: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int, page_size: int) -> bool:
+    """What the tcgen05 kernel of differential attention takes: maps of 64 channels over values of 128, a power of two of up to
+    64 heads on a key/value head, 16-byte aligned rows."""
+    group = heads // kv_heads
+    return (qkv.dtype == torch.bfloat16 and dk == 64 and dv == 128 and 128 % (2 * group) == 0 and page_size > 0 and page_size & (page_size - 1) == 0
+            and (qkv.stride(0) | gate.stride(0)) % 8 == 0 and (qkv.data_ptr() | gate.data_ptr()) % 16 == 0)
+
+
+def differential_attention_tcgen05(qkv: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
+                                   block_table: torch.Tensor, cu_q: torch.Tensor, q_start_pos: torch.Tensor, tiles: torch.Tensor, heads: int,
+                                   kv_heads: int, dk: int, dv: int, page_size: int, window: int, scale: float, lam: float, gain: float,
+                                   eps: float) -> None:
+    """``differential_attention_mma`` for runs, on the tcgen05 tensor cores: ``tiles`` int32 [n, 3] are (entry, tile of 128 rows
+    (token, map, head of the group), 1)."""
+    _check_differential(qkv, gate, out, heads, kv_heads, dk, dv)
+    if not differential_attention_tcgen05_supports(qkv, gate, heads, kv_heads, dk, dv, page_size) or tiles.dim() != 2 or tiles.shape[1] != 3:
+        raise KernelError(f"differential_attention_tcgen05: unsupported sizes {dk}/{dv}, {heads} heads on {kv_heads}, pages of {page_size}")
+    _check(_fn("q25_attention_prefill_differential_bf16",
+               [_P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P])(
+        qkv.data_ptr(), qkv.stride(0), gate.data_ptr(), gate.stride(0), out.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], cu_q.data_ptr(), q_start_pos.data_ptr(), tiles.data_ptr(), tiles.shape[0], int(heads), int(kv_heads), int(page_size),
+        int(window or 0), float(scale), float(lam), float(gain), float(eps), error_flag(qkv.device).data_ptr(), _stream()), "differential_attention_tcgen05")
 
 
 # ---- the gated delta rule -------------------------------------------------------------------------------------

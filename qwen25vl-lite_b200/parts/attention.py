@@ -331,7 +331,7 @@ class SinkAttention(Mixer):
 
     def plan_key(self):
         if self._tcgen05_runs:
-            return ("sink_attention_tcgen05", self.num_heads // self.num_kv_heads, self.num_kv_heads)
+            return ("sink_attention_tcgen05", self.num_heads // self.num_kv_heads, self.num_kv_heads, self.window or 0, self.keep_first)
         return ("biased_window_attention", self.num_heads // self.num_kv_heads, self.window or 0, self.keep_first)
 
     def plan_step(self, host):
@@ -339,7 +339,7 @@ class SinkAttention(Mixer):
         plan = attention_ops.plan_biased(host, group, self.window or 0, self.keep_first)
         if self._tcgen05_runs:
             places = 2 * kernels.sm_count() // self.num_kv_heads           # two CTAs of the tcgen05 kernel fit an SM
-            wide = attention_ops.plan_step(host, group, 0, places)
+            wide = attention_ops.plan_step(host, group, self.window or 0, places)
             plan.update({name: wide[name] for name in ("tiles128", "merge128", "pairs128")})
         return plan
 
@@ -449,10 +449,18 @@ class DifferentialAttention(Mixer):
         self.lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + self.diff
 
     def plan_key(self):
-        return ("biased_window_attention", 2 * self.group, self.window or 0, 0)
+        return ("differential_attention" if self._tcgen05_runs else "biased_window_attention", 2 * self.group, self.window or 0, 0)
+
+    @property
+    def _tcgen05_runs(self) -> bool:
+        """Whether this mixer's runs of tokens can go to the tcgen05 prefill kernel (bfloat16 permitting)."""
+        return self.head_dim == 64 and self.value_dim == 128 and 128 % (2 * self.group) == 0
 
     def plan_step(self, host):
-        return attention_ops.plan_biased(host, 2 * self.group, self.window or 0, 0)
+        plan = attention_ops.plan_biased(host, 2 * self.group, self.window or 0, 0)
+        if self._tcgen05_runs:                 # whole tiles: a cut one's maps would be combined before they are added up
+            plan["tiles128"] = attention_ops.plan_step(host, 2 * self.group, self.window or 0, 0)["tiles128"]
+        return plan
 
     def forward(self, ctx, h, stop, residual=None, residual_scale=None):
         """Returns the update of the residual stream, or None after adding it into ``residual``."""

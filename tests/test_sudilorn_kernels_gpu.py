@@ -159,15 +159,20 @@ class PagedCase:
         self.ctx = SimpleNamespace(cu_q=i32(np.cumsum([0] + lens)), q_start_pos=i32(starts), token_seq=i32(np.repeat(np.arange(len(lens)), lens)),
                                    n_seqs=len(lens), max_kv_len=max(self.total))
 
-    def plan(self, group, window, keep):
-        return {k: (i32(v) if len(v) else None) for k, v in attention_ops.plan_biased(self.host, group, window or 0, keep).items()}
+    def plan(self, group, window, keep, wide=False):
+        """``wide``: with the row tiles of the tcgen05 kernels."""
+        lists = attention_ops.plan_biased(self.host, group, window or 0, keep)
+        if wide:
+            lists["tiles128"] = attention_ops.plan_step(self.host, group, window or 0, 0)["tiles128"]
+        return {k: (i32(v) if len(v) else None) for k, v in lists.items()}
 
 
-def differential_case(dtype, heads, kv, dk, dv, page, window, entries, peaks, seed, lam=0.6, diff=0.4, scale=0.25):
+def differential_case(dtype, heads, kv, dk, dv, page, window, entries, peaks, seed, lam=0.6, diff=0.4, scale=0.25, wide=None):
     """``peaks``: (entry, token of the step, head, map, key): that map's score on that key stands out by far.  Returns the
     kernels' result and the float64 one, [tokens, heads, dv]."""
     case = PagedCase(dtype, entries, kv, 2 * dk, dv, page, seed)
     group = heads // kv
+    wide = (dk, dv) == (64, 128) and 128 % (2 * group) == 0 if wide is None else wide
     qs = [case.rnd(n, heads, 2, dk) * 0.3 for _, n in entries]
     for e, t, h, m, j in peaks:
         unit = torch.zeros(dk, device=DEV)
@@ -178,9 +183,12 @@ def differential_case(dtype, heads, kv, dk, dv, page, window, entries, peaks, se
     n = sum(case.lens)
     q = torch.cat(qs).to(dtype)
     # the kernels' order: by kv head, map, head of the group; the row goes on behind the queries
-    rows = torch.cat([q.view(n, kv, group, 2, dk).transpose(2, 3).reshape(n, -1), torch.zeros(n, 10, dtype=dtype, device=DEV)], dim=1)
-    gate = torch.cat([torch.zeros(n, 6, dtype=dtype, device=DEV), case.rnd(n, heads * dv).to(dtype)], dim=1)[:, 6:]
-    got = attention_ops.attend_differential(case.ctx, case.plan(2 * group, window, 0), rows, gate, case.kv_step, heads, kv, dk, dv, window, scale, lam, 1.0 - diff, 1e-5)
+    rows = torch.cat([q.view(n, kv, group, 2, dk).transpose(2, 3).reshape(n, -1), torch.zeros(n, 8 if wide else 10, dtype=dtype, device=DEV)], dim=1)
+    pad = 8 if wide else 6
+    gate = torch.cat([torch.zeros(n, pad, dtype=dtype, device=DEV), case.rnd(n, heads * dv).to(dtype)], dim=1)[:, pad:]
+    if dtype == torch.bfloat16 and wide:
+        assert kernels.differential_attention_tcgen05_supports(rows, gate, heads, kv, dk, dv, page)
+    got = attention_ops.attend_differential(case.ctx, case.plan(2 * group, window, 0, wide), rows, gate, case.kv_step, heads, kv, dk, dv, window, scale, lam, 1.0 - diff, 1e-5)
     at, want = 0, []
     for e, (s, m) in enumerate(entries):
         k, v = npy(case.keys[e].to(dtype)).reshape(s + m, kv, 2, dk), npy(case.values[e].to(dtype))
@@ -192,7 +200,7 @@ def differential_case(dtype, heads, kv, dk, dv, page, window, entries, peaks, se
     return npy(got).reshape(n, heads, dv), np.concatenate(want) * plain.sigmoid(npy(gate)).reshape(n, heads, dv)
 
 
-DIFF_SIZES = [(4, 2, 32, 64, 16), (6, 3, 20, 28, 8), (8, 1, 64, 128, 16), (5, 1, 128, 128, 32), (10, 1, 32, 32, 16), (20, 2, 64, 64, 16), (2, 2, 128, 32, 8), (3, 1, 7, 10, 4)]
+DIFF_SIZES = [(4, 2, 32, 64, 16), (6, 3, 20, 28, 8), (8, 1, 64, 128, 16), (4, 4, 64, 128, 8), (4, 2, 64, 128, 4), (16, 1, 64, 128, 16), (5, 1, 64, 128, 16), (5, 1, 128, 128, 32), (10, 1, 32, 32, 16), (20, 2, 64, 64, 16), (2, 2, 128, 32, 8), (3, 1, 7, 10, 4)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -201,8 +209,8 @@ def test_differential_attention_at_the_windows_edges(dtype, heads, kv, dk, dv, p
     """Keys that would carry a map's whole weight, at the last place a query sees and at the first that it does not, on the
     first map, the second, and both; in runs and for single tokens; at page borders; a token's own key and the next one's."""
     window = 37
-    entries = [(150, 1), (0, 70), (61, 1), (30, 45), (0, 1), (36, 1), (100, 2)]
-    peaks = [(0, 0, 0, 0, 150 - 36), (0, 0, 1, 1, 150 - 37), (1, 69, 0, 0, 33), (1, 68, 1, 1, 31), (1, 40, 0, 1, 16), (1, 41, 1, 0, 16), (1, 36, 0, 0, 0), (1, 37, 1, 1, 0),
+    entries = [(150, 1), (0, 70), (61, 1), (30, 45), (0, 1), (36, 1), (100, 2), (70, 300)]
+    peaks = [(7, 299, 0, 0, 369 - 36), (7, 298, 1, 1, 368 - 37), (7, 127, 0, 1, 197 - 36), (7, 128, 1, 0, 198), (0, 0, 0, 0, 150 - 36), (0, 0, 1, 1, 150 - 37), (1, 69, 0, 0, 33), (1, 68, 1, 1, 31), (1, 40, 0, 1, 16), (1, 41, 1, 0, 16), (1, 36, 0, 0, 0), (1, 37, 1, 1, 0),
              (2, 0, 0, 1, 61 - 36), (2, 0, 1, 0, 61 - 37), (3, 10, 0, 0, 4), (3, 11, 1, 1, 4), (3, 44, 0, 1, 74), (3, 20, 1, 0, 51), (5, 0, 0, 0, 0), (6, 1, 0, 1, 65), (6, 0, 1, 0, 63)]
     peaks = [p for p in peaks if p[2] < heads]
     got, want = differential_case(dtype, heads, kv, dk, dv, page, window, entries, peaks, 4)
@@ -221,9 +229,11 @@ def test_differential_attention_over_everything(dtype, heads, kv, dk, dv, page):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_differential_attention_is_each_request_alone(dtype):
+@pytest.mark.parametrize("dk,dv", [(32, 64), (64, 128)])
+def test_differential_attention_is_each_request_alone(dtype, dk, dv):
     """Bit for bit: a request's rows do not depend on the others of its step."""
-    heads, kv, dk, dv, page, window = 4, 2, 32, 64, 16, 50
+    heads, kv, page, window = 4, 2, 16, 50
+    wide = (dk, dv) == (64, 128)
     entries = [(150, 1), (0, 70), (61, 1), (30, 45)]
     together, _ = differential_case(dtype, heads, kv, dk, dv, page, window, entries, [], 6)
     lone = PagedCase(dtype, entries, kv, 2 * dk, dv, page, 6)
@@ -236,7 +246,10 @@ def test_differential_attention_is_each_request_alone(dtype):
     for e, (s, m) in enumerate(entries):
         host = HostStep([m], [s], m, 1)
         ctx = SimpleNamespace(cu_q=i32([0, m]), q_start_pos=i32([s]), token_seq=i32([0] * m), n_seqs=1, max_kv_len=lone.ctx.max_kv_len)
-        plan = {k: (i32(v) if len(v) else None) for k, v in attention_ops.plan_biased(host, 2 * heads // kv, window, 0).items()}
+        lists = attention_ops.plan_biased(host, 2 * heads // kv, window, 0)
+        if wide:
+            lists["tiles128"] = attention_ops.plan_step(host, 2 * heads // kv, window, 0)["tiles128"]
+        plan = {k: (i32(v) if len(v) else None) for k, v in lists.items()}
         kv_step = KVStep(lone.kv_step.k_pages, lone.kv_step.v_pages, None, lone.kv_step.block_table[e:e + 1].contiguous(), page)
         got = attention_ops.attend_differential(ctx, plan, rows[at:at + m], gate[at:at + m], kv_step, heads, kv, dk, dv, window, 0.25, 0.6, 0.6, 1e-5)
         np.testing.assert_array_equal(npy(got).reshape(m, heads, dv), together[at:at + m])
@@ -248,16 +261,18 @@ def test_differential_attention_is_each_request_alone(dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("nq,nkv,dk,dv,page,window,keep", [(4, 2, 64, 64, 16, 20, 5), (6, 2, 24, 20, 8, 9, 3), (8, 8, 128, 128, 16, 64, 20), (4, 1, 32, 128, 8, 4, 9),
-                                                           (2, 1, 128, 128, 32, 33, 40), (20, 1, 64, 32, 16, 12, 2)])
+                                                           (2, 1, 128, 128, 32, 33, 40), (20, 1, 64, 32, 16, 12, 2), (4, 1, 128, 128, 16, 70, 66), (16, 2, 128, 128, 16, 150, 4),
+                                                           (3, 1, 128, 128, 4, 90, 130), (4, 2, 128, 128, 16, 64, 0)])
 def test_window_and_kept_tokens_into_columns_of_wider_rows(dtype, nq, nkv, dk, dv, page, window, keep):
     """Keys that carry the whole weight as the last kept token, the first that is not kept, the last the window shows and the
     first it does not; the result goes into columns of wider rows and leaves the others alone."""
-    entries = [(100, 1), (0, 90), (40, 1), (50, 30), (0, 1)]
-    group = nq // nkv
+    entries = [(100, 1), (0, 90), (40, 1), (50, 30), (0, 1), (120, 260)]
+    group, tiles128 = nq // nkv, dk == 128 and dv == 128          # those runs go to the tcgen05 kernel
+    assert not tiles128 or attention_ops.tcgen05_runs(dk, dv, group, window, keep, None, 0, 0.0)
     case = PagedCase(dtype, entries, nkv, dk, dv, page, 7)
     qs = [case.rnd(n, nq, dk) * 0.3 for _, n in entries]
     places = lambda p: (keep - 1, keep, p - window + 1, p - window, p, 0)
-    for e, t in ((0, 0), (1, 89), (1, 60), (2, 0), (3, 3), (3, 29)):
+    for e, t in ((0, 0), (1, 89), (1, 60), (2, 0), (3, 3), (3, 29), (5, 259), (5, 100), (5, 64)):
         p = entries[e][0] + t
         for h, j in enumerate(places(p)[:nq]):
             if 0 <= j <= p:
@@ -269,7 +284,7 @@ def test_window_and_kept_tokens_into_columns_of_wider_rows(dtype, nq, nkv, dk, d
     n = sum(case.lens)
     q = torch.cat(qs).to(dtype)
     wide = torch.full((n, nq * dv + 24), 7.0, dtype=dtype, device=DEV)
-    attention_ops.attend_biased(case.ctx, case.plan(group, window, keep), q.reshape(n, -1), case.kv_step, nq, nkv, dk, dv, window, keep, 0.25, None, None, out=wide[:, 16:16 + nq * dv])
+    attention_ops.attend_biased(case.ctx, case.plan(group, window, keep, tiles128), q.reshape(n, -1), case.kv_step, nq, nkv, dk, dv, window, keep, 0.25, None, None, out=wide[:, 16:16 + nq * dv])
     assert (wide[:, :16] == 7.0).all() and (wide[:, 16 + nq * dv:] == 7.0).all()
     got, at = npy(wide[:, 16:16 + nq * dv]).reshape(n, nq, dv), 0
     for e, (s, m) in enumerate(entries):
