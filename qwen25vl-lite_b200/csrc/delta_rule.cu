@@ -317,13 +317,15 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_prepare_kernel(DeltaArgs 
       kk = fmaf(k.x, k.x, fmaf(k.y, k.y, kk)); qq = fmaf(q.x, q.x, fmaf(q.y, q.y, qq));
     }
     kk = warp_sum(kk); qq = warp_sum(qq);
-    if (lane == 0) {
-      const float ik = 1.0f / sqrtf(kk + p.unit_eps), iq = p.q_scale / sqrtf(qq + p.unit_eps), ec = expf(num[r]);
-      num[2 * DL + r] = ik; num[3 * DL + r] = iq; num[4 * DL + r] = num[DL + r] * ec * ik;
-      out.row[ch * 2 * DL + r] = ec * iq;
-      out.row[(ch * 2 + 1) * DL + r] = expf(num[DL - 1] - num[r]) * ik;
-      if (r == 0) out.keep[ch] = expf(num[DL - 1]);
-    }
+    if (lane == 0) { num[2 * DL + r] = kk; num[3 * DL + r] = qq; }
+  }
+  __syncthreads();
+  if (tid < DL) {
+    const float ik = 1.0f / sqrtf(num[2 * DL + tid] + p.unit_eps), iq = p.q_scale / sqrtf(num[3 * DL + tid] + p.unit_eps), ec = expf(num[tid]);
+    num[2 * DL + tid] = ik; num[3 * DL + tid] = iq; num[4 * DL + tid] = num[DL + tid] * ec * ik;
+    out.row[ch * 2 * DL + tid] = ec * iq;
+    out.row[(ch * 2 + 1) * DL + tid] = expf(num[DL - 1] - num[tid]) * ik;
+    if (tid == 0) out.keep[ch] = expf(num[DL - 1]);
   }
   __syncthreads();
   // scores: 10 tiles of 16 x 16 on and below the diagonal, of K K^T (jobs 0 .. 9) and Q K^T (10 .. 19)
@@ -396,7 +398,13 @@ __global__ void __launch_bounds__(DL_THREADS, 3) delta_prepare_kernel(DeltaArgs 
     for (int i = tid; i < (4 - d) * 256; i += DL_THREADS) {
       const int J = i >> 8, I = J + d, r = (i >> 4) & 15, c = i & 15;
       float v = 0.f;
-      for (int k = J * 16; k < I * 16; ++k) v = fmaf(A[(I * 16 + r) * FP + k], Ti[k * FP + J * 16 + c], v);
+      for (int k = J * 16; k < I * 16; k += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(A + (I * 16 + r) * FP + k);
+        v = fmaf(a.x, Ti[k * FP + J * 16 + c], v);
+        v = fmaf(a.y, Ti[(k + 1) * FP + J * 16 + c], v);
+        v = fmaf(a.z, Ti[(k + 2) * FP + J * 16 + c], v);
+        v = fmaf(a.w, Ti[(k + 3) * FP + J * 16 + c], v);
+      }
       W[J * 16 * 17 + r * 17 + c] = v;
     }
     __syncthreads();

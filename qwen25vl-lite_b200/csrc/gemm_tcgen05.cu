@@ -85,11 +85,23 @@ __device__ __forceinline__ void t5_emit32(const float (&v)[32], int m, int n, in
     }
   } else if constexpr (EPI == T5_F32 || EPI == T5_RESIDUAL) {
     float* dst = reinterpret_cast<float*>(out) + (size_t)m * ldo + n;
+    if (n + 32 <= N && (reinterpret_cast<uintptr_t>(dst) & 15) == 0) {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) {
-      if (n + j >= N) break;
-      if constexpr (EPI == T5_RESIDUAL) dst[j] += v[j];
-      else dst[j] = v[j];
+      for (int q = 0; q < 8; ++q) {
+        float4 y = make_float4(v[q * 4], v[q * 4 + 1], v[q * 4 + 2], v[q * 4 + 3]);
+        if constexpr (EPI == T5_RESIDUAL) {
+          const float4 old = *reinterpret_cast<const float4*>(dst + q * 4);
+          y.x += old.x; y.y += old.y; y.z += old.z; y.w += old.w;
+        }
+        *reinterpret_cast<float4*>(dst + q * 4) = y;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) {
+        if (n + j >= N) break;
+        if constexpr (EPI == T5_RESIDUAL) dst[j] += v[j];
+        else dst[j] = v[j];
+      }
     }
   } else {
     bf16* dst = reinterpret_cast<bf16*>(out) + (size_t)m * ldo + n;

@@ -69,32 +69,12 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ router, cons
   }
 }
 
-// The router of a mixture whose scores are a softmax over all `outputs` router rows (sigmoid != 0: each row's sigmoid), the
-// last `outputs - experts` of which stand for experts without matrices (a choice among them takes no row of the grouped products).  The choice looks
-// at score + correction[e]; the rows form `groups` equal runs of neighbours, a run's mark is its largest such number
-// (mark_two != 0: the sum of its two largest), and only the `keep` runs with the largest marks can be chosen from (the others count as minus infinity).  The `top`
-// largest are chosen (ties to the lower index, among runs too); a choice weighs in with its plain score: as it is, or
-// with renorm divided by the sum of the token's chosen scores (+ 1e-20); either way times weight_scale.  counts: one per
-// expert with matrices.  One block of 8 warps per TOK tokens as above, then a warp per token.
-template <typename T, int TOK>
-__global__ void __launch_bounds__(256)
-moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
-                         int* __restrict__ topk_idx, float* __restrict__ topk_w, int* __restrict__ counts, int n_tokens, int hidden,
-                         int experts, int outputs, int top, int groups, int keep, int renorm, float weight_scale,
-                         int sigmoid, int mark_two) {
-  pdl_trigger();
-  pdl_wait();
-  extern __shared__ __align__(16) float route_smem[];       // TOK rows of hidden floats, then TOK x 3 x (MOE_MAX_EXPERTS + 1) numbers
-  route_logits<T, TOK>(h, router, nullptr, route_smem, n_tokens, hidden, outputs);
-  const int pitch = (hidden + 3) & ~3;
-  float* zs = route_smem + TOK * pitch;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n0 = blockIdx.x * TOK;
-  if (warp >= TOK || n0 + warp >= n_tokens) return;
-  const int n = n0 + warp;
-  float* score = zs + warp * (MOE_MAX_EXPERTS + 1);                          // logits, then scores
-  float* choice = zs + (TOK + 2 * warp) * (MOE_MAX_EXPERTS + 1);             // score + correction
-  float* mark = choice + (MOE_MAX_EXPERTS + 1);                              // a run's mark
+// One token's choice by a warp: score: its `outputs` logits (shared memory), which become scores; choice and mark: room for as
+// many numbers each.  See moe_route_softmax_kernel for the rules.
+__device__ __forceinline__ void moe_choose(float* score, float* choice, float* mark, const float* __restrict__ correction, int* __restrict__ topk_idx,
+                                           float* __restrict__ topk_w, int* __restrict__ counts, int n, int experts, int outputs, int top, int groups,
+                                           int keep, int renorm, float weight_scale, int sigmoid, int mark_two) {
+  const int lane = threadIdx.x & 31;
   float top_z = -INFINITY, sum = 0.f;
   if (!sigmoid) {
     for (int e = lane; e < outputs; e += 32) top_z = fmaxf(top_z, score[e]);
@@ -175,8 +155,8 @@ moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ rout
       mark[k] = none ? 0.f : score[arg];                        // the marks of the runs have served: the chosen scores wait here
       if (!none) {
         choice[arg] = -INFINITY;
-        if (arg < experts) atomicAdd(&counts[arg], 1);
-      } else {
+        if (counts && arg < experts) atomicAdd(&counts[arg], 1);
+      } else if (counts) {
         atomicAdd(&counts[0], 1);
       }
     }
@@ -185,6 +165,50 @@ moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ rout
   float chosen = 0.f;                                           // in the order of the choices, the same in every lane
   if (renorm) for (int k = 0; k < top; ++k) chosen += mark[k];
   for (int k = lane; k < top; k += 32) topk_w[(size_t)n * top + k] = (renorm ? mark[k] / (chosen + 1e-20f) : mark[k]) * weight_scale;
+}
+
+// The router of a mixture whose scores are a softmax over all `outputs` router rows (sigmoid != 0: each row's sigmoid), the
+// last `outputs - experts` of which stand for experts without matrices (a choice among them takes no row of the grouped products).  The choice looks
+// at score + correction[e]; the rows form `groups` equal runs of neighbours, a run's mark is its largest such number
+// (mark_two != 0: the sum of its two largest), and only the `keep` runs with the largest marks can be chosen from (the others count as minus infinity).  The `top`
+// largest are chosen (ties to the lower index, among runs too); a choice weighs in with its plain score: as it is, or
+// with renorm divided by the sum of the token's chosen scores (+ 1e-20); either way times weight_scale.  counts: one per
+// expert with matrices.  One block of 8 warps per TOK tokens as above, then a warp per token.
+template <typename T, int TOK>
+__global__ void __launch_bounds__(256)
+moe_route_softmax_kernel(const T* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
+                         int* __restrict__ topk_idx, float* __restrict__ topk_w, int* __restrict__ counts, int n_tokens, int hidden,
+                         int experts, int outputs, int top, int groups, int keep, int renorm, float weight_scale,
+                         int sigmoid, int mark_two) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ __align__(16) float route_smem[];       // TOK rows of hidden floats, then TOK x 3 x (MOE_MAX_EXPERTS + 1) numbers
+  route_logits<T, TOK>(h, router, nullptr, route_smem, n_tokens, hidden, outputs);
+  const int pitch = (hidden + 3) & ~3;
+  float* zs = route_smem + TOK * pitch;
+  const int warp = threadIdx.x >> 5;
+  const int n0 = blockIdx.x * TOK;
+  if (warp >= TOK || n0 + warp >= n_tokens) return;
+  const int n = n0 + warp;
+  moe_choose(zs + warp * (MOE_MAX_EXPERTS + 1), zs + (TOK + 2 * warp) * (MOE_MAX_EXPERTS + 1), zs + (TOK + 2 * warp + 1) * (MOE_MAX_EXPERTS + 1), correction,
+             topk_idx, topk_w, counts, n, experts, outputs, top, groups, keep, renorm, weight_scale, sigmoid, mark_two);
+}
+
+// The same from logits that a product has left (float, [n_tokens, outputs]): a warp per token.
+__global__ void __launch_bounds__(256)
+moe_choose_kernel(const float* __restrict__ z, const float* __restrict__ correction, int* __restrict__ topk_idx, float* __restrict__ topk_w,
+                  int* __restrict__ counts, int n_tokens, int experts, int outputs, int top, int groups, int keep, int renorm, float weight_scale,
+                  int sigmoid, int mark_two) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float rows[8 * 3 * (MOE_MAX_EXPERTS + 1)];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockIdx.x * 8 + warp;
+  if (n >= n_tokens) return;
+  float* score = rows + warp * 3 * (MOE_MAX_EXPERTS + 1);
+  for (int e = lane; e < outputs; e += 32) score[e] = z[(size_t)n * outputs + e];
+  __syncwarp();
+  moe_choose(score, score + MOE_MAX_EXPERTS + 1, score + 2 * (MOE_MAX_EXPERTS + 1), correction, topk_idx, topk_w, counts, n, experts, outputs, top, groups,
+             keep, renorm, weight_scale, sigmoid, mark_two);
 }
 
 // One block: where every expert's rows begin (each expert filled up to whole tiles of `tile` rows),
@@ -228,6 +252,54 @@ __global__ void moe_scatter_kernel(const int* __restrict__ topk_idx, const int* 
 #define MOE_GATE_UP 1
 #define MOE_UP_RELU2 2
 __device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.f); return v * v; }
+
+// The two of a step of few pairs, by one block that counts for itself (nothing has to be zero before): counts, the rows'
+// places and every pair's row.
+#define MOE_SMALL_PAIRS 2048
+__global__ void __launch_bounds__(256) moe_sort_small_kernel(const int* __restrict__ topk_idx, int* __restrict__ plan, int* __restrict__ row_pair,
+                                                            int* __restrict__ pair_row, int n_pairs, int experts, int tile, int max_rows) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ int count[MOE_MAX_EXPERTS], place[MOE_MAX_EXPERTS];
+  for (int e = threadIdx.x; e < experts; e += 256) count[e] = 0;
+  for (int r = threadIdx.x; r < max_rows; r += 256) row_pair[r] = -1;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_pairs; i += 256) {
+    const int e = topk_idx[i];
+    if (e < experts) atomicAdd(&count[e], 1);
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {                                    // a warp: eight neighbouring experts a lane, then a scan over the lanes
+    const int lane = threadIdx.x, per = (experts + 31) / 32;
+    int tiles = 0;
+    for (int i = 0; i < per; ++i) { const int e = lane * per + i; if (e < experts) tiles += (count[e] + tile - 1) / tile; }
+    int before = tiles;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, before, o); if (lane >= o) before += v; }
+    const int total = __shfl_sync(0xffffffffu, before, 31);
+    before -= tiles;
+    int* tile_expert = plan + 2 + experts;
+    for (int i = 0; i < per; ++i) {
+      const int e = lane * per + i;
+      if (e < experts) {
+        const int mine = (count[e] + tile - 1) / tile;
+        plan[1 + e] = before * tile;
+        place[e] = before * tile;
+        for (int t = 0; t < mine; ++t) tile_expert[before + t] = e;
+        before += mine;
+      }
+    }
+    if (lane == 0) { plan[0] = total; plan[1 + experts] = total * tile; }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < n_pairs; i += 256) {
+    const int e = topk_idx[i];
+    if (e >= experts) { pair_row[i] = -1; continue; }
+    const int r = atomicAdd(&place[e], 1);
+    row_pair[r] = i;
+    pair_row[i] = r;
+  }
+}
 
 // Grouped product on the CUDA cores.  MOE_GATE_UP: rows are the tile's pairs, a = weight * h[token];
 // two chains per element (gate, up), activation in the epilogue, out = act [rows, N] in T.  MOE_UP_RELU2: the same rows,
@@ -629,6 +701,15 @@ Q25_EXPORT int q25_moe_route_bf16(const void* h, const float* r, const float* g,
   return moe_route<bf16>(h, r, g, ti, tw, sg, counts, n, hidden, experts, top, s);
 }
 
+// Steps of up to MOE_SMALL_PAIRS pairs: no counts, no cursor, one kernel.
+Q25_EXPORT int q25_moe_sort_small(const int* topk_idx, int* plan, int* row_pair, int* pair_row, int n_pairs, int experts, int tile, void* stream) {
+  if (n_pairs <= 0) return 0;
+  if (n_pairs > MOE_SMALL_PAIRS || experts <= 0 || experts > MOE_MAX_EXPERTS) return (int)cudaErrorInvalidValue;
+  launch(moe_sort_small_kernel, dim3(1), dim3(256), 0, (cudaStream_t)stream, topk_idx, plan, row_pair, pair_row, n_pairs, experts, tile,
+         q25_moe_max_rows(n_pairs, experts, tile));
+  return launch_status();
+}
+
 // counts and cursor: `experts` ints each, zero on entry (cursor is left as the counts).
 Q25_EXPORT int q25_moe_sort(const int* topk_idx, const int* counts, int* cursor, int* plan, int* row_pair, int* pair_row, int n_pairs,
                             int experts, int tile, void* stream) {
@@ -814,4 +895,15 @@ Q25_EXPORT int q25_moe_combine_weighted_f32(const float* y, const int* pr, const
 }
 Q25_EXPORT int q25_moe_combine_weighted_bf16(const float* y, const int* pr, const float* tw, const void* h, const void* sh, void* out, float* x, const float* xs, int n, int hd, int top, void* s) {
   return moe_combine_weighted<bf16>(y, pr, tw, h, sh, out, x, xs, n, hd, top, s);
+}
+
+// The choice from logits that a product has left; the rules of q25_moe_route_softmax.  counts may be nullptr.
+Q25_EXPORT int q25_moe_choose(const float* z, const float* corr, int* ti, float* tw, int* counts, int n, int experts, int outputs, int top, int groups, int keep,
+                              int renorm, float wscale, int sig, int two, void* s) {
+  if (n <= 0) return 0;
+  if (experts <= 0 || outputs < experts || outputs > MOE_MAX_EXPERTS || top <= 0 || top > MOE_MAX_TOP || groups < 1 || outputs % groups || keep < 1 ||
+      keep > groups || top > keep * (outputs / groups))
+    return (int)cudaErrorInvalidValue;
+  launch(moe_choose_kernel, dim3((n + 7) / 8), dim3(256), 0, (cudaStream_t)s, z, corr, ti, tw, counts, n, experts, outputs, top, groups, keep, renorm, wscale, sig, two);
+  return launch_status();
 }

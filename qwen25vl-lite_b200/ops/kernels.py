@@ -1033,6 +1033,18 @@ def moe_sort(topk_idx: torch.Tensor, counts: torch.Tensor, cursor: torch.Tensor,
     count_replayed(1)                          # two kernels in one call
 
 
+MOE_SMALL_PAIRS = 2048           # up to this many (token, expert) pairs one block sorts a step
+
+
+def moe_sort_small(topk_idx: torch.Tensor, plan: torch.Tensor, row_pair: torch.Tensor, pair_row: torch.Tensor, experts: int, tile: int) -> None:
+    """``moe_sort`` for a step of up to ``MOE_SMALL_PAIRS`` pairs: one kernel that counts for itself."""
+    n_pairs = topk_idx.numel()
+    if n_pairs > MOE_SMALL_PAIRS or plan.numel() < 2 + experts + moe_max_rows(n_pairs, experts, tile) // tile or row_pair.numel() < moe_max_rows(n_pairs, experts, tile):
+        raise KernelError("moe_sort_small: too many pairs, or the plan or the row list is too short")
+    _check(_fn("q25_moe_sort_small", [_P, _P, _P, _P, _I, _I, _I, _P])(
+        topk_idx.data_ptr(), plan.data_ptr(), row_pair.data_ptr(), pair_row.data_ptr(), n_pairs, experts, tile, _stream()), "moe_sort_small")
+
+
 def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, act: torch.Tensor, plan: torch.Tensor, row_pair: torch.Tensor,
                 topk_w: Optional[torch.Tensor], top: int, limit: float, alpha: float, tile: int, shift: float = 1.0,
                 n_pairs: Optional[int] = None, gated: bool = True) -> None:
@@ -1122,6 +1134,18 @@ def moe_route_softmax(h: torch.Tensor, router: torch.Tensor, correction: Optiona
                                                     counts.data_ptr(), n, hidden, int(experts), outputs, int(top), int(groups), int(keep),
                                                     int(bool(renorm)), float(weight_scale), int(scores == "sigmoid"), int(mark == "two_largest"),
                                                     _stream()), "moe_route_softmax")
+
+
+def moe_choose(z: torch.Tensor, correction: Optional[torch.Tensor], experts: int, top: int, groups: int, keep: int, topk_idx: torch.Tensor,
+               topk_w: torch.Tensor, counts: Optional[torch.Tensor], renorm: bool = False, weight_scale: float = 1.0, scores: str = "softmax",
+               mark: str = "largest") -> None:
+    """``moe_route_softmax`` from logits that a product has left (float32 [N, outputs]); ``counts`` may be None."""
+    _dev(z, torch.float32, "moe_choose logits"); _dev(topk_idx, torch.int32, "moe_choose idx"); _dev(topk_w, torch.float32, "moe_choose weights")
+    if correction is not None:
+        _dev(correction, torch.float32, "moe_choose correction")
+    _check(_fn("q25_moe_choose", [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P])(
+        z.data_ptr(), _ptr(correction), topk_idx.data_ptr(), topk_w.data_ptr(), _ptr(counts), z.shape[0], int(experts), z.shape[1], int(top), int(groups),
+        int(keep), int(bool(renorm)), float(weight_scale), int(scores == "sigmoid"), int(mark == "two_largest"), _stream()), "moe_choose")
 
 
 def moe_combine_weighted(y: torch.Tensor, pair_row: torch.Tensor, topk_w: torch.Tensor, h: torch.Tensor, out: Optional[torch.Tensor], top: int,

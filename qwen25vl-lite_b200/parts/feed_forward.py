@@ -174,13 +174,15 @@ class RoutedGLU(FeedForward):
         return out
 
 
-def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, limit: float, alpha: float, shift: float, gated: bool = True):
+def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, limit: float, alpha: float, shift: float, gated: bool = True,
+                 uncounted: bool = False):
     """The grouped products of a routed feed-forward.  ``route(topk_idx, topk_w, counts)`` launches the router, which
     writes every token's ``top`` choices (int32 [N, top]; a choice beyond the experts that have matrices takes no row),
     their weights (float32) and how many tokens chose each expert.  The pairs are sorted by expert on the device and
     two grouped products walk them: ``act = g * sigmoid(alpha g) * (u + shift)`` with ``g = min(Wg a, limit)``,
     ``u = clamp(Wu a, -limit, limit)``, then ``Wd act``; ``a`` is the token's row times the pair's weight
-    (``weigh_input``) or the row as it is.  ``gated`` False: the experts have up rows alone, ``act = max(Wu a, 0)^2``.  Returns (float32 rows in the sorted order, the row of every pair or -1,
+    (``weigh_input``) or the row as it is.  ``gated`` False: the experts have up rows alone, ``act = max(Wu a, 0)^2``.
+    ``uncounted``: ``route`` takes None for its counts.  Returns (float32 rows in the sorted order, the row of every pair or -1,
     the weights)."""
     experts, ff2, hidden = w_gate_up.shape
     expert_size = ff2 // 2 if gated else ff2
@@ -195,17 +197,22 @@ def _run_experts(ctx, h, w_gate_up, w_down, top: int, route, weigh_input: bool, 
     tcgen05 = (many and hidden >= TCGEN05_MIN_WIDTH and kernels.gemm_tcgen05_grouped_supports(ctx.dtype, hidden, expert_size))
     tile = 16 if pairs <= 16 * experts else (128 if many else 64)
     rows = kernels.moe_max_rows(pairs, experts, tile)
-    # counts | cursor (zero) | plan | row of every pair | pair of every row
+    # counts | cursor (zero) | plan | row of every pair | pair of every row; a step of few pairs is sorted by one kernel that
+    # needs no counts (``uncounted``: the route does not either)
     n_plan = 2 + experts + rows // tile
-    ints = torch.zeros(2 * experts + n_plan + pairs + rows, dtype=torch.int32, device=dev)
+    small = uncounted and pairs <= kernels.MOE_SMALL_PAIRS
+    ints = (torch.empty if small else torch.zeros)(2 * experts + n_plan + pairs + rows, dtype=torch.int32, device=dev)
     counts, cursor = ints[:experts], ints[experts:2 * experts]
     plan = ints[2 * experts:2 * experts + n_plan]
     pair_row = ints[2 * experts + n_plan:2 * experts + n_plan + pairs]
     row_pair = ints[2 * experts + n_plan + pairs:]
     topk_idx = torch.empty((n, top), dtype=torch.int32, device=dev)
     topk_w = torch.empty((n, top), dtype=torch.float32, device=dev)
-    route(topk_idx, topk_w, counts)
-    kernels.moe_sort(topk_idx, counts, cursor, plan, row_pair, pair_row, experts, tile)
+    route(topk_idx, topk_w, None if small else counts)
+    if small:
+        kernels.moe_sort_small(topk_idx, plan, row_pair, pair_row, experts, tile)
+    else:
+        kernels.moe_sort(topk_idx, counts, cursor, plan, row_pair, pair_row, experts, tile)
     act = torch.empty((rows, expert_size), dtype=ctx.dtype, device=dev)
     y = torch.empty((rows, hidden), dtype=torch.float32, device=dev)
     in_w = topk_w if weigh_input else None
@@ -308,7 +315,9 @@ class GroupedRoutedMLP(FeedForward):
     largest are chosen; their outputs weigh in with their plain scores ``s``, not renormalised.  Tensors: ``router``,
     ``correction``, ``e<i>.up|down``.
 
-    Router, sort by expert and grouped products are those of the other mixtures (``csrc/moe.cu``, and the grouped mode of
+    In bfloat16 the router's logits are a product whose result stays in float32, when the checkpoint's router is bfloat16
+    numbers: products of bfloat16 numbers are exact, so this is the float32 router up to the order of its sums.  Router,
+    sort by expert and grouped products are those of the other mixtures (``csrc/moe.cu``, and the grouped mode of
     ``csrc/gemm_tcgen05.cu`` with the square of relu as its epilogue); the kernel that sums a token's choices can add the
     sum, scaled per channel, into the residual stream."""
 
@@ -340,12 +349,21 @@ class GroupedRoutedMLP(FeedForward):
         self.w_up, self.w_down = stack("up"), stack("down")
         self.router = tensors["router"].to(device=device, dtype=torch.float32).contiguous()
         self.correction = tensors["correction"].to(device=device, dtype=torch.float32).contiguous() if self.has_correction else None
+        self.router_proj = None
+        if dtype == torch.bfloat16 and bool((self.router.to(dtype).float() == self.router).all()):
+            self.router_proj = Linear(self.router.to(dtype).contiguous())
 
     def forward(self, ctx, h, residual=None, residual_scale=None):
         """Returns the update of the residual stream, or None after adding it (scaled) into ``residual``."""
-        route = lambda idx, w, counts: kernels.moe_route_softmax(h, self.router, self.correction, self.experts, self.top, self.groups,
-                                                                 self.keep, idx, w, counts, scores="sigmoid", mark="two_largest")
-        y, pair_row, topk_w = _run_experts(ctx, h, self.w_up, self.w_down, self.top, route, False, 0.0, 0.0, 0.0, gated=False)
+        choice = dict(scores="sigmoid", mark="two_largest")
+        if self.router_proj is not None:
+            z = self.router_proj(h, out_dtype=torch.float32)
+            route = lambda idx, w, counts: kernels.moe_choose(z, self.correction, self.experts, self.top, self.groups, self.keep, idx, w, counts, **choice)
+        else:
+            route = lambda idx, w, counts: kernels.moe_route_softmax(h, self.router, self.correction, self.experts, self.top, self.groups, self.keep, idx, w,
+                                                                     counts, **choice)
+        y, pair_row, topk_w = _run_experts(ctx, h, self.w_up, self.w_down, self.top, route, False, 0.0, 0.0, 0.0, gated=False,
+                                           uncounted=self.router_proj is not None)
         out = None if residual is not None else torch.empty((h.shape[0], self.hidden_size), dtype=ctx.dtype, device=h.device)
         kernels.moe_combine_weighted(y, pair_row, topk_w, h, out, self.top, residual=residual, residual_scale=residual_scale)
         return out

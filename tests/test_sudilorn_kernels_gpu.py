@@ -473,11 +473,39 @@ def test_router_by_the_two_largest_of_a_group(dtype, experts, count, keep, top):
                 np.testing.assert_allclose(npy(w[t]), weights, rtol=1e-4, atol=1e-6)
         assert same >= 0.98 * rows                       # the rest: numbers within float32's rounding of one another
         assert counts.sum().item() == rows * top and torch.equal(torch.bincount(idx.reshape(-1).long(), minlength=experts).int(), counts)
+        # the choice from logits that are there already, with and without counts
+        idx2, w2, counts2 = torch.empty_like(idx), torch.empty_like(w), torch.zeros_like(counts)
+        for c in (counts2, None):
+            kernels.moe_choose(f32(z[:rows]), corr, experts, top, count, keep, idx2, w2, c, scores="sigmoid", mark="two_largest")
+            agree = (idx2 == idx).all(dim=1)
+            assert agree.float().mean() >= 0.98 and torch.allclose(w2[agree], w[agree], rtol=1e-4, atol=1e-6)
+        assert torch.equal(torch.bincount(idx2.reshape(-1).long(), minlength=experts).int(), counts2)
     if 1 < count < experts and keep < count:
         other = torch.empty_like(idx)
         kernels.moe_route_softmax(h[:3], router, corr, experts, top, count, keep, other, w, counts, scores="sigmoid")
         marks = lambda k: [[np.sort(part)[::-1][:k].sum() for part in (plain.sigmoid(z[t]) + npy(corr)).reshape(count, -1)] for t in range(n)]
         assert any(np.argsort(a)[::-1][:keep].tolist() != np.argsort(b)[::-1][:keep].tolist() for a, b in zip(marks(1), marks(2)))
+
+
+@pytest.mark.parametrize("pairs,experts,tile", [(1, 1, 16), (16, 8, 16), (2048, 256, 16), (2000, 7, 64), (300, 200, 128), (40, 33, 64)])
+def test_pairs_sorted_by_one_block(pairs, experts, tile):
+    """Every pair has a row of its own in its expert's tiles, the other rows are empty, and the tiles are its experts' in order;
+    choices beyond the experts take no row; nothing has to be cleared before."""
+    idx = torch.tensor(np.random.default_rng(3).integers(0, experts + 2, size=pairs) % (experts + 1), dtype=torch.int32, device=DEV)
+    rows = kernels.moe_max_rows(pairs, experts, tile)
+    plan, row_pair, pair_row = (torch.full((k,), 12345, dtype=torch.int32, device=DEV) for k in (2 + experts + rows // tile, rows, pairs))
+    kernels.moe_sort_small(idx, plan, row_pair, pair_row, experts, tile)
+    chosen, plan, row_pair, pair_row = (t.cpu().numpy() for t in (idx, plan, row_pair, pair_row))
+    counts = np.bincount(chosen[chosen < experts], minlength=experts)
+    tiles = -(-counts // tile)
+    assert plan[0] == tiles.sum() and plan[1:2 + experts].tolist() == np.concatenate([[0], np.cumsum(tiles)]).__mul__(tile).tolist()
+    assert plan[2 + experts:2 + experts + plan[0]].tolist() == np.repeat(np.arange(experts), tiles).tolist()
+    for i in range(pairs):
+        if chosen[i] == experts:
+            assert pair_row[i] == -1
+        else:
+            assert row_pair[pair_row[i]] == i and plan[2 + experts + pair_row[i] // tile] == chosen[i]
+    assert (row_pair >= 0).sum() == counts.sum() and (row_pair == -1).sum() == rows - counts.sum()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
