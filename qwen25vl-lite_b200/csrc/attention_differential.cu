@@ -370,28 +370,58 @@ __global__ void __launch_bounds__(128) diff_decode_kernel(DiffArgs a) {
   }
 }
 
-// Adds the key ranges of a token's maps up, in order, and finishes the heads: a warp per (item, head).
+// Adds the key ranges of a token's maps up, in order, and finishes the heads: a warp per (item, head), DV / 32 neighbouring
+// channels a lane.  A lane holds the (max, sum) of up to two ranges of each map; both maps' ranges are in flight together.
+#define DIFF_MAX_SPLITS 64
 template <int DV>
 __global__ void __launch_bounds__(128) diff_combine_kernel(DiffArgs a) {
   pdl_trigger();
   pdl_wait();
-  const int item = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5);
+  constexpr int CPL = DV / 32;
+  const int item = blockIdx.x, head = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (head >= a.heads) return;
   const int group = a.heads / a.nkv, kvh = head / group;
   const int token = a.cu_q[a.items[item]];
-  diff_finish_head<DV>(a, token, head, [&](int map, int c) {
-    const size_t base = ((size_t)item * 2 * a.heads + (kvh * 2 + map) * group + head % group) * a.n_splits;
-    float mm = -INFINITY;
-    for (int s = 0; s < a.n_splits; ++s) mm = fmaxf(mm, a.part_ml[(base + s) * 2]);
-    float sum = 0.f, acc = 0.f;
-    for (int s = 0; s < a.n_splits; ++s) {
-      const float ms = a.part_ml[(base + s) * 2];
-      const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
-      sum = fmaf(a.part_ml[(base + s) * 2 + 1], f, sum);
-      acc = fmaf(a.part_o[(base + s) * DV + c], f, acc);
+  float w[2][2], acc[2][CPL], inv[2];
+  size_t base[2];
+#pragma unroll
+  for (int map = 0; map < 2; ++map) {
+    base[map] = ((size_t)item * 2 * a.heads + (kvh * 2 + map) * group + head % group) * a.n_splits;
+    float2 ml[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = lane + 32 * i;
+      ml[i] = s < a.n_splits ? *reinterpret_cast<const float2*>(a.part_ml + (base[map] + s) * 2) : make_float2(-INFINITY, 0.f);
     }
-    return sum > 0.f ? acc / sum : 0.f;
-  });
+    const float mm = warp_max(fmaxf(ml[0].x, ml[1].x));
+#pragma unroll
+    for (int i = 0; i < 2; ++i) w[map][i] = ml[i].x == -INFINITY ? 0.f : exp2f(ml[i].x - mm);
+    const float sum = warp_sum(fmaf(ml[0].y, w[map][0], ml[1].y * w[map][1]));
+    inv[map] = sum > 0.f ? 1.0f / sum : 0.f;
+#pragma unroll
+    for (int c = 0; c < CPL; ++c) acc[map][c] = 0.f;
+  }
+#pragma unroll 4
+  for (int s = 0; s < a.n_splits; ++s)
+#pragma unroll
+    for (int map = 0; map < 2; ++map) {
+      const float f = __shfl_sync(0xffffffffu, s < 32 ? w[map][0] : w[map][1], s & 31);
+      const float* o = a.part_o + (base[map] + s) * DV + lane * CPL;
+      float v[CPL];
+      if constexpr (CPL == 4) { const float4 t = *reinterpret_cast<const float4*>(o); v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w; }
+      else if constexpr (CPL == 2) { const float2 t = *reinterpret_cast<const float2*>(o); v[0] = t.x; v[1] = t.y; }
+      else v[0] = o[0];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) acc[map][c] = fmaf(v[c], f, acc[map][c]);
+    }
+  float y[CPL], sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) { y[c] = acc[0][c] * inv[0] - a.lam * (acc[1][c] * inv[1]); sq = fmaf(y[c], y[c], sq); }
+  const float f = a.gain / sqrtf(warp_sum(sq) / (float)DV + a.eps);
+  const bf16* gate = (const bf16*)a.gate + (size_t)token * a.gate_stride + (size_t)head * DV + lane * CPL;
+  bf16* out = (bf16*)a.out + ((size_t)token * a.heads + head) * DV + lane * CPL;
+#pragma unroll
+  for (int c = 0; c < CPL; ++c) out[c] = __float2bfloat16_rn(y[c] * f * gate_one(gate + c));
 }
 
 template <int DK, int DV>
@@ -439,7 +469,7 @@ Q25_EXPORT int q25_differential_attention_mma_bf16(const void* q, int q_stride, 
                                                    int n_items, int heads, int nkv, int dk, int dv, int ps, int window, float scale, float lam, float gain,
                                                    float eps, int n_splits, float* part_o, float* part_ml, void* stream) {
   if (n_tiles <= 0 && n_items <= 0) return 0;
-  if (nkv <= 0 || heads <= 0 || heads % nkv || ps <= 0 || window < 0 || n_splits < 1 || (n_items > 0 && heads / nkv > 8) || q_stride % 2 || gate_stride % 2 ||
+  if (nkv <= 0 || heads <= 0 || heads % nkv || ps <= 0 || window < 0 || n_splits < 1 || n_splits > DIFF_MAX_SPLITS || (((uintptr_t)part_o | (uintptr_t)part_ml) & 15) || (n_items > 0 && heads / nkv > 8) || q_stride % 2 || gate_stride % 2 ||
       (((uintptr_t)q | (uintptr_t)gate | (uintptr_t)out) & 3) || (((uintptr_t)kp | (uintptr_t)vp) & 15) || (n_splits > 1 && (!part_o || !part_ml)))
     return (int)cudaErrorInvalidValue;
   DiffArgs a;
